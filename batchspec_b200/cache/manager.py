@@ -11,12 +11,16 @@ a windowed group also gives back pages that the window has passed (their table
 entries become -1; no kernel reads them), and a chunked group the pages before the
 chunk that the next position falls into.
 
+A mixer that also keeps one entry per whole block of P tokens (``CacheSpec.pool``) gets a second group for
+those: a request of length L has floor(L / P) entries there, kept while it lives, and its windowed group
+keeps the tokens of the block that is not yet whole, which its mean will need.
+
 The pool is zeroed once when it is made and never again: what a kernel loads past a request's length is
 masked, it only has to be finite.
 """
 from __future__ import annotations
 
-from dataclasses import dataclass, field
+from dataclasses import dataclass, field, replace
 from typing import Dict, List, Optional, Sequence, Tuple
 
 import torch
@@ -105,6 +109,7 @@ class CacheGroup:
     page_size: int
     pool: PagePool
     runs: List[int] = field(default_factory=list)        # indices into the model's order
+    stride: int = 1                            # tokens per entry (P in a group of pooled blocks)
     pages: Optional[torch.Tensor] = None       # [len(runs), num_pages, spec.tensors, page_size * entry_elems]
 
     @property
@@ -113,6 +118,10 @@ class CacheGroup:
         for s in self.spec.entry_shape:
             n *= s
         return n
+
+    def pages_for(self, length: int) -> int:
+        """Table entries of a request of ``length`` tokens: only whole blocks of ``stride`` tokens have an entry."""
+        return -(-(length // self.stride) // self.page_size)
 
 
 @dataclass
@@ -130,7 +139,8 @@ class CacheManager:
 
     ``page_size`` is the default tokens-per-page; a mixer's ``CacheSpec.page_size`` overrides it for its group.
     ``num_pages`` is the size of every group's pool in pages of the default size (a group with pages of its own
-    size gets as many as hold the same number of tokens), or a list with one count per group.
+    size gets as many as hold the same number of tokens; a group of pooled blocks as many as their entries need, and
+    one more per request), or a list with one count per group.
     ``allocate=False`` keeps the bookkeeping only (tests, planning)."""
 
     def __init__(self, needs, page_size: int, num_pages, max_requests: int, dtype: torch.dtype, device,
@@ -146,23 +156,33 @@ class CacheManager:
         self.requests: Dict[object, RequestCache] = {}
         key_to_group: Dict[Tuple, int] = {}
         run_group: Dict[int, Tuple[int, int]] = {}           # run -> (group, index in group)
+        run_pooled: Dict[int, Tuple[int, int]] = {}          # the same for the runs' pooled blocks
+
+        def join_group(run, c: CacheSpec, stride: int) -> Tuple[int, int]:
+            group_page = int(c.page_size or self.page_size)
+            key = (c.policy, c.window, tuple(c.entry_shape), c.tensors, group_page, c.pool, stride)
+            if key not in key_to_group:
+                key_to_group[key] = len(self.groups)
+                if isinstance(num_pages, (list, tuple)):
+                    n = num_pages[len(self.groups)]
+                else:                                        # the same number of tokens in this group's pages
+                    n = -(-num_pages * self.page_size // (group_page * stride)) + (self.max_requests if stride > 1 else 0)
+                self.groups.append(CacheGroup(c, group_page, PagePool(n, reserved=int(scratch_page)), stride=stride))
+            g = key_to_group[key]
+            self.groups[g].runs.append(run)
+            return g, len(self.groups[g].runs) - 1
+
         for e, need in enumerate(needs):
             if need.cache is None or need.cache_from is not None:
                 continue
             c = need.cache
             if c.tensors < 1 or (c.page_size is not None and c.page_size <= 0):
                 raise ValueError(f"run {e}: a cache entry has at least one tensor and a positive page size, got {c}")
-            group_page = int(c.page_size or self.page_size)
-            key = (c.policy, c.window, tuple(c.entry_shape), c.tensors, group_page)
-            if key not in key_to_group:
-                key_to_group[key] = len(self.groups)
-                n = num_pages[len(self.groups)] if isinstance(num_pages, (list, tuple)) else num_pages
-                if not isinstance(num_pages, (list, tuple)) and group_page != self.page_size:
-                    n = -(-n * self.page_size // group_page)         # the same number of tokens in pages of its own size
-                self.groups.append(CacheGroup(c, group_page, PagePool(n, reserved=int(scratch_page))))
-            g = key_to_group[key]
-            run_group[e] = (g, len(self.groups[g].runs))
-            self.groups[g].runs.append(e)
+            run_group[e] = join_group(e, c, 1)
+            if c.pool:
+                if c.pool < 0:
+                    raise ValueError(f"run {e}: a pooled block holds at least one token, got {c}")
+                run_pooled[e] = join_group(e, replace(c, policy="full", window=None, pool=0), c.pool)
         if allocate:
             for grp in self.groups:
                 # zeroed once: kernels may load (and mask) rows of a page that no token has been written to yet,
@@ -187,7 +207,10 @@ class CacheManager:
             if kv is None and state is None and need.cache is None and need.state is None:
                 self.layer_caches.append(None)
             else:
-                self.layer_caches.append(LayerCache(kv=kv, group=g, state=state, owner=need.cache_from is None))
+                pg, pidx = run_pooled.get(owner_run, (-1, 0))
+                self.layer_caches.append(LayerCache(kv=kv, group=g, state=state, owner=need.cache_from is None,
+                                                    pooled=self.groups[pg].pages[pidx] if allocate and pg >= 0 else None,
+                                                    pooled_group=pg))
 
     def page_bytes(self) -> int:
         """Bytes of all pools' page tensors (whether or not they were allocated)."""
@@ -227,7 +250,7 @@ class CacheManager:
 
     def pages_needed(self, length: int, n_new: int) -> List[int]:
         """Per group, the table entries a request of ``length`` tokens lacks for ``n_new`` more."""
-        return [-(-(length + n_new) // g.page_size) - (-(-length // g.page_size)) for g in self.groups]
+        return [g.pages_for(length + n_new) - g.pages_for(length) for g in self.groups]
 
     def peak_pages(self, total_len: int, portion: int) -> List[int]:
         """Per group, the most pages one request of ``total_len`` tokens holds at any time when it is fed in
@@ -237,9 +260,9 @@ class CacheManager:
         out = []
         for g in self.groups:
             ps = g.page_size
-            n = -(-total_len // ps)
+            n = g.pages_for(total_len)
             if g.spec.policy in ("window", "chunk"):
-                n = min(n, (g.spec.window - 1 + max(1, portion) + ps - 1) // ps + 1)
+                n = min(n, (max(g.spec.window, g.spec.pool) - 1 + max(1, portion) + ps - 1) // ps + 1)
             out.append(n)
         return out
 
@@ -247,7 +270,7 @@ class CacheManager:
         """Per group, the pages a live request still has to get before it can take n_new more tokens (pages it
         already holds beyond its length, from a reservation that was never committed, count as held)."""
         rc = self.requests[req_id]
-        return [max(0, -(-(rc.length + n_new) // g.page_size) - len(t)) for g, t in zip(self.groups, rc.tables)]
+        return [max(0, g.pages_for(rc.length + n_new) - len(t)) for g, t in zip(self.groups, rc.tables)]
 
     def free_pages(self) -> List[int]:
         return [g.pool.num_free for g in self.groups]
@@ -255,7 +278,8 @@ class CacheManager:
     def room_for(self, length: int, free: Sequence[int]) -> int:
         """How many more tokens a request of ``length`` tokens (holding exactly the pages of that length) can
         take with at most ``free[g]`` new pages of each group."""
-        return min((f * g.page_size + (-length) % g.page_size for g, f in zip(self.groups, free)), default=1 << 60)
+        return min((((g.pages_for(length) + f) * g.page_size + 1) * g.stride - 1 - length
+                    for g, f in zip(self.groups, free)), default=1 << 60)
 
     def can_reserve(self, demands: Sequence[Tuple[int, int]]) -> bool:
         """demands: (current length, new tokens) per request; True if every pool
@@ -284,9 +308,11 @@ class CacheManager:
         rc = self.requests[req_id]
         rc.length += n_new
         for gi, (g, table) in enumerate(zip(self.groups, rc.tables)):
-            assert len(table) == -(-rc.length // g.page_size), "block table out of step"
+            assert len(table) == g.pages_for(rc.length), "block table out of step"
             if g.spec.policy == "window":
                 first_needed = max(0, rc.length - g.spec.window + 1)
+                if g.spec.pool:
+                    first_needed = min(first_needed, rc.length // g.spec.pool * g.spec.pool)
             elif g.spec.policy == "chunk":
                 first_needed = (rc.length // g.spec.window) * g.spec.window      # start of the next position's chunk
             else:

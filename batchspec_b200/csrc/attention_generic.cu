@@ -15,6 +15,11 @@
 // a score s (after the scale) becomes c tanh(s / c).  ``v_is_k``: the values are the keys; a page then holds
 // [Hkv][page_size][hd] only.  ``gate`` (float32 rows [Hq*vd] of stride gate_stride, or null): the output is multiplied
 // element by element by sigmoid(gate); ``out_scale`` multiplies it too; output rows have stride out_stride.
+//
+// ``slopes`` (float32 per query head, or null): slope_h * (query - key) is taken off a token's score.  ``pool`` P > 0
+// (with a window W): before the window a query also sees one entry per block of P tokens that lies wholly before it,
+// floor((query - W + 1) / P) of them; they have pages and a table of their own (same page layout, entry b = block b)
+// and take part in the same softmax, first.
 #include "common.cuh"
 #include <math.h>
 using namespace bspec;
@@ -31,7 +36,9 @@ attn_generic_kernel(const T* __restrict__ q, long long q_row_stride, T* __restri
                     const int* __restrict__ kv_indices, int Hq, int Hkv, int hd, int page_size, float scale,
                     int window, long long n_pages, int vd, int chunk, const float* __restrict__ sink,
                     float softcap, int v_is_k, const float* __restrict__ gate, long long gate_stride,
-                    long long out_stride, float out_scale, int gate_per_head) {
+                    long long out_stride, float out_scale, int gate_per_head, const float* __restrict__ slopes,
+                    int pool, const T* __restrict__ pool_cache, const int* __restrict__ pool_indptr,
+                    const int* __restrict__ pool_indices, long long pool_pages) {
   bspec::pdl_prologue(7);
   __shared__ float qs[WARPS][MAX_HD];
   const int e = blockIdx.y, h = blockIdx.z;
@@ -61,22 +68,25 @@ attn_generic_kernel(const T* __restrict__ q, long long q_row_stride, T* __restri
 #pragma unroll
   for (int i = 0; i < ND; ++i) acc[i] = 0.f;
   float m = -INFINITY, l = 0.f;
-  for (int kb = (lo / 32) * 32; kb <= hi; kb += 32) {
+  const float slope = slopes != nullptr ? slopes[h] : 0.f;
+  // one chunk of 32 keys (of a request's tokens, or of its pooled blocks) into the running softmax
+  auto visit = [&](int kb, int lo_, int hi_, const int* tab, const T* base, long long pages, float bias_slope) {
     const int key = kb + lane;
-    bool valid = key >= lo && key <= hi;
+    bool valid = key >= lo_ && key <= hi_;
     long long koff = 0, voff = 0;
     float s = -INFINITY;
-    if (valid && !bspec::in_range(table[key / page_size], n_pages, 107)) valid = false;
+    if (valid && !bspec::in_range(tab[key / page_size], pages, 107)) valid = false;
     if (valid) {
-      const int page = table[key / page_size];
+      const int page = tab[key / page_size];
       koff = (long long)((size_t)page * page_elems + head_off + (size_t)(key % page_size) * hd);
       voff = v_is_k ? koff
                     : (long long)((size_t)page * page_elems + k_elems + ((size_t)kvh * page_size + (size_t)(key % page_size)) * vd);
-      const T* kp = cache + koff;
+      const T* kp = base + koff;
       float dot = 0.f;
       for (int d = 0; d < hd; ++d) dot += qs[warp][d] * to_f32(kp[d]);
       s = dot * scale;
       if (softcap > 0.f) s = softcap * tanhf(s / softcap);
+      if (bias_slope != 0.f) s -= bias_slope * (float)(pos - key);
     }
     const float m_new = fmaxf(m, warp_max(s));        // finite: the chunk holds at least one valid key
     const float p = valid ? expf(s - m_new) : 0.f;
@@ -84,12 +94,12 @@ attn_generic_kernel(const T* __restrict__ q, long long q_row_stride, T* __restri
     l = l * corr + warp_sum(p);
 #pragma unroll
     for (int i = 0; i < ND; ++i) acc[i] *= corr;
-    const int nk = min(32, hi - kb + 1);
+    const int nk = min(32, hi_ - kb + 1);
     for (int kk = 0; kk < nk; ++kk) {
       const float pk = __shfl_sync(0xffffffffu, p, kk);
       const long long off = __shfl_sync(0xffffffffu, voff, kk);
       if (pk != 0.f) {
-        const T* vp = cache + off;
+        const T* vp = base + off;
 #pragma unroll
         for (int i = 0; i < ND; ++i) {
           const int d = lane + 32 * i;
@@ -98,7 +108,13 @@ attn_generic_kernel(const T* __restrict__ q, long long q_row_stride, T* __restri
       }
     }
     m = m_new;
+  };
+  if (pool > 0) {
+    const int blocks = bspec::pooled_seen(pos, window, pool);
+    for (int kb = 0; kb < blocks; kb += 32)
+      visit(kb, 0, blocks - 1, pool_indices + pool_indptr[e], pool_cache, pool_pages, 0.f);
   }
+  for (int kb = (lo / 32) * 32; kb <= hi; kb += 32) visit(kb, lo, hi, table, cache, n_pages, slope);
   if (sink != nullptr) {                                // one more term of the denominator only
     const float sk = sink[h];
     const float m_new = fmaxf(m, sk);
@@ -131,8 +147,11 @@ static int launch_attention_generic(const void* q, long long q_row_stride, void*
                                     int page_size, float scale, int window, long long n_pages, int vd, int chunk,
                                     const float* sink, float softcap, int v_is_k, const float* gate,
                                     long long gate_stride, long long out_stride, float out_scale, int gate_per_head,
-                                    cudaStream_t stream) {
+                                    const float* slopes, int pool, const void* pool_cache, const int* pool_indptr,
+                                    const int* pool_indices, long long pool_pages, cudaStream_t stream) {
   if (n_entries <= 0 || max_q_len <= 0) return 0;
+  if (pool < 0 || (pool > 0 && (window <= 0 || v_is_k || pool_cache == nullptr || pool_indptr == nullptr)))
+    return (int)cudaErrorInvalidValue;
   if (v_is_k && vd != hd) return (int)cudaErrorInvalidValue;
   if (hd > MAX_HD || hd <= 0 || vd > MAX_HD || vd <= 0 || Hq % Hkv != 0) return (int)cudaErrorInvalidValue;
   dim3 grid((max_q_len + WARPS - 1) / WARPS, n_entries, Hq);
@@ -141,12 +160,13 @@ static int launch_attention_generic(const void* q, long long q_row_stride, void*
     BSPEC_LAUNCH((attn_generic_kernel<float>), grid, WARPS * 32, 0, stream, 
         (const float*)q, q_row_stride, (float*)out, (const float*)cache, qo_indptr, positions, kv_indptr, kv_indices,
         Hq, Hkv, hd, page_size, scale, window, n_pages, vd, chunk, sink, softcap, v_is_k, gate, gate_stride, out_stride,
-        out_scale, gate_per_head);
+        out_scale, gate_per_head, slopes, pool, (const float*)pool_cache, pool_indptr, pool_indices, pool_pages);
   else
     BSPEC_LAUNCH((attn_generic_kernel<__nv_bfloat16>), grid, WARPS * 32, 0, stream, 
         (const __nv_bfloat16*)q, q_row_stride, (__nv_bfloat16*)out, (const __nv_bfloat16*)cache, qo_indptr, positions,
         kv_indptr, kv_indices, Hq, Hkv, hd, page_size, scale, window, n_pages, vd, chunk, sink, softcap, v_is_k, gate,
-        gate_stride, out_stride, out_scale, gate_per_head);
+        gate_stride, out_stride, out_scale, gate_per_head, slopes, pool, (const __nv_bfloat16*)pool_cache, pool_indptr,
+        pool_indices, pool_pages);
   return BSPEC_LAUNCH_CHECK();
 }
 
@@ -157,21 +177,27 @@ BSPEC_API int bspec_attention_generic(const void* q, long long q_row_stride, voi
                                       cudaStream_t stream) {
   return launch_attention_generic(q, q_row_stride, out, cache, dtype, qo_indptr, positions, kv_indptr, kv_indices,
                                   n_entries, max_q_len, Hq, Hkv, hd, page_size, scale, window, n_pages, hd, 0, nullptr,
-                                  0.f, 0, nullptr, 0, (long long)Hq * hd, 1.f, 0, stream);
+                                  0.f, 0, nullptr, 0, (long long)Hq * hd, 1.f, 0, nullptr, 0, nullptr, nullptr, nullptr,
+                                  0, stream);
 }
 
 // The same with values of their own size ``vd``, a chunk mask (0: none), a sink per query head (null: none), a soft
-// cap on the scores (0: none), values that are the keys, a sigmoid gate on the output (per number, or per head), an output scale and stride.
+// cap on the scores (0: none), values that are the keys, a sigmoid gate on the output (per number, or per head), an
+// output scale and stride, a distance bias (slopes per query head, null: none) and pooled blocks before the window
+// (0: none).
 BSPEC_API int bspec_attention_masked(const void* q, long long q_row_stride, void* out, const void* cache, int dtype,
                                      const int* qo_indptr, const int* positions, const int* kv_indptr,
                                      const int* kv_indices, int n_entries, int max_q_len, int Hq, int Hkv, int hd,
                                      int vd, int page_size, float scale, int window, int chunk, const float* sink,
                                      long long n_pages, float softcap, int v_is_k, const float* gate,
                                      long long gate_stride, long long out_stride, float out_scale,
-                                     int gate_per_head, cudaStream_t stream) {
+                                     int gate_per_head, const float* slopes, int pool, const void* pool_cache,
+                                     const int* pool_indptr, const int* pool_indices, long long pool_pages,
+                                     cudaStream_t stream) {
   return launch_attention_generic(q, q_row_stride, out, cache, dtype, qo_indptr, positions, kv_indptr, kv_indices,
                                   n_entries, max_q_len, Hq, Hkv, hd, page_size, scale, window, n_pages, vd, chunk, sink,
-                                  softcap, v_is_k, gate, gate_stride, out_stride, out_scale, gate_per_head, stream);
+                                  softcap, v_is_k, gate, gate_stride, out_stride, out_scale, gate_per_head, slopes, pool,
+                                  pool_cache, pool_indptr, pool_indices, pool_pages, stream);
 }
 
 // ---------------------------------------------------------------- q/k/v preparation
@@ -181,9 +207,28 @@ BSPEC_API int bspec_attention_masked(const void* q, long long q_row_stride, void
 // a weight per number of a head, when given; before the rotation with ``norm_first``),
 // all in float32; then write q to ``q_out`` [n, Hq*hd] and k and v into the cache page of the token's position.
 // Rows of the input have stride ``ld`` (they may hold more columns).  vd == 0: there are no values (they are the
-// keys); a page then holds keys only.  One warp per head.
+// keys); a page then holds keys only.  One warp per head.  ``pool`` P > 0 (only for steps whose entries have one token
+// each): a token that completes a block of P also leaves the block's mean key and value, of the rows as the cache
+// holds them, in the pooled pages; larger portions take ``pool_append`` below after this kernel.
 namespace {
 constexpr int PREP_WARPS = 8;
+
+// Mean over the ``pool`` rows (from position p0, pages through ``table``) of one column of a kv head, in row order:
+// float32 sum, one division, the cache's rounding.  ``part``: the column's offset in a page's row 0, ``width`` the
+// distance from row to row.
+template <typename T>
+__device__ __forceinline__ float pooled_mean(const T* __restrict__ cache, const int* __restrict__ table, size_t page_elems,
+                                             size_t part, int width, int p0, int pool, int page_size,
+                                             long long n_pages) {
+  float s = 0.f;
+#pragma unroll 4
+  for (int r = 0; r < pool; ++r) {
+    const int p = p0 + r, page = table[p / page_size];
+    if (bspec::in_range(page, n_pages, 116))
+      s += to_f32(cache[(size_t)page * page_elems + part + (size_t)(p % page_size) * width]);
+  }
+  return s / (float)pool;
+}
 
 __device__ __forceinline__ void prep_sincos(int pos, const float* __restrict__ inv_freq, int half, int j, float* s,
                                             float* c) {
@@ -212,7 +257,8 @@ qkv_prepare_kernel(const float* __restrict__ qkv, long long ld, int Hq, int Hkv,
                    const int* __restrict__ kv_indptr, const int* __restrict__ kv_indices, T* __restrict__ q_out,
                    T* __restrict__ cache, int page_size, int write_kv, long long n_pages,
                    const void* __restrict__ q_norm_w, const void* __restrict__ k_norm_w, int norm_w_dtype,
-                   int norm_first) {
+                   int norm_first, int pool, T* __restrict__ pool_cache, const int* __restrict__ pool_indptr,
+                   const int* __restrict__ pool_indices, long long pool_pages) {
   bspec::pdl_prologue(19);
   __shared__ __align__(16) float xs[PREP_WARPS][MAX_HD];
   __shared__ float cs[MAX_HD];                                // [rot/2] cosines, then [rot/2] sines, of this token
@@ -316,16 +362,84 @@ qkv_prepare_kernel(const float* __restrict__ qkv, long long ld, int Hq, int Hkv,
       for (int d = lane; d < width; d += 32) dst[d] = from_f32<T>(x[d] * r);
     }
   }
+  if (pool > 0 && dst != nullptr && slot >= Hq && (pos + 1) % pool == 0) {
+    // this token completes its block, and the block's other rows are of earlier steps
+    __syncwarp();                                            // the row just written is read back by other lanes
+    const int e = tok_entry[t], b = pos / pool;
+    const int* ptab = pool_indices + pool_indptr[e];
+    const size_t k_elems = (size_t)Hkv * page_size * hd, page_elems = k_elems + (size_t)Hkv * page_size * vd;
+    const size_t head = is_v ? k_elems + (size_t)(slot - Hq - Hkv) * page_size * vd : (size_t)(slot - Hq) * page_size * hd;
+    if (bspec::in_range(b / page_size, pool_indptr[e + 1] - pool_indptr[e], 117) &&
+        bspec::in_range(ptab[b / page_size], pool_pages, 118)) {
+      T* to = pool_cache + (size_t)ptab[b / page_size] * page_elems + head + (size_t)(b % page_size) * width;
+      for (int d = lane; d < width; d += 32)
+        to[d] = from_f32<T>(pooled_mean<T>(cache, kv_indices + kv_indptr[e], page_elems, head + d, width, b * pool, pool,
+                                           page_size, n_pages));
+    }
+  }
+}
+
+// The pooled entries of the blocks that a step's portions complete: block (x, e, z) takes the x-th such block of
+// entry e; a thread per column of [k of every kv head | v of every kv head].
+template <typename T>
+__global__ void __launch_bounds__(256)
+pool_append_kernel(const T* __restrict__ cache, const int* __restrict__ qo_indptr, const int* __restrict__ positions,
+                   const int* __restrict__ kv_indptr, const int* __restrict__ kv_indices, T* __restrict__ pool_cache,
+                   const int* __restrict__ pool_indptr, const int* __restrict__ pool_indices, int Hkv, int hd, int vd,
+                   int page_size, int pool, long long n_pages, long long pool_pages) {
+  bspec::pdl_prologue(21);
+  const int e = blockIdx.y;
+  const int t0 = qo_indptr[e], nt = qo_indptr[e + 1] - t0;
+  if (nt <= 0) return;
+  const int pos0 = positions[t0];
+  const int b = pos0 / pool + (int)blockIdx.x;
+  if ((long long)(b + 1) * pool > pos0 + nt) return;
+  const int col = blockIdx.z * blockDim.x + threadIdx.x;
+  if (col >= Hkv * (hd + vd)) return;
+  const bool is_v = col >= Hkv * hd;
+  const int width = is_v ? vd : hd, c = is_v ? col - Hkv * hd : col;
+  const int g = c / width, d = c - g * width;
+  const size_t k_elems = (size_t)Hkv * page_size * hd, page_elems = k_elems + (size_t)Hkv * page_size * vd;
+  const size_t head = (is_v ? k_elems : (size_t)0) + (size_t)g * page_size * width;
+  const int* ptab = pool_indices + pool_indptr[e];
+  if (!bspec::in_range(b / page_size, pool_indptr[e + 1] - pool_indptr[e], 117) ||
+      !bspec::in_range(ptab[b / page_size], pool_pages, 118))
+    return;
+  pool_cache[(size_t)ptab[b / page_size] * page_elems + head + (size_t)(b % page_size) * width + d] =
+      from_f32<T>(pooled_mean<T>(cache, kv_indices + kv_indptr[e], page_elems, head + d, width, b * pool, pool,
+                                 page_size, n_pages));
 }
 }  // namespace
+
+// Portions of any length; max_q_len: the longest of the step.
+BSPEC_API int bspec_pool_append(const void* cache, int dtype, const int* qo_indptr, const int* positions,
+                                const int* kv_indptr, const int* kv_indices, void* pool_cache, const int* pool_indptr,
+                                const int* pool_indices, int n_entries, int max_q_len, int Hkv, int hd, int vd,
+                                int page_size, int pool, long long n_pages, long long pool_pages, cudaStream_t stream) {
+  if (n_entries <= 0 || max_q_len <= 0) return 0;
+  if (pool <= 0 || Hkv <= 0 || hd <= 0 || vd < 0 || page_size <= 0 || n_entries > 65535) return (int)cudaErrorInvalidValue;
+  const dim3 grid((max_q_len + pool - 1) / pool, n_entries, (Hkv * (hd + vd) + 255) / 256);
+  if (grid.z > 65535) return (int)cudaErrorInvalidConfiguration;
+  if (dtype == BSPEC_F32)
+    BSPEC_LAUNCH((pool_append_kernel<float>), grid, 256, 0, stream, (const float*)cache, qo_indptr, positions, kv_indptr,
+                 kv_indices, (float*)pool_cache, pool_indptr, pool_indices, Hkv, hd, vd, page_size, pool, n_pages, pool_pages);
+  else
+    BSPEC_LAUNCH((pool_append_kernel<__nv_bfloat16>), grid, 256, 0, stream, (const __nv_bfloat16*)cache, qo_indptr,
+                 positions, kv_indptr, kv_indices, (__nv_bfloat16*)pool_cache, pool_indptr, pool_indices, Hkv, hd, vd,
+                 page_size, pool, n_pages, pool_pages);
+  return BSPEC_LAUNCH_CHECK();
+}
 
 BSPEC_API int bspec_qkv_prepare(const float* qkv, long long ld, int n, int Hq, int Hkv, int hd, int vd, const void* bias,
                                 int bias_dtype, const float* inv_freq, int rot, int interleaved, float magnitude,
                                 float norm_eps, const int* positions, const int* tok_entry, const int* kv_indptr,
                                 const int* kv_indices, void* q_out, void* cache, int dtype, int page_size, int write_kv,
                                 long long n_pages, const void* q_norm_w, const void* k_norm_w, int norm_w_dtype,
-                                int norm_first, cudaStream_t stream) {
+                                int norm_first, int pool, void* pool_cache, const int* pool_indptr,
+                                const int* pool_indices, long long pool_pages, cudaStream_t stream) {
   if (n <= 0) return 0;
+  if (pool < 0 || (pool > 0 && (pool_cache == nullptr || pool_indptr == nullptr || !write_kv)))
+    return (int)cudaErrorInvalidValue;
   if (hd <= 0 || hd > MAX_HD || vd < 0 || vd > MAX_HD || ld < (long long)(Hq + Hkv) * hd + (long long)Hkv * vd || rot < 0 || rot > hd || rot % 2 != 0 ||
       (rot > 0 && inv_freq == nullptr))
     return (int)cudaErrorInvalidValue;
@@ -334,12 +448,13 @@ BSPEC_API int bspec_qkv_prepare(const float* qkv, long long ld, int n, int Hq, i
   if (dtype == BSPEC_F32)
     BSPEC_LAUNCH((qkv_prepare_kernel<float>), grid, PREP_WARPS * 32, 0, stream, qkv, ld, Hq, Hkv, hd, vd, bias, bias_dtype,
                  inv_freq, rot, interleaved, magnitude, norm_eps, positions, tok_entry, kv_indptr, kv_indices,
-                 (float*)q_out, (float*)cache, page_size, write_kv, n_pages, q_norm_w, k_norm_w, norm_w_dtype, norm_first);
+                 (float*)q_out, (float*)cache, page_size, write_kv, n_pages, q_norm_w, k_norm_w, norm_w_dtype, norm_first,
+                 pool, (float*)pool_cache, pool_indptr, pool_indices, pool_pages);
   else
     BSPEC_LAUNCH((qkv_prepare_kernel<__nv_bfloat16>), grid, PREP_WARPS * 32, 0, stream, qkv, ld, Hq, Hkv, hd, vd, bias,
                  bias_dtype, inv_freq, rot, interleaved, magnitude, norm_eps, positions, tok_entry, kv_indptr,
                  kv_indices, (__nv_bfloat16*)q_out, (__nv_bfloat16*)cache, page_size, write_kv, n_pages, q_norm_w, k_norm_w,
-                 norm_w_dtype, norm_first);
+                 norm_w_dtype, norm_first, pool, (__nv_bfloat16*)pool_cache, pool_indptr, pool_indices, pool_pages);
   return BSPEC_LAUNCH_CHECK();
 }
 

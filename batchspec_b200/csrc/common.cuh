@@ -43,6 +43,11 @@ __device__ __forceinline__ float warp_max(float v) {
 __device__ __forceinline__ int mask_lo(int pos, int window) {
   return window > 0 ? max(0, pos - window + 1) : (window < 0 ? (pos / -window) * -window : 0);
 }
+// Blocks of ``pool`` positions that lie wholly before the window of a query at ``pos``: block b is seen when its last
+// position b pool + pool - 1 is at most pos - window.
+__device__ __forceinline__ int pooled_seen(int pos, int window, int pool) {
+  return pos - window + 1 > 0 ? (pos - window + 1) / pool : 0;
+}
 // A softmax sink is a logit per head that adds exp(sink) to the denominator and nothing to the numerator.  With the running maximum ``m`` and sum ``l``
 // in base-2 units and ``sink_l2`` = sink * log2(e) per query head (null: none): the sum with the sink's term.
 __device__ __forceinline__ float with_sink(float l, float m, const float* __restrict__ sink_l2, int h) {
@@ -106,7 +111,8 @@ __device__ __forceinline__ void trace_mark(int kid, unsigned long long t_from) {
 // {code, value, limit, block} and the access is skipped: a wrong table then costs a wrong result and a report,
 // not a fault.  Each translation unit has its own record; BSPEC_DEFINE_BOUNDS_REPORT exports its reader.
 // Codes: 101 token id (embedding), 102 row (gather), 103 block-table slot and 104 page id (rotary + cache append),
-// 105 / 106 the same in the q/k/v product's epilogue, 107 / 108 page id (attention over plain loads, float32 / bfloat16).  Copies through
+// 105 / 106 the same in the q/k/v product's epilogue, 107 / 108 page id (attention over plain loads, float32 / bfloat16),
+// 115 row (branch join), 116 page id of a block's rows, 117 / 118 block-table slot and page id of a pooled entry.  Copies through
 // TMA need no such check: the tensor map clips them.
 #ifdef BSPEC_BOUNDS
 static __device__ int g_bounds[4] = {0, 0, 0, 0};

@@ -314,7 +314,7 @@ delta_recurrence_kernel(const float* __restrict__ mix, const float* __restrict__
 }
 
 // out[t, h*V + j] = o[t, h, j] / sqrt(mean_j o^2 + eps) * w[j] * act(gate[t, h*V + j]), act = silu (gate_kind 0) or
-// sigmoid (1); one warp per (token, head).
+// sigmoid (1), w null: no weight; one warp per (token, head).
 template <typename T>
 __global__ void __launch_bounds__(128)
 gated_rmsnorm_kernel(const float* __restrict__ o, const float* __restrict__ gate, long long gate_stride,
@@ -331,7 +331,7 @@ gated_rmsnorm_kernel(const float* __restrict__ o, const float* __restrict__ gate
   const float r = 1.f / sqrtf(ss / (float)V + eps);
   const float* gp = gate + (size_t)t * gate_stride + (size_t)h * V;
   T* op = out + ((size_t)t * H + h) * V;
-  for (int j = lane; j < V; j += 32) op[j] = from_f32<T>(x[j] * r * load_as_f32(w, w_dtype, j) * (gate_kind == 1 ? 1.f / (1.f + expf(-gp[j])) : silu_f(gp[j])));
+  for (int j = lane; j < V; j += 32) op[j] = from_f32<T>(x[j] * r * (w != nullptr ? load_as_f32(w, w_dtype, j) : 1.f) * (gate_kind == 1 ? 1.f / (1.f + expf(-gp[j])) : silu_f(gp[j])));
 }
 
 // The same for wide groups (all heads normed together: V in the thousands), where a warp per group would leave a
@@ -359,7 +359,7 @@ gated_rmsnorm_wide_kernel(const float* __restrict__ o, const float* __restrict__
   const float* gp = gate + (size_t)t * gate_stride + (size_t)h * V;
   T* op = out + ((size_t)t * H + h) * V;
   for (int j = threadIdx.x; j < V; j += 256)
-    op[j] = from_f32<T>(x[j] * r * load_as_f32(w, w_dtype, j) * (gate_kind == 1 ? 1.f / (1.f + expf(-gp[j])) : silu_f(gp[j])));
+    op[j] = from_f32<T>(x[j] * r * (w != nullptr ? load_as_f32(w, w_dtype, j) : 1.f) * (gate_kind == 1 ? 1.f / (1.f + expf(-gp[j])) : silu_f(gp[j])));
 }
 }  // namespace
 

@@ -6,14 +6,17 @@
 //             groups stay (the others count as minus infinity); the `top` largest choices are taken, ties to the
 //             lower index; weights = s of the chosen * scale (no renormalisation).  With `softmax_top` instead:
 //             choice = z + bias (the `correction` tensor), the `top` largest are taken, and the weights are the
-//             softmax over the chosen logits alone
+//             softmax over the chosen logits alone.  Or with softmax scores: s = softmax(z) over all experts, choice =
+//             s + correction.  A group's score may also be its largest choice, and the weights may be divided by
+//             their sum (+ 1e-20) before `scale`
 //   plan      one block: counts per expert, a stable counting sort of the n*top slots by expert (row r of the
 //             sorted order holds slot perm[r]; inv[slot] = r), and the list of row tiles (expert, first row, rows)
 //   grouped   C[r, :] = act(A[src(r), :] . W[expert(r)]^T) over the tiles of the plan; every output element is one
 //             thread's sum over k in ascending order, so a row's result does not depend on where it was sorted to
 //             (act: GELU on the outputs, or none; the operand A may be gated instead: its rows are [gate | up] and
 //             silu(gate) * up is formed while they are staged, which is how gated experts run their down projection)
-//   combine   out[t, :] = sum_k weight[t, k] * Y[inv[t*top + k], :], k ascending, float32
+//   combine   out[t, :] = add[t, :] + sum_k weight[t, k] * Y[inv[t*top + k], :], k ascending, float32 (``add``: a
+//             shared expert's rows, or none)
 //
 // Nothing here reads a count on the host: grids are sized by upper bounds and surplus blocks leave at once, so the
 // kernels can be captured in a graph.
@@ -24,14 +27,19 @@ using namespace bspec;
 namespace {
 
 constexpr int ROUTE_THREADS = 128;
+// the router's rule: bits 0-1 what the scores are, then options
+constexpr int ROUTE_SIGMOID = 0, ROUTE_SOFTMAX_TOP = 1, ROUTE_SOFTMAX = 2, ROUTE_SCORES = 3;
+constexpr int ROUTE_GROUP_MAX = 4, ROUTE_RENORMALISE = 8;
 constexpr int MAX_EXPERTS = 1024;
 
 template <typename T>
 __global__ void __launch_bounds__(ROUTE_THREADS)
 moe_route_kernel(const T* __restrict__ h, int d, const T* __restrict__ wr, const void* __restrict__ corr,
                  int corr_dtype, int E, int G, int keep, int top, float scale, int* __restrict__ ids,
-                 float* __restrict__ wts, const float* __restrict__ logits, int softmax_top) {
+                 float* __restrict__ wts, const float* __restrict__ logits, int rule) {
   bspec::pdl_prologue(50);
+  const int scores = rule & ROUTE_SCORES;
+  const bool softmax_top = scores == ROUTE_SOFTMAX_TOP;
   extern __shared__ float sm[];
   float* hs = sm;                 // [d]
   float* sc = hs + d;             // [E] sigmoid scores
@@ -40,7 +48,7 @@ moe_route_kernel(const T* __restrict__ h, int d, const T* __restrict__ wr, const
   if (logits != nullptr) {            // the logits were formed by a matrix product (many tokens)
     for (int e = threadIdx.x; e < E; e += blockDim.x) {
       const float z = logits[(size_t)t * E + e], b = corr != nullptr ? load_as_f32(corr, corr_dtype, e) : 0.f;
-      const float s = softmax_top ? z + b : 1.f / (1.f + expf(-z));
+      const float s = softmax_top ? z + b : (scores == ROUTE_SOFTMAX ? z : 1.f / (1.f + expf(-z)));
       sc[e] = s;
       ch[e] = softmax_top ? s : s + b;
     }
@@ -54,7 +62,7 @@ moe_route_kernel(const T* __restrict__ h, int d, const T* __restrict__ wr, const
       z = warp_sum(z);
       if (lane == 0) {
         const float b = corr != nullptr ? load_as_f32(corr, corr_dtype, e) : 0.f;
-        const float s = softmax_top ? z + b : 1.f / (1.f + expf(-z));
+        const float s = softmax_top ? z + b : (scores == ROUTE_SOFTMAX ? z : 1.f / (1.f + expf(-z)));
         sc[e] = s;
         ch[e] = softmax_top ? s : s + b;
       }
@@ -62,6 +70,19 @@ moe_route_kernel(const T* __restrict__ h, int d, const T* __restrict__ wr, const
   }
   __syncthreads();
   if (warp != 0) return;
+  if (scores == ROUTE_SOFTMAX) {
+    float mx = -INFINITY, sum = 0.f;
+    for (int i = lane; i < E; i += 32) mx = fmaxf(mx, sc[i]);
+    mx = warp_max(mx);
+    for (int i = lane; i < E; i += 32) sum += expf(sc[i] - mx);
+    sum = warp_sum(sum);
+    // without a correction the logits themselves choose (the softmax keeps their order)
+    for (int i = lane; i < E; i += 32) {
+      sc[i] = expf(sc[i] - mx) / sum;
+      if (corr != nullptr) ch[i] = sc[i] + load_as_f32(corr, corr_dtype, i);
+    }
+    __syncwarp();
+  }
   // The choice is made by warp 0: every lane scans its share of the candidates, a shuffle tree finds the best
   // (the larger value, the lower index among equals), lane 0 marks it as taken (NaN).
   auto best_of = [&](const float* v, int n) -> int {
@@ -87,7 +108,7 @@ moe_route_kernel(const T* __restrict__ h, int d, const T* __restrict__ wr, const
         const float v = ch[g * per + j];
         if (v > a) { b = a; a = v; } else if (v > b) { b = v; }
       }
-      hs[g] = per > 1 ? a + b : a;
+      hs[g] = per > 1 && !(rule & ROUTE_GROUP_MAX) ? a + b : a;
     }
     __syncwarp();
     for (int k = 0; k < keep; ++k) {
@@ -108,6 +129,12 @@ moe_route_kernel(const T* __restrict__ h, int d, const T* __restrict__ wr, const
       ch[best] = NAN;                             // taken
     }
     __syncwarp();
+  }
+  if ((rule & ROUTE_RENORMALISE) && !softmax_top && lane == 0) {
+    float* w = wts + (size_t)t * top;
+    float sum = 0.f;
+    for (int k = 0; k < top; ++k) sum += sc[ids[(size_t)t * top + k]];
+    for (int k = 0; k < top; ++k) w[k] = sc[ids[(size_t)t * top + k]] / (sum + 1e-20f) * scale;
   }
   if (softmax_top && lane == 0) {                 // the weights: softmax over the chosen logits alone
     float* w = wts + (size_t)t * top;
@@ -494,11 +521,15 @@ __global__ void moe_gather_kernel(const T* __restrict__ h, const int* __restrict
 
 template <typename TY, typename TO>
 __global__ void moe_combine_kernel(const TY* __restrict__ y, const int* __restrict__ inv, const float* __restrict__ wts,
-                                   int top, TO* __restrict__ out, int d) {
+                                   int top, TO* __restrict__ out, int d, const TO* __restrict__ add) {
   bspec::pdl_prologue(54);
   const int t = blockIdx.x;
   for (int i = 2 * threadIdx.x; i < d; i += 2 * blockDim.x) {
     float a0 = 0.f, a1 = 0.f;
+    if (add != nullptr) {
+      a0 = to_f32(add[(size_t)t * d + i]);
+      if (i + 1 < d) a1 = to_f32(add[(size_t)t * d + i + 1]);
+    }
     const bool pair = i + 1 < d && (d % 2) == 0;
     for (int k = 0; k < top; ++k) {
       const float w = wts[(size_t)t * top + k];
@@ -516,7 +547,7 @@ __global__ void moe_combine_kernel(const TY* __restrict__ y, const int* __restri
 
 BSPEC_API int bspec_moe_route(const void* h, int dtype, int n, int d, const void* wr, const void* corr, int corr_dtype,
                               int E, int G, int keep, int top, float scale, int* ids, float* wts,
-                              const float* logits, int softmax_top, cudaStream_t stream) {
+                              const float* logits, int rule, cudaStream_t stream) {
   if (n <= 0) return 0;
   if (E <= 0 || E > MAX_EXPERTS || top <= 0 || top > E || G <= 0 || E % G || keep <= 0 || keep > G ||
       (long long)keep * (E / G) < top)
@@ -526,11 +557,11 @@ BSPEC_API int bspec_moe_route(const void* h, int dtype, int n, int d, const void
   if (dtype == BSPEC_F32) {
     if (smem > 48 * 1024) cudaFuncSetAttribute(moe_route_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     BSPEC_LAUNCH((moe_route_kernel<float>), n, ROUTE_THREADS, smem, stream, (const float*)h, d, (const float*)wr, corr,
-                 corr_dtype, E, G, keep, top, scale, ids, wts, logits, softmax_top);
+                 corr_dtype, E, G, keep, top, scale, ids, wts, logits, rule);
   } else {
     if (smem > 48 * 1024) cudaFuncSetAttribute(moe_route_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     BSPEC_LAUNCH((moe_route_kernel<__nv_bfloat16>), n, ROUTE_THREADS, smem, stream, (const __nv_bfloat16*)h, d,
-                 (const __nv_bfloat16*)wr, corr, corr_dtype, E, G, keep, top, scale, ids, wts, logits, softmax_top);
+                 (const __nv_bfloat16*)wr, corr, corr_dtype, E, G, keep, top, scale, ids, wts, logits, rule);
   }
   return BSPEC_LAUNCH_CHECK();
 }
@@ -637,10 +668,10 @@ BSPEC_API int bspec_moe_gather(const void* h, int dtype, const int* perm, int to
 }
 
 BSPEC_API int bspec_moe_combine(const void* y, int y_dtype, const int* inv, const float* wts, int top, void* out,
-                                int out_dtype, int n, int d, cudaStream_t stream) {
+                                int out_dtype, int n, int d, const void* add, cudaStream_t stream) {
   if (n <= 0) return 0;
   const int threads = d >= 1024 ? 256 : 128;
-#define LC(TY, TO) BSPEC_LAUNCH((moe_combine_kernel<TY, TO>), n, threads, 0, stream, (const TY*)y, inv, wts, top, (TO*)out, d)
+#define LC(TY, TO) BSPEC_LAUNCH((moe_combine_kernel<TY, TO>), n, threads, 0, stream, (const TY*)y, inv, wts, top, (TO*)out, d, (const TO*)add)
   if (y_dtype == BSPEC_F32 && out_dtype == BSPEC_F32) LC(float, float);
   else if (y_dtype == BSPEC_F32) LC(float, __nv_bfloat16);
   else if (out_dtype == BSPEC_F32) LC(__nv_bfloat16, float);

@@ -2,7 +2,8 @@
 //
 //   lightning_recurrence   linear attention with a fixed decay per head:
 //                              S <- decay_h S + k v^T,  o = S^T q        S: [dim x vdim] per head
-//                          q, k, v are the silu of float32 projection columns.
+//                          q, k, v are float32 projection columns, through silu or as they are; q and k may be
+//                          rotated by position (pairs i, i + rot/2) and k multiplied by a constant.
 //   scan_conv              short causal convolution per channel with bias, then silu (inputs before the portion come
 //                          from the request's state)
 //   selective_scan         per channel c and state n:  S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c x_c B_n,
@@ -34,6 +35,15 @@ __device__ __forceinline__ float scan_update(float s, float x, float b) {
   return __fadd_rn(s, __fmaf_rn(exp_minus_one(x), s, b));
 }
 
+// The angle position * frequency in float64 (the table holds a frequency as two float32 parts), reduced to [-pi, pi].
+__device__ __forceinline__ void rotation_sincos(int pos, const float* __restrict__ inv_freq, int half, int j, float* s,
+                                                float* c) {
+  const double f = (double)inv_freq[j] + (double)inv_freq[half + j];
+  double a = (double)pos * f;
+  a -= 6.283185307179586476925286766559 * rint(a * 0.15915494309189533576888376337251);
+  sincosf((float)a, s, c);
+}
+
 // ---------------------------------------------------------------- lightning attention
 // Block: COLS value columns of one head of one request, L lanes per column (8, 16 or 32: more lanes mean more warps
 // per SM to hide the chain's latencies, and fewer rows per lane); lane r of a column keeps rows
@@ -52,7 +62,8 @@ __global__ void __launch_bounds__(LT_COLS * L)
 lightning_recurrence_kernel(const float* __restrict__ proj, long long ld, int q_off, int k_off, int v_off,
                             const float* __restrict__ decay, float* __restrict__ state, long long state_stride,
                             const int* __restrict__ qo_indptr, const int* __restrict__ state_slots,
-                            float* __restrict__ out, int H, int dim, int vdim) {
+                            float* __restrict__ out, int H, int dim, int vdim, int act, float k_scale,
+                            const float* __restrict__ inv_freq, int rot, const int* __restrict__ positions) {
   bspec::pdl_prologue_late(65);
   constexpr int LT_THREADS = LT_COLS * L;
   constexpr int DM = L * NR;                                // rows of S this instance holds (dim <= DM)
@@ -115,15 +126,29 @@ lightning_recurrence_kernel(const float* __restrict__ proj, long long ld, int q_
     for (int u = 0; u < NR; ++u) {                           // rows of tokens beyond cnt are never read
       const int x = threadIdx.x + LT_THREADS * u;
       if (x / DM >= cnt) break;
-      qs[x / DM][x % DM] = silu_f(qn[u]);                    // silu(0) = 0: rows beyond dim
-      ks[x / DM][x % DM] = silu_f(kn[u]);
+      qs[x / DM][x % DM] = act ? silu_f(qn[u]) : qn[u];      // silu(0) = 0: rows beyond dim
+      ks[x / DM][x % DM] = (act ? silu_f(kn[u]) : kn[u]) * k_scale;
     }
 #pragma unroll
     for (int u = 0; u < VR; ++u) {
       const int x = threadIdx.x + LT_THREADS * u;
-      if (x < LT_TT * LT_COLS && x / LT_COLS < cnt) vs[x / LT_COLS][x % LT_COLS] = silu_f(vn[u]);
+      if (x < LT_TT * LT_COLS && x / LT_COLS < cnt) vs[x / LT_COLS][x % LT_COLS] = act ? silu_f(vn[u]) : vn[u];
     }
     __syncthreads();
+    if (rot > 0) {                                           // the same for every block of a head: meant for a few tokens
+      const int half = rot / 2;
+      for (int x = threadIdx.x; x < cnt * half; x += LT_THREADS) {
+        const int tt = x / half, i = x - tt * half;
+        float sn, c;
+        rotation_sincos(positions[t0 + base + tt], inv_freq, half, i, &sn, &c);
+        const float qu = qs[tt][i], qv = qs[tt][i + half], ku = ks[tt][i], kv = ks[tt][i + half];
+        qs[tt][i] = qu * c - qv * sn;
+        qs[tt][i + half] = qv * c + qu * sn;
+        ks[tt][i] = ku * c - kv * sn;
+        ks[tt][i + half] = kv * c + ku * sn;
+      }
+      __syncthreads();
+    }
     if (base + LT_TT < nt) fetch(base + LT_TT);
     float* orow = out + (size_t)(t0 + base) * H * vdim + (size_t)h * vdim + j;
     int tt = 0;
@@ -359,8 +384,11 @@ selective_scan_kernel(const float* __restrict__ xz, long long ld, const float* _
 BSPEC_API int bspec_lightning_recurrence(const float* proj, long long ld, int q_off, int k_off, int v_off,
                                          const float* decay, float* state, long long state_stride,
                                          const int* qo_indptr, const int* state_slots, float* out, int n_entries, int H,
-                                         int dim, int vdim, cudaStream_t stream) {
+                                         int dim, int vdim, int act, float k_scale, const float* inv_freq, int rot,
+                                         const int* positions, cudaStream_t stream) {
   if (n_entries <= 0) return 0;
+  if (rot < 0 || rot > dim || rot % 2 || (rot > 0 && (inv_freq == nullptr || positions == nullptr)))
+    return (int)cudaErrorInvalidValue;
   if (dim <= 0 || dim > 256 || vdim <= 0 || H <= 0 || H > 65535 || n_entries > 65535)
     return (int)cudaErrorInvalidValue;
   const dim3 grid((vdim + LT_COLS - 1) / LT_COLS, H, n_entries);
@@ -369,7 +397,8 @@ BSPEC_API int bspec_lightning_recurrence(const float* proj, long long ld, int q_
   const bool few = (long long)grid.x * grid.y * grid.z < 4 * 148;
 #define LL(NR, L)                                                                                                  \
   BSPEC_LAUNCH_SERIALIZED((lightning_recurrence_kernel<NR, L>), grid, LT_COLS * L, 0, stream, proj, ld, q_off,     \
-                          k_off, v_off, decay, state, state_stride, qo_indptr, state_slots, out, H, dim, vdim)
+                          k_off, v_off, decay, state, state_stride, qo_indptr, state_slots, out, H, dim, vdim, act,   \
+                          k_scale, inv_freq, rot, positions)
   if (dim <= 32) LL(4, 8);
   else if (dim <= 64) { if (few) LL(4, 16); else LL(8, 8); }
   else if (dim <= 128) { if (few) LL(4, 32); else LL(16, 8); }

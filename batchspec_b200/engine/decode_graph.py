@@ -43,7 +43,7 @@ class DecodeGraph:
         self.max_kv_len = int(max_kv_len)
         cache = engine.cache
         B, ng = self.B, len(cache.groups)
-        self.P = [-(-self.max_kv_len // g.page_size) for g in cache.groups]      # table entries per row, per group
+        self.P = [max(1, g.pages_for(self.max_kv_len)) for g in cache.groups]      # table entries per row, per group
         off, o = {}, 0
         for name, kind in CONTEXT_FIELDS:
             off[name] = o

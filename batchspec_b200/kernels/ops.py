@@ -51,7 +51,13 @@ _SIGNATURES = {
     "bspec_scale": [c_void_p, c_longlong, c_float, c_void_p],
     "bspec_gate_mul": [c_void_p, c_void_p, c_longlong, c_void_p, c_longlong, c_int, c_int, c_int, c_float, c_void_p],
     "bspec_lightning_recurrence": [c_void_p, c_longlong, c_int, c_int, c_int, c_void_p, c_void_p, c_longlong, c_void_p,
-                                   c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
+                                   c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_int,
+                                   c_void_p, c_void_p],
+    "bspec_branch_join": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
+                          c_float, c_void_p, c_longlong, c_int, c_int, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int,
+                          c_longlong, c_int, c_void_p],
+    "bspec_pool_append": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
+                          c_int, c_int, c_int, c_int, c_int, c_int, c_longlong, c_longlong, c_void_p],
     "bspec_scan_conv": [c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_longlong, c_void_p,
                         c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
     "bspec_selective_scan": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p,
@@ -61,10 +67,12 @@ _SIGNATURES = {
     "bspec_relu_mul": [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
     "bspec_qkv_prepare": [c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_float,
                           c_float, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
-                          c_longlong, c_void_p, c_void_p, c_int, c_int, c_void_p],
+                          c_longlong, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_longlong,
+                          c_void_p],
     "bspec_attention_masked": [c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
                                c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p,
-                               c_longlong, c_float, c_int, c_void_p, c_longlong, c_longlong, c_float, c_int, c_void_p],
+                               c_longlong, c_float, c_int, c_void_p, c_longlong, c_longlong, c_float, c_int, c_void_p,
+                               c_int, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p],
     "bspec_delta_prepare": [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
                             c_longlong, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
                             c_int, c_int, c_int, c_float, c_float, c_void_p],
@@ -113,7 +121,7 @@ _SIGNATURES = {
     "bspec_moe_skinny_mma": [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_int,
                              c_int, c_int, c_void_p],
     "bspec_moe_gather": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p],
-    "bspec_moe_combine": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p],
+    "bspec_moe_combine": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p],
     "bspec_sgemm_tn_batched": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_longlong, c_longlong, c_longlong,
                                c_longlong, c_longlong, c_longlong, c_int, c_void_p],
     "bspec_attention_generic": [c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
@@ -209,13 +217,13 @@ def set_pdl(on: bool) -> None:
 _TRACE_SETTERS = ["bspec_trace_set_attention_tcgen05", "bspec_trace_set_elementwise", "bspec_trace_set_attention_generic", "bspec_trace_set_attention_bf16",
                   "bspec_trace_set_gemm_fp32", "bspec_trace_set_sampling", "bspec_trace_set_gemm_tcgen05", "bspec_trace_set_latent",
                   "bspec_trace_set_moe", "bspec_trace_set_latent_mma", "bspec_trace_set_delta",
-                  "bspec_trace_set_state_mixers", "bspec_trace_set_streams"]
+                  "bspec_trace_set_state_mixers", "bspec_trace_set_streams", "bspec_trace_set_joins"]
 TRACE_KERNEL_NAMES = {1: "embed", 2: "add_rmsnorm", 3: "gather_rows_add", 4: "silu_mul", 5: "rope_kv_append",
                       6: "rope_inplace", 7: "attn_generic", 8: "attn_decode", 9: "attn_prefill", 10: "sgemm",
                       11: "sample_threshold", 12: "sample_pick", 13: "sample_final", 14: "add_layernorm", 15: "clamped_glu",
                       16: "gelu_erf", 17: "tanh_softcap", 18: "residual_update", 19: "qkv_prepare", 60: "delta_prepare",
                       61: "delta_recurrence", 62: "gated_rmsnorm", 63: "bigram_add", 64: "scale", 65: "lightning_recurrence",
-                      66: "scan_conv", 67: "selective_scan", 70: "stream_expand", 71: "stream_norm", 72: "stream_gather", 20: "gemm_tcgen05", 30: "attn_prefill_tc", 40: "latent_prepare",
+                      66: "scan_conv", 67: "selective_scan", 70: "stream_expand", 71: "stream_norm", 72: "stream_gather", 73: "branch_join", 21: "pool_append", 20: "gemm_tcgen05", 30: "attn_prefill_tc", 40: "latent_prepare",
                       41: "latent_attn_generic", 42: "gate_heads", 43: "latent_attn_mma", 44: "latent_attn_join",
                       50: "moe_route", 51: "moe_plan", 52: "moe_grouped", 53: "moe_gather", 54: "moe_combine", 55: "moe_skinny", 56: "moe_skinny_mma", 57: "moe_rank", 58: "moe_offsets", 59: "moe_place"}
 
@@ -393,6 +401,53 @@ def relu_squared_(x: torch.Tensor) -> torch.Tensor:
     assert x.is_contiguous()
     _check(load_library().bspec_relu_squared(x.data_ptr(), _dtype_code(x.dtype), x.numel(), _stream()), "relu_squared")
     return x
+
+
+# ---------------------------------------------------------------------------- branches that are normed before they join
+
+class NormedPair:
+    """Two results of one sublayer, ``a / rms(a) * wa + b / rms(b) * wb``: a branch that ``branch_join`` forms while it
+    joins it (rms with ``eps``; the weights float32 [d])."""
+    __slots__ = ("a", "b", "wa", "wb", "eps")
+
+    def __init__(self, a, b, wa, wb, eps: float):
+        self.a, self.b, self.wa, self.wb, self.eps = a, b, wa, wb, float(eps)
+
+
+def branch_join(src: Optional[torch.Tensor], delta, dst: Optional[torch.Tensor] = None,
+                out: Optional[torch.Tensor] = None, post: Optional[torch.Tensor] = None, branch_eps: float = 0.0,
+                norm_w: Optional[torch.Tensor] = None, eps: float = 0.0, hist: Optional[torch.Tensor] = None,
+                slot: int = 0, store: bool = False, coef: Optional[torch.Tensor] = None,
+                rows: Optional[torch.Tensor] = None) -> None:
+    """One kernel for a branch's way into the float32 residual; every part is optional.  y = ``delta`` [n, d] (or a
+    ``NormedPair``); x = ``src`` + y, with ``post`` (float32 [d]) x = src + y / rms(y) * post; ``store``: hist[slot] = x;
+    ``coef`` (float32 [slot + 1]): x = sum_{j < slot} coef[j] hist[j] + coef[slot] x; ``dst`` = x; ``out`` = x / rms(x) *
+    norm_w, or the cast of x without ``norm_w``.  ``hist`` float32 [slots, n, d].  ``rows`` int32: block i works on row
+    rows[i] of src, delta and hist and writes row i of dst and out."""
+    require("joins")
+    pair = delta if isinstance(delta, NormedPair) else None
+    a, b = (pair.a, pair.b) if pair is not None else (delta, None)
+    if pair is not None:
+        assert post is None or branch_eps == pair.eps, "one eps for all norms on a branch"
+        branch_eps = pair.eps
+    _require_cuda(src, a, b, dst, out, post, norm_w, hist, coef, rows)
+    like = src if src is not None else a
+    n_src, d = like.shape
+    n = rows.numel() if rows is not None else n_src
+    f32 = lambda t, k: t is None or (t.dtype == torch.float32 and t.is_contiguous() and t.numel() == k)
+    assert f32(src, n_src * d) and f32(dst, n * d) and f32(post, d) and f32(norm_w, d) and f32(coef, slot + 1)
+    assert pair is None or (f32(pair.wa, d) and f32(pair.wb, d) and b.dtype == a.dtype and b.shape == a.shape and b.is_contiguous())
+    assert a is None or (a.shape == (n_src, d) and a.is_contiguous())
+    assert out is None or (out.shape == (n, d) and out.is_contiguous())
+    assert hist is None or (hist.dtype == torch.float32 and hist.is_contiguous() and hist.shape[1:] == (n_src, d)
+                            and slot < hist.shape[0])
+    assert rows is None or (rows.dtype == torch.int32 and not store and dst is not src)
+    code = _dtype_code(a.dtype) if a is not None else (_dtype_code(out.dtype) if out is not None else F32)
+    _check(load_library().bspec_branch_join(
+        _ptr(src), _ptr(dst), _ptr(rows), _ptr(a), _ptr(b), code, _ptr(pair.wa) if pair else None,
+        _ptr(pair.wb) if pair else None, _ptr(post), float(branch_eps), _ptr(hist),
+        hist.stride(0) if hist is not None else 0, int(slot), int(bool(store)), _ptr(coef), _ptr(norm_w), float(eps),
+        _ptr(out), _dtype_code(out.dtype) if out is not None else code, n, n_src, d, _stream()), "branch_join")
 
 
 # ---------------------------------------------------------------------------- several residual streams
@@ -728,7 +783,7 @@ def gate_mul(x: torch.Tensor, gate: Optional[torch.Tensor], out: torch.Tensor, f
 def paged_attention(qkv: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, ctx, tables, n_heads: int,
                     n_kv_heads: int, head_dim: int, scale: float, window: int = 0, chunk: int = 0,
                     sink: Optional[torch.Tensor] = None, sink_l2: Optional[torch.Tensor] = None,
-                    softcap: float = 0.0) -> None:
+                    softcap: float = 0.0, slopes: Optional[torch.Tensor] = None, pooled=None) -> None:
     """Causal attention of the step's tokens over their requests' cached keys.
     ``qkv``: [n, >= n_heads*head_dim] rows with the (already rotated) query heads
     first.  ``ctx`` gives qo_indptr / positions / n_entries / max_q_len, ``tables``
@@ -744,7 +799,8 @@ def paged_attention(qkv: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, c
                             and sink_l2.dtype == torch.float32 and sink_l2.numel() == n_heads)
     mask = int(window) if window else -int(chunk)      # the kernels take a chunk mask as a negative window
     lib = load_library()
-    if qkv.dtype == torch.bfloat16 and head_dim in (64, 128, 256) and not FORCE_GENERIC_ATTENTION:
+    if (qkv.dtype == torch.bfloat16 and head_dim in (64, 128, 256) and not FORCE_GENERIC_ATTENTION
+            and slopes is None and pooled is None):
         # Everything that depends on the step and the layer's sizes only is worked out once per step (all layers of
         # a model ask the same question), the scratch included: the layers run one after the other on one stream.
         key = ("attention", n_heads, n_kv_heads, head_dim, id(tables), BALANCED_ATTENTION, USE_TMA_ATTENTION)
@@ -779,8 +835,8 @@ def paged_attention(qkv: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, c
         qkv.data_ptr(), qkv.stride(0), out.data_ptr(), cache.data_ptr(), _dtype_code(qkv.dtype),
         ctx.qo_indptr.data_ptr(), ctx.positions.data_ptr(), tables.kv_indptr.data_ptr(), tables.kv_indices.data_ptr(),
         ctx.n_entries, ctx.max_q_len, n_heads, n_kv_heads, head_dim, head_dim, tables.page_size, float(scale),
-        int(window), int(chunk), _ptr(sink), cache.shape[0], float(softcap), 0, None, 0, out.stride(0), 1.0, 0, _stream()),
-        "attention_generic")
+        int(window), int(chunk), _ptr(sink), cache.shape[0], float(softcap), 0, None, 0, out.stride(0), 1.0, 0, _ptr(slopes),
+        *_pool_args(pooled, cache, tables.page_size), _stream()), "attention_generic")
 
 
 def qkv_prepare(qkv: torch.Tensor, n_heads: int, n_kv_heads: int, head_dim: int, v_dim: int,
@@ -788,14 +844,16 @@ def qkv_prepare(qkv: torch.Tensor, n_heads: int, n_kv_heads: int, head_dim: int,
                 magnitude: float, norm_eps: float, positions: torch.Tensor, tok_entry: torch.Tensor,
                 kv_indptr: torch.Tensor, kv_indices: torch.Tensor, cache: torch.Tensor, page_size: int,
                 write_kv: bool = True, q_norm: Optional[torch.Tensor] = None, k_norm: Optional[torch.Tensor] = None,
-                norm_first: bool = False) -> torch.Tensor:
+                norm_first: bool = False, pooled=None) -> torch.Tensor:
     """From the float32 rows [q | k | v] of the fused projection: bias, rotation of the first ``rotary_dim`` numbers
     of every q and k head (cosine and sine times ``magnitude``), division of every q and k head by its root mean
     square (``norm_eps`` > 0; times ``q_norm`` / ``k_norm``, a weight per number of a head shared by the heads, when
     given; before the rotation with ``norm_first``, else after it), in float32; returns q [n, n_heads * head_dim] in the cache's dtype and writes k and v
     into the cache page of each token's position.  Page layout: [k: kv head, row, head_dim | v: kv head, row, v_dim].
     ``qkv`` may be a view of the leading columns of wider rows.  ``v_dim`` 0: no values (the keys serve as values)
-    and a page holds keys only."""
+    and a page holds keys only.  ``pooled`` = (P, pages, tables), for steps whose entries have one token each: a token
+    that completes a block of P also writes the block's mean key and value there (``pool_append`` does it for longer
+    portions)."""
     _require_cuda(qkv, cache, positions)
     n = qkv.shape[0]
     assert qkv.dtype == torch.float32 and qkv.stride(1) == 1 and cache.is_contiguous()
@@ -815,22 +873,49 @@ def qkv_prepare(qkv: torch.Tensor, n_heads: int, n_kv_heads: int, head_dim: int,
         float(magnitude), float(norm_eps), positions.data_ptr(), tok_entry.data_ptr(), kv_indptr.data_ptr(),
         kv_indices.data_ptr(), q.data_ptr(), cache.data_ptr(), _dtype_code(cache.dtype), int(page_size),
         int(bool(write_kv)), cache.shape[0], _ptr(q_norm), _ptr(k_norm),
-        _dtype_code(q_norm.dtype) if q_norm is not None else F32, int(bool(norm_first)), _stream()), "qkv_prepare")
+        _dtype_code(q_norm.dtype) if q_norm is not None else F32, int(bool(norm_first)), *_pool_args(pooled, cache, page_size),
+        _stream()), "qkv_prepare")
     return q
+
+
+def _pool_args(pooled, cache, page_size: int):
+    """(P, pages, table starts, table, number of pages) of the kernels that read or write pooled entries; their pages
+    have the layout and the number of rows of the tokens' pages."""
+    if pooled is None:
+        return 0, None, None, None, 0
+    pool, pages, tables = pooled
+    assert pages.dtype == cache.dtype and pages.is_contiguous() and pages.shape[1:] == cache.shape[1:]
+    assert tables.page_size == page_size and pool > 0
+    return int(pool), pages.data_ptr(), tables.kv_indptr.data_ptr(), tables.kv_indices.data_ptr(), pages.shape[0]
+
+
+def pool_append(cache: torch.Tensor, ctx, tables, pooled, n_kv_heads: int, head_dim: int, v_dim: int) -> None:
+    """The mean key and value of every block of P tokens that the step's portions complete, of the rows as ``cache``
+    holds them, into the pooled pages; ``pooled`` = (P, pages, tables)."""
+    _require_cuda(cache)
+    pool, pages, indptr, indices, n_pool = _pool_args(pooled, cache, tables.page_size)
+    _check(load_library().bspec_pool_append(
+        cache.data_ptr(), _dtype_code(cache.dtype), ctx.qo_indptr.data_ptr(), ctx.positions.data_ptr(),
+        tables.kv_indptr.data_ptr(), tables.kv_indices.data_ptr(), pages, indptr, indices, ctx.n_entries, ctx.max_q_len,
+        n_kv_heads, head_dim, v_dim, tables.page_size, pool, cache.shape[0], n_pool, _stream()), "pool_append")
 
 
 def masked_attention(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, ctx, tables, n_heads: int,
                      n_kv_heads: int, head_dim: int, v_dim: int, scale: float, window: int = 0, chunk: int = 0,
                      sink: Optional[torch.Tensor] = None, softcap: float = 0.0, values_are_keys: bool = False,
-                     gate: Optional[torch.Tensor] = None, out_scale: float = 1.0, gate_per_head: bool = False) -> None:
+                     gate: Optional[torch.Tensor] = None, out_scale: float = 1.0, gate_per_head: bool = False,
+                     slopes: Optional[torch.Tensor] = None, pooled=None) -> None:
     """Causal attention with optional masks and sink over pages laid out [k | v] with values of size ``v_dim``:
     ``window`` > 0 keeps the last ``window`` keys, ``chunk`` > 0 the keys of the query's own chunk of positions;
     ``sink`` (float32 per query head) adds exp(sink) to the softmax denominator; ``softcap`` c > 0 turns a scaled
     score s into c tanh(s / c); ``values_are_keys``: pages hold keys only and a key is its own value;  ``gate``
     (a float32 view [n, n_heads * v_dim] of rows that may be wider; [n, n_heads] with ``gate_per_head``, one logit for
     all numbers of a head): the output is multiplied by sigmoid(gate);
-    ``out_scale`` multiplies it.  ``out`` may be a view of the leading columns of wider rows.  float32 arithmetic."""
-    _require_cuda(q, out, cache, sink, gate)
+    ``out_scale`` multiplies it.  ``slopes`` (float32 per query head): slope * (query - key) is taken off a score.
+    ``pooled`` = (P, pages, tables), with a window: before the window the mean key and value of every block of P tokens
+    is seen too.  ``out`` may be a view of the leading columns of wider rows.  float32 arithmetic."""
+    _require_cuda(q, out, cache, sink, gate, slopes)
+    assert slopes is None or (slopes.dtype == torch.float32 and slopes.numel() == n_heads and slopes.is_contiguous())
     assert q.stride(1) == 1 and out.stride(1) == 1 and out.dtype == q.dtype == cache.dtype
     assert out.shape == (q.shape[0], n_heads * v_dim) and (not values_are_keys or v_dim == head_dim)
     assert sink is None or (sink.dtype == torch.float32 and sink.numel() == n_heads and sink.is_contiguous())
@@ -841,8 +926,8 @@ def masked_attention(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, ct
         ctx.positions.data_ptr(), tables.kv_indptr.data_ptr(), tables.kv_indices.data_ptr(), ctx.n_entries,
         ctx.max_q_len, n_heads, n_kv_heads, head_dim, v_dim, tables.page_size, float(scale), int(window), int(chunk),
         _ptr(sink), cache.shape[0], float(softcap), int(bool(values_are_keys)), _ptr(gate),
-        gate.stride(0) if gate is not None else 0, out.stride(0), float(out_scale), int(bool(gate_per_head)), _stream()),
-        "attention_masked")
+        gate.stride(0) if gate is not None else 0, out.stride(0), float(out_scale), int(bool(gate_per_head)), _ptr(slopes),
+        *_pool_args(pooled, cache, tables.page_size), _stream()), "attention_masked")
 
 
 # ---------------------------------------------------------------------------- gated delta rule
@@ -888,19 +973,19 @@ def delta_recurrence(mix: torch.Tensor, gates: torch.Tensor, proj: torch.Tensor,
     return out
 
 
-def gated_rmsnorm(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: float, n_heads: int, v_dim: int,
+def gated_rmsnorm(o: torch.Tensor, gate: torch.Tensor, weight: Optional[torch.Tensor], eps: float, n_heads: int, v_dim: int,
                   out_dtype: torch.dtype, gate_act: str = "silu") -> torch.Tensor:
     """o float32 [n, H * V]; gate a float32 view [n, H * V] of rows that may be wider.  Returns
-    o / rms_V(o) * weight * act(gate) in ``out_dtype``, act = "silu" or "sigmoid".  With H = 1 the norm runs over the
+    o / rms_V(o) * weight * act(gate) in ``out_dtype``, act = "silu" or "sigmoid"; ``weight`` None: no weight.  With H = 1 the norm runs over the
     whole row."""
     assert gate_act in ("silu", "sigmoid")
     _require_cuda(o, gate, weight)
     n = o.shape[0]
     assert o.dtype == torch.float32 and o.is_contiguous() and gate.dtype == torch.float32 and gate.stride(1) == 1
-    assert gate.shape == o.shape == (n, n_heads * v_dim) and weight.numel() == v_dim
+    assert gate.shape == o.shape == (n, n_heads * v_dim) and (weight is None or weight.numel() == v_dim)
     out = torch.empty((n, n_heads * v_dim), dtype=out_dtype, device=o.device)
-    _check(load_library().bspec_gated_rmsnorm(o.data_ptr(), gate.data_ptr(), gate.stride(0), weight.data_ptr(),
-                                              _dtype_code(weight.dtype), out.data_ptr(), _dtype_code(out_dtype), n,
+    _check(load_library().bspec_gated_rmsnorm(o.data_ptr(), gate.data_ptr(), gate.stride(0), _ptr(weight),
+                                              _dtype_code(weight.dtype) if weight is not None else F32, out.data_ptr(), _dtype_code(out_dtype), n,
                                               n_heads, v_dim, float(eps), int(gate_act == "sigmoid"), _stream()),
            "gated_rmsnorm")
     return out
@@ -909,9 +994,12 @@ def gated_rmsnorm(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps
 # ---------------------------------------------------------------------------- lightning attention, selective scan
 
 def lightning_recurrence(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, decay: torch.Tensor,
-                         state: torch.Tensor, ctx, n_heads: int, dim: int, v_dim: int) -> torch.Tensor:
+                         state: torch.Tensor, ctx, n_heads: int, dim: int, v_dim: int, activation: Optional[str] = "silu",
+                         k_scale: float = 1.0, inv_freq: Optional[torch.Tensor] = None, rotary_dim: int = 0) -> torch.Tensor:
     """Linear attention with a fixed decay per head over every entry's portion: S <- decay_h S + k v^T, o = S^T q, with
-    q, k, v = silu of the float32 columns of ``proj`` at ``q_off`` / ``k_off`` (H * dim each) and ``v_off`` (H * v_dim).
+    q, k, v = the float32 columns of ``proj`` at ``q_off`` / ``k_off`` (H * dim each) and ``v_off`` (H * v_dim), through
+    silu or, with ``activation`` None, as they are; k times ``k_scale``.  ``rotary_dim`` > 0: q and k are rotated here
+    (numbers i and i + rotary_dim / 2; every block of a head forms the angles, so this is for steps of few tokens).
     ``state[slot]`` holds S as [head, value column, key row] float32 and is read and written.  Returns o float32
     [n, H * v_dim]."""
     _require_cuda(proj, decay, state)
@@ -919,12 +1007,14 @@ def lightning_recurrence(proj: torch.Tensor, q_off: int, k_off: int, v_off: int,
     assert proj.dtype == torch.float32 and proj.stride(1) == 1 and state.dtype == torch.float32 and state.stride(1) == 1
     assert decay.dtype == torch.float32 and decay.numel() == n_heads and decay.is_contiguous()
     assert state.shape[1] >= n_heads * v_dim * dim and dim <= 256
-    assert max(q_off, k_off) + n_heads * dim <= ld and v_off + n_heads * v_dim <= ld
+    assert max(q_off, k_off) + n_heads * dim <= ld and v_off + n_heads * v_dim <= ld and activation in ("silu", None)
+    assert not rotary_dim or (inv_freq.dtype == torch.float32 and inv_freq.shape == (2, rotary_dim // 2) and rotary_dim <= dim)
     out = torch.empty((n, n_heads * v_dim), dtype=torch.float32, device=proj.device)
     _check(load_library().bspec_lightning_recurrence(
         proj.data_ptr(), proj.stride(0), int(q_off), int(k_off), int(v_off), decay.data_ptr(), state.data_ptr(),
         state.stride(0), ctx.qo_indptr.data_ptr(), ctx.state_slots.data_ptr(), out.data_ptr(), ctx.n_entries, n_heads,
-        dim, v_dim, _stream()), "lightning_recurrence")
+        dim, v_dim, int(activation == "silu"), float(k_scale), _ptr(inv_freq) if rotary_dim else None, int(rotary_dim),
+        ctx.positions.data_ptr() if rotary_dim else None, _stream()), "lightning_recurrence")
     return out
 
 
@@ -1032,14 +1122,15 @@ def check_status() -> None:
 _BOUNDS_REPORTS = ["bspec_bounds_report_state_mixers", "bspec_bounds_report_elementwise", "bspec_bounds_report_gemm_tcgen05",
                    "bspec_bounds_report_attention_generic", "bspec_bounds_report_attention_bf16",
                    "bspec_bounds_report_latent", "bspec_bounds_report_latent_mma", "bspec_bounds_report_delta",
-                   "bspec_bounds_report_streams"]
+                   "bspec_bounds_report_streams", "bspec_bounds_report_joins"]
 BOUNDS_CODES = {101: "token id (embedding)", 102: "row (gather)", 103: "block-table slot (rotary + cache append)",
                 104: "page id (rotary + cache append)", 105: "block-table slot (q/k/v product's epilogue)",
                 106: "page id (q/k/v product's epilogue)", 107: "page id (attention over plain loads)",
                 108: "page id (bfloat16 attention over plain loads)", 109: "block-table slot (latent entry append)",
                 110: "page id (latent entry append)", 111: "page id (latent attention over plain loads)",
                 112: "page id (latent attention on the tensor cores)", 113: "block-table slot (q/k/v preparation)",
-                114: "page id (q/k/v preparation)"}
+                114: "page id (q/k/v preparation)", 115: "row (branch join)", 116: "page id (a block's rows)",
+                117: "block-table slot (pooled entry)", 118: "page id (pooled entry)"}
 
 
 def bounds_reports() -> list:
@@ -1312,10 +1403,15 @@ MOE_SKINNY = True                # bfloat16 steps with fewer rows per expert: th
 
 
 def moe_route(h: torch.Tensor, router: torch.Tensor, correction: Optional[torch.Tensor], n_groups: int, keep: int,
-              top: int, scale: float, softmax_top: bool = False):
+              top: int, scale: float, softmax_top: bool = False, softmax: bool = False, group_max: bool = False,
+              renormalise: bool = False):
     """(expert ids int32 [n, top], weights float32 [n, top]) of every token; the rule is in ``csrc/moe.cu``.
     ``softmax_top``: the logits plus ``correction`` (a bias) choose, and the weights are the softmax over the chosen
-    logits alone; otherwise sigmoid scores."""
+    logits alone; ``softmax``: the scores are the softmax over all experts; otherwise sigmoid scores.  ``group_max``: a
+    group's score is its largest choice instead of the sum of its two largest.  ``renormalise``: the weights are the
+    chosen scores divided by their sum."""
+    assert not (softmax and softmax_top)
+    rule = (1 if softmax_top else 2 if softmax else 0) + (4 if group_max else 0) + (8 if renormalise else 0)
     _require_cuda(h, router)
     n, d = h.shape
     E = router.shape[0]
@@ -1327,18 +1423,20 @@ def moe_route(h: torch.Tensor, router: torch.Tensor, correction: Optional[torch.
     _check(load_library().bspec_moe_route(h.data_ptr(), _dtype_code(h.dtype), n, d, router.data_ptr(), _ptr(correction),
                                           _dtype_code(correction.dtype) if correction is not None else F32, E,
                                           int(n_groups), int(keep), int(top), float(scale), ids.data_ptr(),
-                                          wts.data_ptr(), _ptr(logits), int(bool(softmax_top)), _stream()), "moe_route")
+                                          wts.data_ptr(), _ptr(logits), rule, _stream()), "moe_route")
     return ids, wts
 
 
 def moe_experts(h: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor,
-                out_dtype: torch.dtype, glu: bool = False) -> torch.Tensor:
+                out_dtype: torch.dtype, glu: bool = False, add: Optional[torch.Tensor] = None) -> torch.Tensor:
     """sum_k wts[t, k] * Wdown[e] gelu(Wup[e] h[t]) with e = ids[t, k].  ``w_up`` [E, ff, d], ``w_down`` [E, d, ff].
     ``glu``: the experts are gated, Wdown[e] (silu(Wgate[e] h) * (Wup[e] h)), and ``w_up`` holds [gate; up] as
     [E, 2 ff, d]; the first product then leaves its result as it is, and this package's grouped kernels form
     silu(gate) * up while they stage the rows of the second product (the vendor's grouped product is followed by
     ``silu_mul`` instead).
+    ``add`` [n, d] in ``out_dtype`` (a shared expert's result) is added to the sum.
     The (token, choice) rows are sorted by expert on the device; no count is read on the host."""
+    assert add is None or (add.shape == h.shape and add.dtype == out_dtype and add.is_contiguous())
     _require_cuda(h, ids, wts, w_up, w_down)
     lib = load_library()
     n, d = h.shape
@@ -1416,7 +1514,7 @@ def moe_experts(h: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, w_up: tor
                "moe_grouped_down")
     out = torch.empty((n, d), dtype=out_dtype, device=dev)
     _check(lib.bspec_moe_combine(y.data_ptr(), _dtype_code(y.dtype), inv.data_ptr(), wts.data_ptr(), top,
-                                 out.data_ptr(), _dtype_code(out_dtype), n, d, _stream()), "moe_combine")
+                                 out.data_ptr(), _dtype_code(out_dtype), n, d, _ptr(add), _stream()), "moe_combine")
     return out
 
 

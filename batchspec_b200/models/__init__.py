@@ -13,6 +13,7 @@ from .decoder import CacheNeed, DecoderModel, LayerCache
 from .finolix import build_finolix
 from .llama import build_llama
 from .lupusun import build_lupusun
+from .podizen import build_podizen
 from .tokolorn import build_tokolorn
 from .spec import LayerSpec, ModelSpec, RunEntry, prenorm_layer
 from .vabanex import build_vabanex
@@ -36,6 +37,7 @@ register_model("Vabanex", build_vabanex)
 register_model("Lupusun", build_lupusun)
 register_model("Tokolorn", build_tokolorn)
 register_model("Finolix", build_finolix)
+register_model("Podizen", build_podizen)
 
 __all__ = ["MODEL_REGISTRY", "register_model", "get_model", "DecoderModel", "LayerCache", "CacheNeed",
-           "ModelSpec", "LayerSpec", "RunEntry", "prenorm_layer", "build_finolix", "build_llama", "build_lupusun", "build_tokolorn", "build_vabanex"]
+           "ModelSpec", "LayerSpec", "RunEntry", "prenorm_layer", "build_finolix", "build_llama", "build_lupusun", "build_podizen", "build_tokolorn", "build_vabanex"]

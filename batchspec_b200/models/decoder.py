@@ -25,11 +25,14 @@ class LayerCache:
     page_size * entry elements] of its group's pool (None if the mixer asked for no pages);
     ``group``: index of the block tables in the step context; ``state``:
     [max_requests, *state_shape] or None; ``owner``: False for a run that reads
-    another run's cache."""
+    another run's cache.  ``pooled`` / ``pooled_group``: the same two for the entries of
+    pooled blocks, if the mixer asked for them."""
     kv: Optional[torch.Tensor]
     group: int
     state: Optional[torch.Tensor]
     owner: bool
+    pooled: Optional[torch.Tensor] = None
+    pooled_group: int = -1
 
 
 @dataclass
@@ -152,9 +155,16 @@ class DecoderModel:
             # [n, S, d]; the first run's norm fills it from the embedding rows (``expand_from``)
             expand = resid
             resid = torch.empty((n, s.streams, s.hidden_size), dtype=torch.float32, device=self.runtime.device)
-        pending, scale, vec, mix = None, 1.0, None, None
+        pending, scale, vec, mix, join = None, 1.0, None, None, None
+        history = None
+        if s.depth_average:
+            if first is not None or s.streams:
+                raise ValueError("a model that averages over depth has one residual stream and adds no input again")
+            history = torch.empty((len(s.order) + 1, n, s.hidden_size), dtype=torch.float32, device=self.runtime.device)
         for e, run in enumerate(s.order):
             if run.add_input:
+                if join is not None:
+                    raise ValueError("a branch that is normed before it joins cannot be followed by the input again")
                 ops.residual_update(resid, pending, scale, first, vec)
                 pending, scale, vec = None, 1.0, None
             block = self.blocks[run.layer]
@@ -167,9 +177,13 @@ class DecoderModel:
                 extra["pending_mix"] = mix
             if s.streams and e == 0:
                 extra["expand_from"] = expand
+            if join is not None:
+                extra["pending_join"] = join
+            if history is not None:
+                extra["history"], extra["slot"] = history, e
             resid, pending = block.forward(resid, pending, ctx, self.caches[e], **extra)
             scale, vec = getattr(block, "residual_mult", 1.0), getattr(block, "residual_vec", None)
-            mix = getattr(block, "residual_mix", None)
+            mix, join = getattr(block, "residual_mix", None), getattr(block, "residual_join", None)
             if s.streams and (mix is None or scale != 1.0):
                 raise ValueError(f"block kind {block.kind!r} does not keep several residual streams")
             if self.layer_probe is not None:
@@ -177,6 +191,10 @@ class DecoderModel:
                     after = torch.empty((n, s.hidden_size), dtype=torch.float32, device=self.runtime.device)
                     every = torch.arange(n, dtype=torch.int32, device=self.runtime.device)
                     ops.stream_gather(resid, pending, vec, mix, every, after)
+                elif join is not None:
+                    after = torch.empty_like(resid)
+                    ops.branch_join(resid, pending, dst=after, post=join.post, branch_eps=join.eps, hist=history,
+                                    slot=e + 1 if history is not None else 0, coef=join.coef)
                 else:
                     after = resid.clone()
                     ops.residual_update(after, pending, scale, vec=vec)
@@ -184,12 +202,16 @@ class DecoderModel:
         n_out = ctx.n_logit_rows
         if n_out == 0:
             return torch.empty((0, s.vocab_size), dtype=torch.float32, device=self.runtime.device)
-        picked = torch.empty((n_out, s.hidden_size), dtype=torch.float32, device=self.runtime.device)
-        if s.streams:
-            ops.stream_gather(resid, pending, vec, mix, ctx.logit_rows, picked)
+        if join is not None:          # the last branch's join, on the wanted rows only, and the final norm in one kernel
+            z = self.final_norm.forward_join(resid, pending, join, history, len(s.order) if history is not None else 0,
+                                             rows=ctx.logit_rows)
         else:
-            ops.gather_rows_add(resid, pending, ctx.logit_rows, picked, scale, vec)
-        z = self.final_norm.forward(picked, None)
+            picked = torch.empty((n_out, s.hidden_size), dtype=torch.float32, device=self.runtime.device)
+            if s.streams:
+                ops.stream_gather(resid, pending, vec, mix, ctx.logit_rows, picked)
+            else:
+                ops.gather_rows_add(resid, pending, ctx.logit_rows, picked, scale, vec)
+            z = self.final_norm.forward(picked, None)
         with bucket("lm_head"):
             logits = ops.linear(z, self.head, out_dtype=torch.float32)
         if self.logits_part is not None:

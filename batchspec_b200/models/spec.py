@@ -63,3 +63,6 @@ class ModelSpec:
     # the embedding (after the input part); the blocks' kinds must be ones that take such a residual, and the sum
     # of the streams goes to the final norm
     streams: int = 0
+    # the blocks average over depth: the executor keeps the residual that entered every run and hands it to them
+    # (``history``); the blocks' kinds must be ones that take it
+    depth_average: bool = False

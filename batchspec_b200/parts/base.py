@@ -9,7 +9,7 @@ checkpoint names.  The reference fixes the parts by subclass hooks
 one model may mix different mixers and feed-forwards.
 
 Registries: ``MIXERS``, ``FEED_FORWARDS``, ``NORMS``, ``POSITION_ENCODINGS``,
-``BLOCKS``, ``BRANCH_SCALES``, ``STREAM_MIXES``, ``INPUT_PARTS``, ``LOGITS_PARTS``.  ``register_part(registry, kind)``
+``BLOCKS``, ``BRANCH_SCALES``, ``STREAM_MIXES``, ``DEPTH_AVERAGES``, ``INPUT_PARTS``, ``LOGITS_PARTS``.  ``register_part(registry, kind)``
 is a class decorator; ``build_part(registry, spec, runtime)`` instantiates
 ``spec.kind`` with ``spec.params``.
 """
@@ -57,12 +57,17 @@ class CacheSpec:
     keys and values, 1 for a mixer that stores a single (compressed) entry.
     ``page_size``: tokens per page of this mixer's group, or None for the
     engine's default; groups with different page sizes have block tables of
-    different lengths for the same request."""
+    different lengths for the same request.
+    ``pool`` P > 0: besides, every whole block of P tokens has one more entry of the
+    same shape, which is kept while the request lives.  These entries have a group of
+    their own (pages of as many entries, a block table: entry b is block b), and a
+    windowed group keeps the tokens of the block that is not yet whole."""
     policy: str
     entry_shape: Tuple[int, ...]
     window: Optional[int] = None
     tensors: int = 2
     page_size: Optional[int] = None
+    pool: int = 0
 
 
 @dataclass(frozen=True)
@@ -129,7 +134,9 @@ class Mixer(Part):
     layer (None if the mixer declared no needs): ``cache.kv`` the layer's page
     tensor and ``cache.group`` the index of its block tables in ``ctx``,
     ``cache.state`` its per-request state tensor [max_requests, *shape],
-    ``cache.owner`` False when the layer only reads another layer's cache."""
+    ``cache.owner`` False when the layer only reads another layer's cache;
+    ``cache.pooled`` and ``cache.pooled_group`` the pages and the group of the blocks'
+    entries (a spec with ``pool``)."""
 
     def cache_spec(self) -> Optional[CacheSpec]:
         return None
@@ -177,8 +184,19 @@ POSITION_ENCODINGS: Dict[str, type] = {}
 BLOCKS: Dict[str, type] = {}
 BRANCH_SCALES: Dict[str, type] = {}
 STREAM_MIXES: Dict[str, type] = {}
+DEPTH_AVERAGES: Dict[str, type] = {}
 INPUT_PARTS: Dict[str, type] = {}
 LOGITS_PARTS: Dict[str, type] = {}
+
+
+@dataclass
+class BranchJoin:
+    """How a branch y joins the residual x when it is normed on its way: x + y / rms(y) * ``post`` (float32 [d]; rms
+    with ``eps``), and then, with ``coef`` (float32 [j + 1]), the average sum_{i < j} coef[i] X_i + coef[j] x over the
+    residuals X_i that went into the layers so far, which the executor keeps (``ModelSpec.depth_average``)."""
+    post: Optional[torch.Tensor] = None
+    eps: float = 0.0
+    coef: Optional[torch.Tensor] = None
 
 
 class Block:
@@ -198,12 +216,15 @@ class Block:
     the vector as ``pending_vec``).  A block of a model that keeps several residual streams per token gets them as
     ``resid`` [n, S, d]; the coefficients with which its last branch joins the streams are its ``residual_mix``
     (float32 [S * S + S]: the mix matrix indexed (from, to), then the factor of the branch per stream), handed on as
-    ``pending_mix``."""
+    ``pending_mix``.  A block whose branches are normed before they join says so in ``residual_join`` (a ``BranchJoin``),
+    handed on as ``pending_join``; in a model that averages over depth its forward also takes ``history`` (float32
+    [layer runs + 1, n, d]) and ``slot``: the residual that enters the run is stored as history[slot]."""
     SLOTS: Dict[str, Dict[str, type]] = {}
     MIXER_SLOT = "mixer"
     residual_mult = 1.0
     residual_vec = None
     residual_mix = None
+    residual_join = None
 
     def __init__(self, **parts):
         missing, extra = set(self.SLOTS) - set(parts), set(parts) - set(self.SLOTS)

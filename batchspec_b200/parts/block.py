@@ -10,8 +10,8 @@ from typing import Dict
 import torch
 
 from ..kernels import ops
-from .base import (BLOCKS, BRANCH_SCALES, FEED_FORWARDS, MIXERS, NORMS, STREAM_MIXES, Block, ParamSpec, Part, Runtime,
-                   register_part)
+from .base import (BLOCKS, BRANCH_SCALES, DEPTH_AVERAGES, FEED_FORWARDS, MIXERS, NORMS, STREAM_MIXES, Block, BranchJoin,
+                   ParamSpec, Part, Runtime, register_part)
 
 
 @register_part(BLOCKS, "prenorm")
@@ -164,3 +164,64 @@ class HyperPreNormMixerBlock(Block):
         assert pending_scale == 1.0 and (pending is None or pending_mix is not None)
         a = self.norm1.forward_streams(resid, pending, pending_vec, pending_mix, self.hc1.read, expand_from)
         return resid, self.mixer.forward(a, ctx, cache)
+
+
+@register_part(DEPTH_AVERAGES, "learned")
+class LearnedDepthAverage(Part):
+    """The average over depth after a layer: sum over i < ``count`` of w[i] X_i, X_0 the input of the first layer and the
+    last X the layer's own result.  Held in float32."""
+    graph_safe = True
+
+    def __init__(self, runtime: Runtime, count: int):
+        self.runtime, self.count = runtime, int(count)
+        self.weight = None
+
+    def param_specs(self) -> Dict[str, ParamSpec]:
+        return {"weight": ParamSpec((self.count,), role="vector", init="ones_normal")}
+
+    def bind(self, params):
+        self.weight = params["weight"].to(torch.float32).contiguous()
+
+
+class _Sandwich(Block):
+    """Blocks whose branches are normed before they join: h = x + norm1b(mixer(norm1(x))), x' = h + norm2b(ffn(norm2(h))).
+    The norm of a branch, its sum, the average over depth and the next norm are one kernel (``RMSNorm.forward_join``);
+    the last branch is returned as it is, with its ``residual_join``.  A mixer that offers ``forward_branches`` (its
+    result as a pair that the join forms) is asked for that."""
+
+    @property
+    def residual_join(self):
+        post = self.norm2b if "norm2b" in self.parts else self.norm1b
+        return BranchJoin(post.weight_f32, post.eps, self.average.weight if "average" in self.parts else None)
+
+    def forward(self, resid, pending, ctx, cache, pending_scale: float = 1.0, pending_join=None, history=None,
+                slot: int = 0):
+        assert pending_scale == 1.0
+        a = self.norm1.forward_join(resid, pending, pending_join, history, slot)
+        y = (getattr(self.mixer, "forward_branches", None) or self.mixer.forward)(a, ctx, cache)
+        if "ffn" not in self.parts:
+            return resid, y
+        f = self.norm2.forward_join(resid, y, BranchJoin(self.norm1b.weight_f32, self.norm1b.eps))
+        return resid, self.ffn.forward(f, ctx)
+
+
+@register_part(BLOCKS, "sandwich")
+class SandwichBlock(_Sandwich):
+    SLOTS = {"norm1": NORMS, "mixer": MIXERS, "norm1b": NORMS, "norm2": NORMS, "ffn": FEED_FORWARDS, "norm2b": NORMS}
+
+
+@register_part(BLOCKS, "sandwich_mixer")
+class SandwichMixerBlock(_Sandwich):
+    """The same without a feed-forward."""
+    SLOTS = {"norm1": NORMS, "mixer": MIXERS, "norm1b": NORMS}
+
+
+@register_part(BLOCKS, "sandwich_averaged")
+class AveragedSandwichBlock(_Sandwich):
+    """The same, and what goes on is a learned average of the layer's result, all earlier ones and the first input."""
+    SLOTS = {**SandwichBlock.SLOTS, "average": DEPTH_AVERAGES}
+
+
+@register_part(BLOCKS, "sandwich_mixer_averaged")
+class AveragedSandwichMixerBlock(_Sandwich):
+    SLOTS = {**SandwichMixerBlock.SLOTS, "average": DEPTH_AVERAGES}

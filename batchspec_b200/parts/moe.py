@@ -17,6 +17,7 @@ import torch
 from ..kernels import ops
 from ..profiler import bucket
 from .base import FEED_FORWARDS, FeedForward, ParamSpec, Runtime, register_part
+from .mlp import SwiGLU
 
 
 @register_part(FEED_FORWARDS, "routed_gelu")
@@ -60,17 +61,34 @@ class RoutedGelu(FeedForward):
 
 @register_part(FEED_FORWARDS, "routed_glu")
 class RoutedGLU(FeedForward):
-    """Routed gated experts with a softmax over the chosen logits: z = Wr h + b in float32; the ``top`` experts of
-    largest z are taken and weighted by the softmax over those ``top`` logits alone; expert e is
-    Wdown_e (silu(Wgate_e h) * (Wup_e h)), no biases; the output is the weighted sum.  [gate; up] of every expert is
-    one stacked matrix, so the first grouped product gives both halves."""
+    """Routed gated experts.  z = Wr h + b in float32, and by ``scores``
+
+    * "softmax_top": the ``top`` experts of largest z are taken and weighted by the softmax over those logits alone;
+    * "softmax": s = softmax(z) over all experts; the experts come in ``n_groups`` equal groups of neighbours whose score
+      is their largest s, only experts of the best ``keep_groups`` groups can be chosen, the ``top`` largest s are taken
+      and weighted by s divided by the sum over the chosen.
+
+    Expert e is Wdown_e (silu(Wgate_e h) * (Wup_e h)), no biases; the output is the weighted sum.  ``shared`` > 0: one
+    more expert of that inner size runs for every token and is added.  [gate; up] of every expert is one stacked matrix,
+    so the first grouped product gives both halves."""
     graph_safe = True
 
-    def __init__(self, runtime: Runtime, dim: int, intermediate: int, n_experts: int, top: int, bias: bool = True):
+    def __init__(self, runtime: Runtime, dim: int, intermediate: int, n_experts: int, top: int, bias: bool = True,
+                 scores: str = "softmax_top", n_groups: int = 1, keep_groups: int = 1, shared: int = 0):
         self.runtime, self.dim, self.intermediate = runtime, int(dim), int(intermediate)
         self.n_experts, self.top, self.bias = int(n_experts), int(top), bool(bias)
+        self.scores, self.n_groups, self.keep_groups = scores, int(n_groups), int(keep_groups)
+        if scores not in ("softmax_top", "softmax"):
+            raise ValueError(f"router scores {scores!r} are not known ('softmax_top', 'softmax')")
         if not 0 < self.top <= self.n_experts:
             raise ValueError(f"cannot choose {top} of {n_experts} experts")
+        G = self.n_groups
+        if not (G > 0 and self.n_experts % G == 0 and 0 < self.keep_groups <= G
+                and self.keep_groups * (self.n_experts // G) >= self.top) or (G > 1 and scores != "softmax"):
+            raise ValueError(f"routing of {top} of {n_experts} experts in {G} groups keeping {keep_groups} is not possible")
+        if scores == "softmax" and self.bias:
+            raise ValueError("softmax scores take no bias")
+        self.shared = SwiGLU(runtime, dim, shared) if shared else None
 
     def param_specs(self) -> Dict[str, ParamSpec]:
         specs = {"router": ParamSpec((self.n_experts, self.dim))}
@@ -80,6 +98,8 @@ class RoutedGLU(FeedForward):
             specs[f"gate{e}"] = ParamSpec((self.intermediate, self.dim))
             specs[f"up{e}"] = ParamSpec((self.intermediate, self.dim))
             specs[f"down{e}"] = ParamSpec((self.dim, self.intermediate))
+        if self.shared is not None:
+            specs.update({"shared." + k: v for k, v in self.shared.param_specs().items()})
         return specs
 
     def bind(self, params):
@@ -90,9 +110,16 @@ class RoutedGLU(FeedForward):
         self.w_up = torch.stack([torch.cat([params[f"gate{e}"], params[f"up{e}"]], dim=0)
                                  for e in range(self.n_experts)]).contiguous()               # [E, 2 ff, d]
         self.w_down = torch.stack([params[f"down{e}"] for e in range(self.n_experts)]).contiguous()
+        if self.shared is not None:
+            self.shared.bind({k[7:]: v for k, v in params.items() if k.startswith("shared.")})
 
     def forward(self, x, ctx):
         with bucket("mlp.router"):
-            ids, wts = ops.moe_route(x, self.w_router, self.b_router, 1, 1, self.top, 1.0, softmax_top=True)
+            if self.scores == "softmax":
+                ids, wts = ops.moe_route(x, self.w_router, None, self.n_groups, self.keep_groups, self.top, 1.0,
+                                         softmax=True, group_max=True, renormalise=True)
+            else:
+                ids, wts = ops.moe_route(x, self.w_router, self.b_router, 1, 1, self.top, 1.0, softmax_top=True)
+        shared = self.shared.forward(x, ctx) if self.shared is not None else None
         with bucket("mlp.experts"):
-            return ops.moe_experts(x, ids, wts, self.w_up, self.w_down, x.dtype, glu=True)
+            return ops.moe_experts(x, ids, wts, self.w_up, self.w_down, x.dtype, glu=True, add=shared)

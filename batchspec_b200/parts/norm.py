@@ -26,6 +26,7 @@ class RMSNorm(Norm):
         self.single_rounding = bool(single_rounding) or self.one_plus
         self.scalar_weight = bool(scalar_weight)
         self.weight: Optional[torch.Tensor] = None
+        self._weight_f32: Optional[torch.Tensor] = None
 
     def param_specs(self) -> Dict[str, ParamSpec]:
         return {"weight": ParamSpec(() if self.scalar_weight else (self.dim,), role="vector",
@@ -35,6 +36,7 @@ class RMSNorm(Norm):
         self.weight = params["weight"].reshape(1).contiguous() if self.scalar_weight else params["weight"]
         if self.one_plus:
             self.weight = (1.0 + self.weight.to(torch.float32)).contiguous()
+        self._weight_f32 = None
 
     def forward(self, resid, delta=None, delta_scale: float = 1.0, delta_vec=None):
         out = torch.empty(resid.shape, dtype=self.runtime.dtype, device=resid.device)
@@ -42,6 +44,28 @@ class RMSNorm(Norm):
             ops.add_rmsnorm(resid, delta, self.weight, self.eps, out, delta_scale, self.single_rounding, delta_vec)
         return out
 
+
+    @property
+    def weight_f32(self) -> torch.Tensor:
+        """The factor per column in float32, for kernels that norm a branch on its way into the residual."""
+        if self._weight_f32 is None:
+            w = self.weight.to(torch.float32).reshape(-1)
+            self._weight_f32 = (w.expand(self.dim) if self.scalar_weight else w).contiguous()
+        return self._weight_f32
+
+    def forward_join(self, resid, delta=None, join=None, history=None, slot: int = 0, rows=None):
+        """The counterpart of ``forward`` for branches that are normed before they join (``join``, a ``BranchJoin``; None
+        adds ``delta`` as it is): one kernel norms the branch, adds it, averages over depth, updates ``resid`` and norms
+        the result.  ``history``: the residual before the average is kept as history[slot].  ``rows`` (the rows that go
+        to the head): only these are formed, and nothing is written back."""
+        n = rows.numel() if rows is not None else resid.shape[0]
+        out = torch.empty((n, self.dim), dtype=self.runtime.dtype, device=resid.device)
+        post, eps, coef = (join.post, join.eps, join.coef) if join is not None else (None, 0.0, None)
+        with bucket("norm"):
+            ops.branch_join(resid, delta, dst=resid if rows is None and delta is not None else None, out=out, post=post,
+                            branch_eps=eps, norm_w=self.weight_f32, eps=self.eps, hist=history, slot=slot,
+                            store=history is not None and rows is None, coef=coef, rows=rows)
+        return out
 
     def forward_streams(self, streams, delta=None, delta_vec=None, delta_mix=None, read=None, expand=None):
         """For a residual kept as several streams [n, S, d]: ``delta`` (times ``delta_vec`` per column) first joins

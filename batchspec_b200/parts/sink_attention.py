@@ -12,6 +12,10 @@
   out_h(i) = sum_j exp(s_ij) v_j / (exp(sink_h) + sum_j exp(s_ij));  ``fixed_sink``: the same with one given logit for
   all heads and no tensor (0.0 adds one to the denominator);
 * ``softcap`` c: a scaled score s becomes c tanh(s / c);
+* ``bias_slopes``: a distance bias, slope_h * (i - j) taken off the scaled score of query i and key j;
+* ``pool`` P, with a window W: beside the W tokens a query sees one entry for each block of P tokens that lies wholly
+  before its window (last position at most i - W): the mean of the block's keys and of its values, as the cache holds
+  them; tokens that have left the window and whose block is not yet seen are not seen at all;
 * ``values_are_keys``: there is no value projection, a key as projected is its own value, and only keys are cached;
 * ``gate``: the concatenated heads are multiplied element by element by sigmoid(Wg h) before the output projection;
   ``gate="head"``: Wg has one row per head and the head's whole output is multiplied by one number.
@@ -20,11 +24,13 @@ Launch sequence: one product for [Wq; Wk; Wv] with float32 output -> q/k/v prepa
 float32; q in the run dtype, k and v into their cache pages) -> attention over the pages -> output projection.
 ``pre_projection`` is everything before the output projection; a mixer that runs this one beside another writes both
 results into one buffer and projects them together.
+The entries of pooled blocks are written once, when a block's last token is (steps whose entries have one token each:
+by the q/k/v preparation; else by ``pool_append`` after it), into pages of a group of their own.
 A page holds its keys [kv head, row, head_dim] and then its values [kv head, row, v_dim].  With a chunk mask the
 pages that lie wholly before the chunk of the next position are given back."""
 from __future__ import annotations
 
-from typing import Dict, Optional
+from typing import Dict, List, Optional, Sequence
 
 import torch
 
@@ -32,6 +38,11 @@ from ..kernels import ops
 from ..profiler import bucket
 from .base import (MIXERS, POSITION_ENCODINGS, CacheSpec, Mixer, ParamSpec, PartSpec, Runtime, build_part,
                    register_part)
+
+
+def geometric_slopes(n_heads: int) -> List[float]:
+    """Distance-bias slopes 2^(-8 (h + 1) / n_heads) of the heads h = 0 .. n_heads - 1."""
+    return [2.0 ** (-8.0 * (h + 1) / n_heads) for h in range(n_heads)]
 
 
 @register_part(MIXERS, "sink_attention")
@@ -43,7 +54,8 @@ class SinkAttention(Mixer):
                  qk_norm_eps: Optional[float] = None, chunk: Optional[int] = None, window: Optional[int] = None,
                  sink: bool = False, fixed_sink: Optional[float] = None, softcap: Optional[float] = None,
                  values_are_keys: bool = False, gate=False, qk_norm_weight: bool = False,
-                 qk_norm_first: bool = False):
+                 qk_norm_first: bool = False, bias_slopes: Optional[Sequence[float]] = None,
+                 pool: Optional[int] = None):
         if n_heads <= 0 or n_kv_heads <= 0 or n_heads % n_kv_heads:
             raise ValueError(f"n_heads {n_heads} must be a positive multiple of n_kv_heads {n_kv_heads}")
         self.runtime = runtime
@@ -67,6 +79,13 @@ class SinkAttention(Mixer):
         self.chunk, self.window = int(chunk) if chunk else 0, int(window) if window else 0
         if self.chunk < 0 or self.window < 0 or (self.chunk and self.window):
             raise ValueError("give a chunk size or a window, both positive, not both")
+        self.pool = int(pool) if pool else 0
+        if self.pool < 0 or (self.pool and (not self.window or self.values_are_keys)):
+            raise ValueError("pooled blocks need a window before which they lie, and values of their own")
+        if bias_slopes is not None and len(bias_slopes) != self.n_heads:
+            raise ValueError(f"{n_heads} heads need {n_heads} slopes, got {len(bias_slopes)}")
+        self.slopes = None if bias_slopes is None else torch.tensor([float(x) for x in bias_slopes], dtype=torch.float32,
+                                                                    device=runtime.device)
         self.position = build_part(POSITION_ENCODINGS, position, runtime)
         self.wqkv = self.wo = self.b = self.sinks = self.sinks_l2 = self.q_norm = self.k_norm = None
         # values that are the keys, at sizes the tensor-core kernels take: those kernels read keys and values from
@@ -125,11 +144,12 @@ class SinkAttention(Mixer):
     def cache_spec(self) -> CacheSpec:
         policy = "chunk" if self.chunk else ("window" if self.window else "full")
         span = self.chunk or self.window or None
+        pool = self.pool
         if self.values_are_keys and not self.copy_keys:
             return CacheSpec(policy, (self.n_kv_heads * self.head_dim,), span, tensors=1)
         if self.v_dim == self.head_dim:
-            return CacheSpec(policy, (self.n_kv_heads, self.head_dim), span)
-        return CacheSpec(policy, (self.n_kv_heads * (self.head_dim + self.v_dim),), span, tensors=1)
+            return CacheSpec(policy, (self.n_kv_heads, self.head_dim), span, pool=pool)
+        return CacheSpec(policy, (self.n_kv_heads * (self.head_dim + self.v_dim),), span, tensors=1, pool=pool)
 
     def forward(self, x, ctx, cache):
         out = self.pre_projection(x, ctx, cache)
@@ -143,6 +163,8 @@ class SinkAttention(Mixer):
         H, G, hd, vd = self.n_heads, self.n_kv_heads, self.head_dim, self.v_dim
         tables = ctx.tables[cache.group]
         pos = self.position
+        pooled = (self.pool, cache.pooled, ctx.tables[cache.pooled_group]) if self.pool else None
+        one_each = ctx.max_q_len == 1             # a token that completes a block finds the block's others in the cache
         with bucket("attn.qkv_proj"):
             proj = ops.linear(x, self.wqkv, out_dtype=torch.float32)
         qkv = proj[:, :self.qkv_width]
@@ -152,7 +174,11 @@ class SinkAttention(Mixer):
                                 getattr(pos, "rotary_dim", 0), getattr(pos, "interleaved", False),
                                 getattr(pos, "magnitude", 1.0), self.qk_norm_eps, ctx.positions, ctx.tok_entry,
                                 tables.kv_indptr, tables.kv_indices, cache.kv, tables.page_size, write_kv=cache.owner,
-                                q_norm=self.q_norm, k_norm=self.k_norm, norm_first=self.qk_norm_first)
+                                q_norm=self.q_norm, k_norm=self.k_norm, norm_first=self.qk_norm_first,
+                                pooled=pooled if one_each and cache.owner else None)
+        if pooled is not None and not one_each and cache.owner:
+            with bucket("attn.pool"):
+                ops.pool_append(cache.kv, ctx, tables, pooled, G, hd, vd)
         if out is None:
             out = torch.empty((n, H * vd), dtype=x.dtype, device=x.device)
         with bucket("attn.compute"):
@@ -163,7 +189,7 @@ class SinkAttention(Mixer):
                 direct = not self.gate and out_scale == 1.0 and out.is_contiguous()
                 heads = out if direct else torch.empty((n, H * vd), dtype=x.dtype, device=x.device)
                 ops.paged_attention(q, heads, cache.kv, ctx, tables, H, G, hd, self.scale, self.window, self.chunk,
-                                    self.sinks, self.sinks_l2, self.softcap)
+                                    self.sinks, self.sinks_l2, self.softcap, self.slopes, pooled)
                 if not direct and self.gate_per_head and out_scale == 1.0 and out.is_contiguous():
                     # one logit per head: the heads [n, H * vd] read as [H, n, vd]
                     ops.gate_heads(heads.view(n, H, vd).transpose(0, 1), gate, out)
@@ -174,5 +200,5 @@ class SinkAttention(Mixer):
             else:
                 ops.masked_attention(q, out, cache.kv, ctx, tables, H, G, hd, vd, self.scale, self.window, self.chunk,
                                      self.sinks, self.softcap, self.values_are_keys and not self.copy_keys, gate,
-                                     out_scale, gate_per_head=self.gate_per_head)
+                                     out_scale, gate_per_head=self.gate_per_head, slopes=self.slopes, pooled=pooled)
         return out
