@@ -74,6 +74,24 @@ struct TileGeom {
   int e, g, q_begin, q_len, pos0, G, rows_total;
 };
 
+// Pooled blocks before a window: ``size`` tokens each (0: none), with their block tables.  Their entries are keys of a
+// second source, visited before the tokens: key number b is block b, seen by a query if b < pooled_seen(query).
+struct Pooled {
+  int size;
+  const int* indptr;
+  const int* indices;
+};
+
+// The distance-bias slopes (times log2 e) of a thread's two rows: rows row0 + lane / 4 and 8 further.
+__device__ __forceinline__ void row_slopes(float (&sl)[2], const float* __restrict__ slopes_l2, int g, int G, int row0,
+                                           int rows_total) {
+#pragma unroll
+  for (int r = 0; r < 2; ++r) {
+    const int row = row0 + ((threadIdx.x & 31) >> 2) + 8 * r;
+    sl[r] = slopes_l2 != nullptr && row < rows_total ? slopes_l2[g * G + row % G] : 0.f;
+  }
+}
+
 // Load K and V rows [k0, k0 + KT) of one kv head into swizzled shared tiles; keys outside [k_lo, k_end) are
 // zero-filled and their table entries (which may be released pages) are not read.
 template <int HD>
@@ -130,11 +148,13 @@ __device__ __forceinline__ float score2(float s, float scale_log2, float softcap
 
 // One warp: scores of its 16 rows against 16 keys (kb .. kb+15 of the tile), online softmax, P*V.
 // qf: A fragments of the rows for every 16-dim step.  Row state (m, l) per thread for rows lane/4 and lane/4+8.
+// ``slope2``: the rows' distance-bias slopes times log2(e) (``biased``): slope (key - limit) joins a score, a row's limit
+// being its own position.
 template <int HD, bool TMA_TILE = false>
 __device__ __forceinline__ void block16(const uint32_t (&qf)[HD / 16][4], const __nv_bfloat16* Ks,
                                         const __nv_bfloat16* Vs, int kb, int key0, int row_lim0, int row_lim1,
-                                        int row_lo0, int row_lo1, int k_end, float scale_log2, float softcap, float (&m)[2],
-                                        float (&l)[2], float (&o)[HD / 8][4]) {
+                                        int row_lo0, int row_lo1, int k_end, float scale_log2, float softcap, bool biased,
+                                        const float (&slope2)[2], float (&m)[2], float (&l)[2], float (&o)[HD / 8][4]) {
   const int lane = threadIdx.x & 31;
   float s[2][4];
 #pragma unroll
@@ -159,6 +179,7 @@ __device__ __forceinline__ void block16(const uint32_t (&qf)[HD / 16][4], const 
       const int lim = (i >> 1) ? row_lim1 : row_lim0, lo = (i >> 1) ? row_lo1 : row_lo0;
       const bool ok = key <= lim && key >= lo && key < k_end;
       s[nt][i] = ok ? score2(s[nt][i], scale_log2, softcap) : -INFINITY;
+      if (biased) s[nt][i] += slope2[i >> 1] * (float)(key - lim);
       mx[i >> 1] = fmaxf(mx[i >> 1], s[nt][i]);
     }
   float corr[2], msafe[2];
@@ -332,7 +353,7 @@ attn_decode_kernel(const __nv_bfloat16* __restrict__ q, long long q_row_stride, 
                    const int* __restrict__ positions, const int* __restrict__ kv_indptr,
                    const int* __restrict__ kv_indices, int Hq, int Hkv, int page_size, float scale_log2, float softcap, int window,
                    int n_splits, int row_tiles, int max_q_short, long long n_pages,
-                    const float* __restrict__ sink_l2) {
+                    const float* __restrict__ sink_l2, const float* __restrict__ slopes_l2) {
   bspec::pdl_prologue(8);
   extern __shared__ __align__(16) unsigned char smem_raw[];
   __nv_bfloat16* Qs = reinterpret_cast<__nv_bfloat16*>(smem_raw);           // [16][HD]
@@ -367,6 +388,8 @@ attn_decode_kernel(const __nv_bfloat16* __restrict__ q, long long q_row_stride, 
     lim[r] = row < t.rows_total ? t.pos0 + qi : -1;
     lo[r] = bspec::mask_lo(t.pos0 + qi, window);
   }
+  float sl[2];
+  row_slopes(sl, slopes_l2, g, t.G, row0, t.rows_total);
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
   float o[HD / 8][4];
 #pragma unroll
@@ -410,7 +433,8 @@ attn_decode_kernel(const __nv_bfloat16* __restrict__ q, long long q_row_stride, 
       __syncthreads();
       const int key0 = k_begin + it * KT;
       if (key0 + 16 * warp < k_end)
-        block16<HD>(qf, Ks, Vs, 16 * warp, key0, lim[0], lim[1], lo[0], lo[1], k_end, scale_log2, softcap, m, l, o);
+        block16<HD>(qf, Ks, Vs, 16 * warp, key0, lim[0], lim[1], lo[0], lo[1], k_end, scale_log2, softcap,
+                    slopes_l2 != nullptr, sl, m, l, o);
       __syncthreads();
     }
   }
@@ -436,7 +460,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap kv_map, const __nv_bf
                        const int* __restrict__ qo_indptr, const int* __restrict__ positions,
                        const int* __restrict__ kv_indptr, const int* __restrict__ kv_indices, int Hq, int Hkv,
                        int page_size, float scale_log2, float softcap, int window, int n_splits, int row_tiles, int max_q_short,
-                    const float* __restrict__ sink_l2) {
+                    const float* __restrict__ sink_l2, const float* __restrict__ slopes_l2) {
   // The step's metadata (lengths, positions, block tables) was uploaded before the step's first kernel, and every
   // cached key below the first new token was written by earlier steps: the producer may fetch those tiles while
   // the kernel before this one (which writes q and the new tokens' keys and values) is still running.
@@ -544,6 +568,8 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap kv_map, const __nv_bf
     lo[r] = bspec::mask_lo(t.pos0 + qi, window);
   }
   if (n_tiles > 0) {
+    float sl[2];
+    row_slopes(sl, slopes_l2, g, t.G, row0, t.rows_total);
     load_q_tile<HD>(Qs, q, q_row_stride, t, row0, 16);
     bar_consumers();
     uint32_t qf[HD / 16][4];
@@ -561,7 +587,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap kv_map, const __nv_bf
       const int key0 = k_begin + it * KT;
       if (key0 + 16 * warp < k_end)
         block16<HD, true>(qf, Ks, Ks + TILE_ELEMS, 16 * warp, key0, lim[0], lim[1], lo[0], lo[1], k_end, scale_log2,
-                          softcap, m, l, o);
+                          softcap, slopes_l2 != nullptr, sl, m, l, o);
       __syncwarp();
       if (lane == 0) mbar_arrive(empty + s);
     }
@@ -601,6 +627,8 @@ struct Shares {
 struct Piece {
   TileGeom t;
   int e, g, rt, row0, k_begin, k_end, n_tiles, lo_key;
+  int n_pool, pool_k0;   // the first n_pool of the n_tiles are tiles of pooled blocks, from block pool_k0
+  int pool_end;          // blocks that the request's last new token sees
   int part, n_parts;     // which partial result of the row tile this is, of how many (1: written at once)
   int tiles_taken;       // tiles of the sequence this piece covers (>= n_tiles: masked tiles are not fetched)
 };
@@ -608,7 +636,7 @@ struct Piece {
 // The piece that starts at position `pos` of the sequence and ends with its row tile or with the CTA's share.
 __device__ __forceinline__ void piece_at(Piece& pc, long long pos, long long share_end, int b, const Shares& sh,
                                          const int* pos0_of, const int* rows_of, int n_entries, int Hq, int Hkv,
-                                         int row_tiles, int window) {
+                                         int row_tiles, int window, int pool) {
   int lo = 0, hi = n_entries;                    // largest e with cum[e] <= pos
   while (hi - lo > 1) {
     const int mid = (lo + hi) >> 1;
@@ -636,17 +664,26 @@ __device__ __forceinline__ void piece_at(Piece& pc, long long pos, long long sha
   t.G = Hq / Hkv;
   t.rows_total = t.q_len * t.G;
   pc.row0 = pc.rt * 16;
-  pc.n_tiles = 0;
+  pc.n_tiles = pc.n_pool = pc.pool_k0 = pc.pool_end = 0;
   pc.k_begin = pc.k_end = pc.lo_key = 0;
   if (pc.row0 >= t.rows_total) return;
+  int skip = 0;                                  // the request's tiles of pooled blocks come before its tokens' tiles
+  if (pool > 0) {
+    pc.pool_end = bspec::pooled_seen(t.pos0 + t.q_len - 1, window, pool);
+    skip = (pc.pool_end + KT - 1) / KT;
+    pc.n_pool = max(0, min(t1, skip) - t0);
+    pc.pool_k0 = t0 * KT;
+  }
+  const int r0 = max(t0 - skip, 0), r1 = max(t1 - skip, 0);
   const int qi_lo = pc.row0 / t.G, qi_hi = min(t.q_len - 1, (pc.row0 + 15) / t.G);
   const int hi_key = t.pos0 + qi_hi;
   pc.lo_key = bspec::mask_lo(t.pos0 + qi_lo, window);
   const int lo_entry = bspec::mask_lo(t.pos0, window);      // the request's tiles start here
   const int lo_al = (lo_entry / KT) * KT;
-  pc.k_begin = lo_al + t0 * KT;
-  pc.k_end = min(hi_key + 1, lo_al + t1 * KT);
-  if (pc.k_begin < pc.k_end && pc.lo_key < pc.k_end) pc.n_tiles = (pc.k_end - pc.k_begin + KT - 1) / KT;
+  pc.k_begin = lo_al + r0 * KT;
+  pc.k_end = min(hi_key + 1, lo_al + r1 * KT);
+  pc.n_tiles = pc.n_pool;
+  if (pc.k_begin < pc.k_end && pc.lo_key < pc.k_end) pc.n_tiles += (pc.k_end - pc.k_begin + KT - 1) / KT;
 }
 
 // Tiles per request and their running sum (all threads of the CTA call this); also every request's first position
@@ -655,7 +692,7 @@ __device__ __forceinline__ void piece_at(Piece& pc, long long pos, long long sha
 __device__ __forceinline__ bool make_shares(Shares& sh, int* cum, int* pos0_of, int* rows_of, int* red, int n_entries,
                                             const int* __restrict__ qo_indptr, const int* __restrict__ positions,
                                             const int* __restrict__ kv_len, int Hkv, int row_tiles, int window,
-                                            int max_parts, int max_q_short, int n_threads, int grid) {
+                                            int max_parts, int max_q_short, int n_threads, int grid, int pool) {
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   int most = 0, fewest = 0x7fffffff, live = 0;
   for (int e = threadIdx.x; e < n_entries; e += n_threads) {
@@ -666,6 +703,7 @@ __device__ __forceinline__ bool make_shares(Shares& sh, int* cum, int* pos0_of, 
       pos0 = kv_len != nullptr ? len_after - ql : positions[qb];
       const int lo_entry = bspec::mask_lo(pos0, window);
       tiles = (pos0 + ql - (lo_entry / KT) * KT + KT - 1) / KT;
+      if (pool > 0) tiles += (bspec::pooled_seen(pos0 + ql - 1, window, pool) + KT - 1) / KT;
     }
     pos0_of[e] = pos0;
     rows_of[e] = qb | (tiles > 0 ? ql << 26 : 0);
@@ -785,8 +823,9 @@ __device__ __forceinline__ void join_parts(float* Wt, __nv_bfloat16* __restrict_
   bar_consumers();
 }
 
-template <int HD>
-__global__ void __launch_bounds__(DECODE_TMA_THREADS)
+// MORE: a distance bias or pooled blocks may be given; without it the code for both is left out.
+template <int HD, bool MORE>
+__global__ void __launch_bounds__(DECODE_TMA_THREADS, HD <= 64 ? 3 : (HD <= 128 ? 2 : 1))
 attn_decode_shares_kernel(const __grid_constant__ CUtensorMap kv_map, const __nv_bfloat16* __restrict__ q,
                           long long q_row_stride, __nv_bfloat16* __restrict__ out, float* __restrict__ o_part,
                           float* __restrict__ ml_part, int* __restrict__ tile_counters, int* __restrict__ status,
@@ -794,8 +833,11 @@ attn_decode_shares_kernel(const __grid_constant__ CUtensorMap kv_map, const __nv
                           const int* __restrict__ kv_len,
                           const int* __restrict__ kv_indptr, const int* __restrict__ kv_indices, int n_entries, int Hq,
                           int Hkv, int page_size, float scale_log2, float softcap, int window, int max_parts, int rows_pe,
-                          int row_tiles, int max_q_short,
-                    const float* __restrict__ sink_l2) {
+                          int row_tiles, int max_q_short, const float* __restrict__ sink_l2,
+                          const float* __restrict__ slopes_in, const __grid_constant__ CUtensorMap pool_map,
+                          const Pooled pooled_in) {
+  const float* __restrict__ slopes_l2 = MORE ? slopes_in : nullptr;
+  const Pooled pooled = MORE ? pooled_in : Pooled{0, nullptr, nullptr};
   // Lengths, positions and block tables were uploaded before the step's first kernel, and every cached key below
   // the first new token was written by earlier steps: all of that may be read, and those tiles fetched, while the
   // kernel before this one (which writes q and the new tokens' keys and values) still runs.
@@ -827,7 +869,7 @@ attn_decode_shares_kernel(const __grid_constant__ CUtensorMap kv_map, const __nv
   }
   Shares sh;
   if (!make_shares(sh, cum, pos0_of, rows_of, red, n_entries, qo_indptr, positions, kv_len, Hkv, row_tiles, window, max_parts,
-                   max_q_short, DECODE_TMA_THREADS, gridDim.x))
+                   max_q_short, DECODE_TMA_THREADS, gridDim.x, pooled.size))
     return;
   const int b = blockIdx.x;
   if (b >= sh.ctas) return;
@@ -842,22 +884,32 @@ attn_decode_shares_kernel(const __grid_constant__ CUtensorMap kv_map, const __nv
     const int pages_per_tile = KT / page_size;
     for (long long pos = share_begin; pos < share_end && ok;) {
       Piece pc;
-      piece_at(pc, pos, share_end, b, sh, pos0_of, rows_of, n_entries, Hq, Hkv, row_tiles, window);
+      piece_at(pc, pos, share_end, b, sh, pos0_of, rows_of, n_entries, Hq, Hkv, row_tiles, window,
+               pooled.size);
       pos += pc.tiles_taken;
       if (pc.n_tiles == 0) continue;
       const int* table = kv_indices + kv_indptr[pc.e];
       const int first_pg = max(pc.k_begin, pc.lo_key) / page_size, last_pg = (pc.k_end - 1) / page_size;
-      const int n_pg = last_pg - first_pg + 1;
-      const bool in_smem = n_pg <= BAL_TBL;
+      const int n_pg = pc.n_tiles > pc.n_pool ? last_pg - first_pg + 1 : 0;
+      // pages of the piece's pooled blocks: in front of the tokens' pages in the shared table
+      const int* ptable = pc.n_pool > 0 ? pooled.indices + pooled.indptr[pc.e] : nullptr;
+      const int first_ppg = pc.pool_k0 / page_size;
+      const int last_ppg = pc.n_pool > 0 ? (min(pc.pool_end, pc.pool_k0 + pc.n_pool * KT) - 1) / page_size : first_ppg - 1;
+      const int n_ppg = last_ppg - first_ppg + 1;
+      const bool in_smem = n_pg + n_ppg <= BAL_TBL;
       __syncwarp();
-      if (in_smem)
-        for (int i = lane; i < n_pg; i += 32) tbl[i] = table[first_pg + i];
+      if (in_smem) {
+        for (int i = lane; i < n_ppg; i += 32) tbl[i] = ptable[first_ppg + i];
+        for (int i = lane; i < n_pg; i += 32) tbl[n_ppg + i] = table[first_pg + i];
+      }
       __syncwarp();
       constexpr uint32_t tile_bytes = 2u * TILE_ELEMS * 2u;
       for (int k = 0; k < pc.n_tiles; ++k, ++tile_no) {
         const int s = tile_no % TMA_STAGES;
         const uint32_t ph = (tile_no / TMA_STAGES) & 1u;
-        if (!waited && (tile_no >= TMA_STAGES || pc.k_begin + (k + 1) * KT > pc.t.pos0)) {
+        const bool blocks = MORE && k < pc.n_pool;
+        const int key0 = blocks ? pc.pool_k0 + k * KT : pc.k_begin + (k - pc.n_pool) * KT;
+        if (!waited && (tile_no >= TMA_STAGES || key0 + KT > (blocks ? pc.t.pos0 / pooled.size : pc.t.pos0))) {
           bspec::pdl_wait();           // this tile holds new keys, or a stage must first be released by consumers
           waited = true;
         }
@@ -872,11 +924,17 @@ attn_decode_shares_kernel(const __grid_constant__ CUtensorMap kv_map, const __nv
         constexpr int PER_PAGE = 2 * (HD / 64);
         for (int bx = lane; bx < pages_per_tile * PER_PAGE; bx += 32) {
           const int pp = bx / PER_PAGE, rem = bx - pp * PER_PAGE, c = rem >> 1, is_v = rem & 1;
-          int pg = (pc.k_begin + k * KT) / page_size + pp;
-          pg = min(max(pg, first_pg), last_pg);
-          const int page = in_smem ? tbl[pg - first_pg] : table[pg];
+          int pg = key0 / page_size + pp, page;
+          if (blocks) {
+            pg = min(pg, last_ppg);
+            page = in_smem ? tbl[pg - first_ppg] : ptable[pg];
+          } else {
+            pg = min(max(pg, first_pg), last_pg);
+            page = in_smem ? tbl[n_ppg + pg - first_pg] : table[pg];
+          }
           const int row = ((page * 2 + is_v) * Hkv + pc.g) * page_size;       // first cache row of this page's K (or V)
-          tma_load_2d(Ks + is_v * TILE_ELEMS + c * (KT * 64) + pp * page_size * 64, &kv_map, full + s, c * 64, row);
+          tma_load_2d(Ks + is_v * TILE_ELEMS + c * (KT * 64) + pp * page_size * 64, blocks ? &pool_map : &kv_map, full + s,
+                      c * 64, row);
         }
       }
     }
@@ -892,7 +950,8 @@ attn_decode_shares_kernel(const __grid_constant__ CUtensorMap kv_map, const __nv
   bool aborted = false;
   for (long long pos = share_begin; pos < share_end;) {
     Piece pc;
-    piece_at(pc, pos, share_end, b, sh, pos0_of, rows_of, n_entries, Hq, Hkv, row_tiles, window);
+    piece_at(pc, pos, share_end, b, sh, pos0_of, rows_of, n_entries, Hq, Hkv, row_tiles, window,
+             pooled.size);
     pos += pc.tiles_taken;
     if (pc.row0 >= pc.t.rows_total) continue;               // no such row tile in this request: nothing to write
     const TileGeom& t = pc.t;
@@ -904,14 +963,17 @@ attn_decode_shares_kernel(const __grid_constant__ CUtensorMap kv_map, const __nv
       for (int j = 0; j < 4; ++j) o[i][j] = 0.f;
     int last_stage = -1;
     if (pc.n_tiles > 0) {
-      int lim[2], lo[2];
+      int lim[2], lo[2], blk[2];
 #pragma unroll
       for (int r = 0; r < 2; ++r) {
         const int row = pc.row0 + (lane >> 2) + 8 * r;
         const int qi = row / t.G;
         lim[r] = row < t.rows_total ? t.pos0 + qi : -1;
         lo[r] = bspec::mask_lo(t.pos0 + qi, window);
+        blk[r] = pooled.size > 0 && row < t.rows_total ? bspec::pooled_seen(t.pos0 + qi, window, pooled.size) - 1 : -1;
       }
+      float sl[2];
+      row_slopes(sl, slopes_l2, pc.g, t.G, pc.row0, t.rows_total);
       load_q_tile<HD>(Qs, q, q_row_stride, t, pc.row0, 16);
       bar_consumers();
       uint32_t qf[HD / 16][4];
@@ -926,10 +988,13 @@ attn_decode_shares_kernel(const __grid_constant__ CUtensorMap kv_map, const __nv
         const uint32_t ph = (tile_no / TMA_STAGES) & 1u;
         if (!mbar_wait(full + s, ph, abort_flag, status, 14)) break;   // the flag is set: all warps leave below
         const __nv_bfloat16* Ks = KV + (size_t)s * 2 * TILE_ELEMS;
-        const int key0 = pc.k_begin + k * KT;
-        if (key0 + 16 * warp < pc.k_end)
-          block16<HD, true>(qf, Ks, Ks + TILE_ELEMS, 16 * warp, key0, lim[0], lim[1], lo[0], lo[1], pc.k_end,
-                            scale_log2, softcap, m, l, o);
+        const bool blocks = MORE && k < pc.n_pool;
+        const int key0 = blocks ? pc.pool_k0 + k * KT : pc.k_begin + (k - pc.n_pool) * KT;
+        const int k_end = blocks ? pc.pool_end : pc.k_end;
+        if (key0 + 16 * warp < k_end)
+          block16<HD, true>(qf, Ks, Ks + TILE_ELEMS, 16 * warp, key0, blocks ? blk[0] : lim[0], blocks ? blk[1] : lim[1],
+                            blocks ? 0 : lo[0], blocks ? 0 : lo[1], k_end, scale_log2, softcap, slopes_l2 != nullptr, sl,
+                            m, l, o);
         __syncwarp();
         if (k + 1 < pc.n_tiles) {
           if (lane == 0) mbar_arrive(empty + s);
@@ -1059,8 +1124,8 @@ template <int HD> size_t decode_shares_smem() {
 template <int HD, bool TMA_TILE>
 __device__ __forceinline__ void block64(const uint32_t (&qf)[HD / 16][4], const __nv_bfloat16* Ks,
                                         const __nv_bfloat16* Vs, int key0, int row_lim0, int row_lim1, int row_lo0,
-                                        int row_lo1, int k_end, bool need_mask, float scale_log2, float softcap, float (&m)[2],
-                                        float (&l)[2], float (&o)[HD / 8][4]) {
+                                        int row_lo1, int k_end, bool need_mask, float scale_log2, float softcap, bool biased,
+                                        const float (&slope2)[2], float (&m)[2], float (&l)[2], float (&o)[HD / 8][4]) {
   const int lane = threadIdx.x & 31;
   const int mat = lane >> 3, r8 = lane & 7;
   float s[8][4];
@@ -1088,6 +1153,7 @@ __device__ __forceinline__ void block64(const uint32_t (&qf)[HD / 16][4], const 
         const int lim = (i >> 1) ? row_lim1 : row_lim0, lo = (i >> 1) ? row_lo1 : row_lo0;
         const bool ok = key <= lim && key >= lo && key < k_end;
         s[nt][i] = ok ? score2(s[nt][i], scale_log2, softcap) : -INFINITY;
+        if (biased) s[nt][i] += slope2[i >> 1] * (float)(key - lim);
         mx[i >> 1] = fmaxf(mx[i >> 1], s[nt][i]);
       }
   } else {
@@ -1096,6 +1162,8 @@ __device__ __forceinline__ void block64(const uint32_t (&qf)[HD / 16][4], const 
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
         s[nt][i] = score2(s[nt][i], scale_log2, softcap);
+        if (biased)
+          s[nt][i] += slope2[i >> 1] * (float)(key0 + 8 * nt + 2 * (lane & 3) + (i & 1) - ((i >> 1) ? row_lim1 : row_lim0));
         mx[i >> 1] = fmaxf(mx[i >> 1], s[nt][i]);
       }
   }
@@ -1144,14 +1212,17 @@ constexpr int PREFILL_ROWS = 128;
 constexpr int PREFILL_TMA_THREADS = 288;
 constexpr int PREFILL_STAGES = 4;     // one CTA per SM (registers): a deep ring hides the load latency instead
 
-template <int HD>
+template <int HD, bool MORE>
 __global__ void __launch_bounds__(PREFILL_TMA_THREADS)
 attn_prefill_tma_kernel(const __grid_constant__ CUtensorMap kv_map, const __nv_bfloat16* __restrict__ q,
                         long long q_row_stride, __nv_bfloat16* __restrict__ out, int* __restrict__ status,
                         const int* __restrict__ qo_indptr, const int* __restrict__ positions,
                         const int* __restrict__ kv_indptr, const int* __restrict__ kv_indices, int Hq, int Hkv,
                         int page_size, float scale_log2, float softcap, int window, int min_q_long,
-                    const float* __restrict__ sink_l2) {
+                        const float* __restrict__ sink_l2, const float* __restrict__ slopes_in,
+                        const __grid_constant__ CUtensorMap pool_map, const Pooled pooled_in) {
+  const float* __restrict__ slopes_l2 = MORE ? slopes_in : nullptr;
+  const Pooled pooled = MORE ? pooled_in : Pooled{0, nullptr, nullptr};
   bspec::pdl_prologue(9);
   extern __shared__ unsigned char smem_dyn[];
   unsigned char* smem = reinterpret_cast<unsigned char*>(((uintptr_t)smem_dyn + 1023) & ~(uintptr_t)1023);
@@ -1174,7 +1245,9 @@ attn_prefill_tma_kernel(const __grid_constant__ CUtensorMap kv_map, const __nv_b
   const int hi_key = t.pos0 + qi_hi;
   const int lo_key = bspec::mask_lo(t.pos0 + qi_lo, window);
   const int k_begin = (lo_key / KT) * KT, k_end = hi_key + 1;
-  const int n_tiles = (k_end - k_begin + KT - 1) / KT;
+  const int pool_end = pooled.size > 0 ? bspec::pooled_seen(hi_key, window, pooled.size) : 0;
+  const int n_pool = (pool_end + KT - 1) / KT;                                // tiles of pooled blocks, before the tokens'
+  const int n_tiles = n_pool + (k_end - k_begin + KT - 1) / KT;
   const int* table = kv_indices + kv_indptr[e];
 
   if (threadIdx.x == 0) {
@@ -1198,17 +1271,20 @@ attn_prefill_tma_kernel(const __grid_constant__ CUtensorMap kv_map, const __nv_b
         if (!mbar_wait(empty + s, ph ^ 1u, abort_flag, status, 21)) break;
         __nv_bfloat16* Ks = KV + (size_t)s * 2 * TILE_ELEMS;
         mbar_expect_tx(full + s, tile_bytes);
-        const int key0 = k_begin + it * KT;
+        const bool blocks = MORE && it < n_pool;
+        const int key0 = blocks ? it * KT : k_begin + (it - n_pool) * KT;
+        const int* tab = blocks ? pooled.indices + pooled.indptr[e] : table;
+        const CUtensorMap* map = blocks ? &pool_map : &kv_map;
         for (int pp = 0; pp < pages_per_tile; ++pp) {
           int pg = (key0 + pp * page_size) / page_size;
-          pg = min(max(pg, first_pg), last_pg);
-          const int page = table[pg];
+          pg = blocks ? min(pg, (pool_end - 1) / page_size) : min(max(pg, first_pg), last_pg);
+          const int page = tab[pg];
           const int row_k = ((page * 2) * Hkv + g) * page_size;
           const int row_v = row_k + Hkv * page_size;
 #pragma unroll
           for (int c = 0; c < HD / 64; ++c) {
-            tma_load_2d(Ks + c * (KT * 64) + pp * page_size * 64, &kv_map, full + s, c * 64, row_k);
-            tma_load_2d(Ks + TILE_ELEMS + c * (KT * 64) + pp * page_size * 64, &kv_map, full + s, c * 64, row_v);
+            tma_load_2d(Ks + c * (KT * 64) + pp * page_size * 64, map, full + s, c * 64, row_k);
+            tma_load_2d(Ks + TILE_ELEMS + c * (KT * 64) + pp * page_size * 64, map, full + s, c * 64, row_v);
           }
         }
       }
@@ -1218,14 +1294,17 @@ attn_prefill_tma_kernel(const __grid_constant__ CUtensorMap kv_map, const __nv_b
 
   // ---- consumers: warps 0..7
   const int wrow0 = row0 + 16 * warp;
-  int lim[2], lo[2];
+  int lim[2], lo[2], blk[2];
 #pragma unroll
   for (int r = 0; r < 2; ++r) {
     const int row = wrow0 + (lane >> 2) + 8 * r;
     const int qi = row / t.G;
     lim[r] = row < t.rows_total ? t.pos0 + qi : -1;
     lo[r] = bspec::mask_lo(t.pos0 + qi, window);
+    blk[r] = pooled.size > 0 && row < t.rows_total ? bspec::pooled_seen(t.pos0 + qi, window, pooled.size) - 1 : -1;
   }
+  float sl[2];
+  row_slopes(sl, slopes_l2, g, t.G, wrow0, t.rows_total);
   const bool warp_live = wrow0 < t.rows_total;
   const int warp_hi = t.pos0 + min(t.q_len - 1, (wrow0 + 15) / t.G);          // last key any row of the warp sees
   const int warp_full = t.pos0 + wrow0 / t.G;                                 // keys <= this are seen by all its rows
@@ -1264,11 +1343,13 @@ attn_prefill_tma_kernel(const __grid_constant__ CUtensorMap kv_map, const __nv_b
     const uint32_t ph = (uint32_t)(it / PREFILL_STAGES) & 1u;
     if (!mbar_wait(full + s, ph, abort_flag, status, 22)) break;
     const __nv_bfloat16* Ks = KV + (size_t)s * 2 * TILE_ELEMS;
-    const int key0 = k_begin + it * KT;
-    if (warp_live && key0 <= warp_hi) {
-      const bool need_mask = key0 + KT - 1 > warp_full || key0 < warp_lo || key0 + KT > k_end;
-      block64<HD, true>(qf, Ks, Ks + TILE_ELEMS, key0, lim[0], lim[1], lo[0], lo[1], k_end, need_mask, scale_log2, softcap, m,
-                        l, o);
+    const bool blocks = MORE && it < n_pool;
+    const int key0 = blocks ? it * KT : k_begin + (it - n_pool) * KT;
+    if (warp_live && (blocks || key0 <= warp_hi)) {
+      const bool need_mask = blocks || key0 + KT - 1 > warp_full || key0 < warp_lo || key0 + KT > k_end;
+      block64<HD, true>(qf, Ks, Ks + TILE_ELEMS, key0, blocks ? blk[0] : lim[0], blocks ? blk[1] : lim[1],
+                        blocks ? 0 : lo[0], blocks ? 0 : lo[1], blocks ? pool_end : k_end, need_mask, scale_log2, softcap,
+                        slopes_l2 != nullptr, sl, m, l, o);
     }
     __syncwarp();
     if (lane == 0) mbar_arrive(empty + s);
@@ -1307,7 +1388,7 @@ attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, long long q_row_stride,
                     const int* __restrict__ positions, const int* __restrict__ kv_indptr,
                     const int* __restrict__ kv_indices, int Hq, int Hkv, int page_size, float scale_log2, float softcap, int window,
                     int min_q_long, long long n_pages,
-                    const float* __restrict__ sink_l2) {
+                    const float* __restrict__ sink_l2, const float* __restrict__ slopes_l2) {
   bspec::pdl_prologue(9);
   extern __shared__ __align__(16) unsigned char smem_raw[];
   __nv_bfloat16* Qs = reinterpret_cast<__nv_bfloat16*>(smem_raw);           // [64][HD]
@@ -1338,6 +1419,8 @@ attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, long long q_row_stride,
   // keys this warp's rows can see at all (skip tiles beyond its own last row)
   const int warp_hi = t.pos0 + min(t.q_len - 1, (wrow0 + 15) / t.G);
   const bool warp_live = wrow0 < t.rows_total;
+  float sl[2];
+  row_slopes(sl, slopes_l2, g, t.G, wrow0, t.rows_total);
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
   float o[HD / 8][4];
 #pragma unroll
@@ -1374,7 +1457,8 @@ attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, long long q_row_stride,
 #pragma unroll
       for (int kb = 0; kb < KT; kb += 16)
         if (key0 + kb <= warp_hi)
-          block16<HD>(qf, Ks, Vs, kb, key0, lim[0], lim[1], lo[0], lo[1], k_end, scale_log2, softcap, m, l, o);
+          block16<HD>(qf, Ks, Vs, kb, key0, lim[0], lim[1], lo[0], lo[1], k_end, scale_log2, softcap,
+                      slopes_l2 != nullptr, sl, m, l, o);
     }
     __syncthreads();
   }
@@ -1411,7 +1495,9 @@ int launch(const __nv_bfloat16* q, long long q_row_stride, __nv_bfloat16* out, f
            const int* kv_indptr, const int* kv_indices, int n_entries, int n_tokens, int max_q_len, int Hq, int Hkv,
            int page_size, float scale, int window, int n_splits, int max_q_short, int run_decode, int run_prefill,
            cudaStream_t stream, int balanced = 0, const int* kv_len = nullptr,
-           long long check_pages = 0x7fffffffffffll, const float* sink_l2 = nullptr, float softcap = 0.f) {
+           long long check_pages = 0x7fffffffffffll, const float* sink_l2 = nullptr, float softcap = 0.f,
+           const float* slopes_l2 = nullptr, const Pooled& pooled = Pooled{0, nullptr, nullptr},
+           const __nv_bfloat16* pool_cache = nullptr, long long pool_rows = 0) {
   const float scale_log2 = scale * 1.4426950408889634f;
   const int G = Hq / Hkv;
   // The opt-in to large shared memory and the resident-CTA count are facts of a device: set up once per device,
@@ -1422,19 +1508,26 @@ int launch(const __nv_bfloat16* q, long long q_row_stride, __nv_bfloat16* out, f
   std::call_once(once_dev[cur_dev], [cur_dev]() {
     cudaFuncSetAttribute(attn_decode_kernel<HD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)decode_smem<HD>());
     cudaFuncSetAttribute(attn_decode_tma_kernel<HD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)decode_tma_smem<HD>());
-    cudaFuncSetAttribute(attn_decode_shares_kernel<HD>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                         (int)decode_shares_smem<HD>());
-    cudaFuncSetAttribute(attn_decode_shares_kernel<HD>, cudaFuncAttributePreferredSharedMemoryCarveout, 100);
+    for (const void* kernel : {(const void*)attn_decode_shares_kernel<HD, false>, (const void*)attn_decode_shares_kernel<HD, true>}) {
+      cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)decode_shares_smem<HD>());
+      cudaFuncSetAttribute(kernel, cudaFuncAttributePreferredSharedMemoryCarveout, 100);
+    }
     cudaFuncSetAttribute(attn_prefill_kernel<HD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)prefill_smem<HD>());
     if constexpr (HD <= 128)
-      cudaFuncSetAttribute(attn_prefill_tma_kernel<HD>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                           (int)prefill_tma_smem<HD>());
+      for (const void* kernel : {(const void*)attn_prefill_tma_kernel<HD, false>, (const void*)attn_prefill_tma_kernel<HD, true>})
+        cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)prefill_tma_smem<HD>());
     int per_sm = 0;
-    cudaOccupancyMaxActiveBlocksPerMultiprocessor(&per_sm, attn_decode_shares_kernel<HD>, DECODE_TMA_THREADS,
+    cudaOccupancyMaxActiveBlocksPerMultiprocessor(&per_sm, attn_decode_shares_kernel<HD, false>, DECODE_TMA_THREADS,
                                                   decode_shares_smem<HD>());
     resident_dev[cur_dev] = bspec::sm_count() * (per_sm > 0 ? per_sm : 1);
   });
-  const int resident = resident_dev[cur_dev];
+  const int resident = resident_dev[cur_dev];      // of the plain kernel; a grid above what is resident only costs time
+  const bool more = slopes_l2 != nullptr || pooled.size > 0;
+  // Pooled blocks are served by the kernels that load K/V through TMA: equal shares for the short requests, 128-row
+  // tiles (HD <= 128) for the others.  Where those cannot run, the call is refused (not run without the blocks).
+  CUtensorMap pool_map;
+  if (pooled.size > 0 && (pool_rows <= 0 || !make_map_2d_bf16(&pool_map, pool_cache, pool_rows, HD, page_size, 64)))
+    return (int)cudaErrorInvalidValue;
   if (run_decode) {
     const int short_q = max_q_len < max_q_short ? max_q_len : max_q_short;
     const int row_tiles = (short_q * G + 15) / 16;
@@ -1446,25 +1539,31 @@ int launch(const __nv_bfloat16* q, long long q_row_stride, __nv_bfloat16* out, f
       if (make_map_2d_bf16(&kv_map, cache, kv_rows, HD, page_size, 64)) {
        if (balanced && n_entries <= BAL_MAX_ENTRIES && n_splits >= 4 && n_splits <= 64 && n_tokens < (1 << 26)) {
         // equal shares of the tiles over as many CTAs as the device holds at once, then the join
-        BSPEC_LAUNCH((attn_decode_shares_kernel<HD>), dim3(resident), DECODE_TMA_THREADS, decode_shares_smem<HD>(),
-                     stream, kv_map, q, q_row_stride, out, o_part, ml_part, tile_counters, status, qo_indptr, positions,
-                     kv_len, kv_indptr, kv_indices, n_entries, Hq, Hkv, page_size, scale_log2, softcap, window, n_splits,
-                     short_q, row_tiles, max_q_short, sink_l2);
+#define GO(MORE) \
+        BSPEC_LAUNCH((attn_decode_shares_kernel<HD, MORE>), dim3(resident), DECODE_TMA_THREADS, decode_shares_smem<HD>(), \
+                     stream, kv_map, q, q_row_stride, out, o_part, ml_part, tile_counters, status, qo_indptr, positions, \
+                     kv_len, kv_indptr, kv_indices, n_entries, Hq, Hkv, page_size, scale_log2, softcap, window, n_splits, \
+                     short_q, row_tiles, max_q_short, sink_l2, slopes_l2, pooled.size > 0 ? pool_map : kv_map, pooled)
+        if (more) GO(true); else GO(false);
+#undef GO
         launched = true;
        }
       }
+      if (!launched && pooled.size > 0) return (int)cudaErrorInvalidValue;
       if (!launched && make_map_2d_bf16(&kv_map, cache, kv_rows, HD, page_size, 64)) {
         BSPEC_LAUNCH((attn_decode_tma_kernel<HD>), grid, DECODE_TMA_THREADS, decode_tma_smem<HD>(), stream, kv_map, q,
                      q_row_stride, out, o_part, ml_part, tile_counters, status, qo_indptr, positions, kv_indptr,
-                     kv_indices, Hq, Hkv, page_size, scale_log2, softcap, window, n_splits, row_tiles, max_q_short, sink_l2);
+                     kv_indices, Hq, Hkv, page_size, scale_log2, softcap, window, n_splits, row_tiles, max_q_short, sink_l2,
+                     slopes_l2);
         launched = true;
       }
     }
+    if (!launched && pooled.size > 0) return (int)cudaErrorInvalidValue;
     if (!launched)
       BSPEC_LAUNCH((attn_decode_kernel<HD>), grid, NTHREADS, decode_smem<HD>(), stream,
                    q, q_row_stride, out, o_part, ml_part, tile_counters, cache, qo_indptr, positions, kv_indptr,
                    kv_indices, Hq, Hkv, page_size, scale_log2, softcap, window, n_splits, row_tiles, max_q_short, check_pages,
-                   sink_l2);
+                   sink_l2, slopes_l2);
     const int err = (int)cudaGetLastError();
     if (err) return err;
   }
@@ -1476,18 +1575,23 @@ int launch(const __nv_bfloat16* q, long long q_row_stride, __nv_bfloat16* out, f
       CUtensorMap kv_map;
       if (make_map_2d_bf16(&kv_map, cache, kv_rows, HD, page_size, 64)) {
         dim3 grid((max_q_len * G + PREFILL_ROWS - 1) / PREFILL_ROWS, Hkv, n_entries);
-        BSPEC_LAUNCH((attn_prefill_tma_kernel<HD>), grid, PREFILL_TMA_THREADS, prefill_tma_smem<HD>(), stream, kv_map,
-                     q, q_row_stride, out, status, qo_indptr, positions, kv_indptr, kv_indices, Hq, Hkv, page_size,
-                     scale_log2, softcap, window, max_q_short + 1, sink_l2);
+#define GO(MORE) \
+        BSPEC_LAUNCH((attn_prefill_tma_kernel<HD, MORE>), grid, PREFILL_TMA_THREADS, prefill_tma_smem<HD>(), stream, kv_map, \
+                     q, q_row_stride, out, status, qo_indptr, positions, kv_indptr, kv_indices, Hq, Hkv, page_size, \
+                     scale_log2, softcap, window, max_q_short + 1, sink_l2, slopes_l2, pooled.size > 0 ? pool_map : kv_map, \
+                     pooled)
+        if (more) GO(true); else GO(false);
+#undef GO
         launched = true;
       }
      }
     }
+    if (!launched && pooled.size > 0) return (int)cudaErrorInvalidValue;
     if (!launched) {
       dim3 grid((max_q_len * G + 63) / 64, Hkv, n_entries);
       BSPEC_LAUNCH((attn_prefill_kernel<HD>), grid, NTHREADS, prefill_smem<HD>(), stream,
                    q, q_row_stride, out, cache, qo_indptr, positions, kv_indptr, kv_indices, Hq, Hkv, page_size,
-                   scale_log2, softcap, window, max_q_short + 1, check_pages, sink_l2);
+                   scale_log2, softcap, window, max_q_short + 1, check_pages, sink_l2, slopes_l2);
     }
     return (int)cudaGetLastError();
   }
@@ -1515,6 +1619,8 @@ BSPEC_API int bspec_attention_bf16_masked(const void* q, long long q_row_stride,
                                           int max_q_len, int Hq, int Hkv, int hd, int page_size, float scale, int window,
                                           int n_splits, int max_q_short, int run_decode, int run_prefill, int balanced,
                                           const int* kv_len, long long pages_in_all, const float* sink_l2, float softcap,
+                                          const float* slopes_l2, int pool, const void* pool_cache,
+                                          const int* pool_indptr, const int* pool_indices, long long pool_pages,
                                           cudaStream_t stream);
 BSPEC_API int bspec_attention_bf16(const void* q, long long q_row_stride, void* out, float* o_part, float* ml_part,
                                    int* tile_counters, int* status, long long n_pages, const void* cache, const int* qo_indptr, const int* positions,
@@ -1525,12 +1631,16 @@ BSPEC_API int bspec_attention_bf16(const void* q, long long q_row_stride, void* 
   return bspec_attention_bf16_masked(q, q_row_stride, out, o_part, ml_part, tile_counters, status, n_pages, cache,
                                      qo_indptr, positions, tok_entry, kv_indptr, kv_indices, n_entries, n_tokens,
                                      max_q_len, Hq, Hkv, hd, page_size, scale, window, n_splits, max_q_short, run_decode,
-                                     run_prefill, balanced, kv_len, pages_in_all, nullptr, 0.f, stream);
+                                     run_prefill, balanced, kv_len, pages_in_all, nullptr, 0.f, nullptr, 0, nullptr, nullptr,
+                                     nullptr, 0, stream);
 }
 
 // The same with the other masks and a sink.  ``window`` < 0: a chunk mask of -window positions (a query sees the
 // keys of its own chunk).  ``sink_l2`` (may be null): float32 per query head, the sink times log2(e); it joins the
-// softmax denominator as exp(sink).  ``softcap`` c > 0: a scaled score s becomes c tanh(s / c).
+// softmax denominator as exp(sink).  ``softcap`` c > 0: a scaled score s becomes c tanh(s / c).  ``slopes_l2`` (may be
+// null): float32 per query head, a slope times log2(e); slope * (query - key) is taken off a token's score.  ``pool`` P >
+// 0, with a window: before the window a query also sees one entry per block of P tokens that lies wholly before it
+// (pages of the same layout; needs n_pages, ``balanced`` for short requests, and head_dim <= 128 for the others).
 BSPEC_API int bspec_attention_bf16_masked(const void* q, long long q_row_stride, void* out, float* o_part, float* ml_part,
                                           int* tile_counters, int* status, long long n_pages, const void* cache,
                                           const int* qo_indptr, const int* positions, const int* tok_entry,
@@ -1538,14 +1648,20 @@ BSPEC_API int bspec_attention_bf16_masked(const void* q, long long q_row_stride,
                                           int max_q_len, int Hq, int Hkv, int hd, int page_size, float scale, int window,
                                           int n_splits, int max_q_short, int run_decode, int run_prefill, int balanced,
                                           const int* kv_len, long long pages_in_all, const float* sink_l2, float softcap,
+                                          const float* slopes_l2, int pool, const void* pool_cache,
+                                          const int* pool_indptr, const int* pool_indices, long long pool_pages,
                                           cudaStream_t stream) {
   if (n_entries <= 0 || n_tokens <= 0) return 0;
+  if (pool < 0 || (pool > 0 && (window <= 0 || slopes_l2 != nullptr || pool_cache == nullptr || pool_indptr == nullptr)))
+    return (int)cudaErrorInvalidValue;
+  const Pooled pooled = {pool, pool_indptr, pool_indices};
   if (Hq % Hkv != 0 || n_splits < 1 || n_splits > 64) return (int)cudaErrorInvalidValue;
 #define GO(HDV)                                                                                                    \
   return launch<HDV>((const __nv_bfloat16*)q, q_row_stride, (__nv_bfloat16*)out, o_part, ml_part, tile_counters,   \
                      status, n_pages * 2 * Hkv * page_size, (const __nv_bfloat16*)cache, qo_indptr, positions, tok_entry, kv_indptr, kv_indices, n_entries, \
                      n_tokens, max_q_len, Hq, Hkv, page_size, scale, window, n_splits, max_q_short, run_decode,      \
-                     run_prefill, stream, balanced, kv_len, pages_in_all > 0 ? pages_in_all : 0x7fffffffffffll, sink_l2, softcap)
+                     run_prefill, stream, balanced, kv_len, pages_in_all > 0 ? pages_in_all : 0x7fffffffffffll, sink_l2, softcap,   \
+                     slopes_l2, pooled, (const __nv_bfloat16*)pool_cache, pool_pages * 2 * Hkv * page_size)
   if (hd == 64) GO(64);
   if (hd == 128) GO(128);
   if (hd == 256) GO(256);

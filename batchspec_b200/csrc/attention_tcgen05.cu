@@ -23,6 +23,8 @@
 // the (blocking) issues of both tiles stood in one line, and that line was the kernel's critical path.
 // Tensor memory: 2 x 2 S buffers of 64 columns, 2 O accumulators of 128 (all 512 columns).  Every mbarrier wait is
 // bounded; on expiry a code goes to `status`, all roles stop and the tensor memory is given back.
+// With pooled blocks before a window an item walks key tiles of two sources: first the request's block entries (their
+// own pages and table, the same layout), then its tokens; both are tiles of the same ring and the same softmax.
 #include "common.cuh"
 #include "tma.cuh"
 #include <math.h>
@@ -151,7 +153,16 @@ struct Item {
   int e, g, row0;
   int lo_key, k_begin, k_end, n_tiles;
   int n_kt[QT], k_end_t[QT];
+  int n_pool, pool_end;        // key tiles of pooled blocks ahead of the tokens' tiles; blocks the item's last row sees
   const int* table;
+  const int* ptable;
+};
+
+// Pooled blocks before the window: ``size`` tokens each (0: none), with their block tables.
+struct Pooled {
+  int size;
+  const int* indptr;
+  const int* indices;
 };
 
 // The launch's items in the order they are dealt: kv head fastest, then request, then the request's 256-row blocks
@@ -160,7 +171,7 @@ struct Item {
 __device__ __forceinline__ bool load_item(Item& it, int idx, int Hq, int Hkv, int n_entries, int window,
                                           int page_size, int min_q_long, const int* __restrict__ qo_indptr,
                                           const int* __restrict__ positions, const int* __restrict__ kv_indptr,
-                                          const int* __restrict__ kv_indices) {
+                                          const int* __restrict__ kv_indices, const Pooled& pooled) {
   const int g = idx % Hkv, ez = idx / Hkv;
   const int e = ez % n_entries, z = ez / n_entries;
   Geom& t = it.t;
@@ -178,13 +189,18 @@ __device__ __forceinline__ bool load_item(Item& it, int idx, int Hq, int Hkv, in
   const int qi_lo = it.row0 / t.G;
   it.lo_key = bspec::mask_lo(t.pos0 + qi_lo, window);
   it.k_begin = (it.lo_key / KT) * KT;
+  it.pool_end = 0;
+  if (pooled.size > 0)
+    it.pool_end = bspec::pooled_seen(t.pos0 + min(t.q_len - 1, (it.row0 + QT * ROWS - 1) / t.G), window, pooled.size);
+  it.n_pool = (it.pool_end + KT - 1) / KT;
+  it.ptable = it.n_pool > 0 ? pooled.indices + pooled.indptr[e] : nullptr;
 #pragma unroll
   for (int tt = 0; tt < QT; ++tt) {
     const int r_first = it.row0 + tt * ROWS;
     if (r_first < t.rows_total) {
       const int qi_hi = min(t.q_len - 1, (r_first + ROWS - 1) / t.G);
       it.k_end_t[tt] = t.pos0 + qi_hi + 1;
-      it.n_kt[tt] = (it.k_end_t[tt] - it.k_begin + KT - 1) / KT;
+      it.n_kt[tt] = it.n_pool + (it.k_end_t[tt] - it.k_begin + KT - 1) / KT;
     } else {
       it.k_end_t[tt] = it.k_begin;
       it.n_kt[tt] = 0;
@@ -214,6 +230,8 @@ constexpr int ITEM_RING = 8;
 // follow; nothing but the tensor memory allocation is shared between items, so the next item's keys and queries
 // are fetched, and its first two S tiles computed, while the softmax threads still finish and store the item
 // before.  The CTA that leaves last puts the counter back to zero for the next launch.
+// MORE: a distance bias or pooled blocks may be given; without it the code for both is left out.
+template <bool MORE>
 __global__ void __launch_bounds__(THREADS, 1)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap kv_map, const __grid_constant__ CUtensorMap q_map,
                        const __nv_bfloat16* __restrict__ q, long long q_row_stride, __nv_bfloat16* __restrict__ out,
@@ -221,7 +239,10 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap kv_map, const __grid_
                        const int* __restrict__ kv_indptr, const int* __restrict__ kv_indices, int Hq, int Hkv,
                        int n_entries, int n_items, int page_size, float scale_log2, int window, int min_q_long,
                        int q_by_tma, int* __restrict__ work, const float* __restrict__ sink_l2, float cap_raw,
-                       float cap_x2) {
+                       float cap_x2, const float* __restrict__ slopes_in, float inv_scale,
+                       const __grid_constant__ CUtensorMap pool_map, const Pooled pooled_in) {
+  const float* __restrict__ slopes = MORE ? slopes_in : nullptr;
+  const Pooled pooled = MORE ? pooled_in : Pooled{0, nullptr, nullptr};
   // The step's lengths, positions and block tables were uploaded before its first kernel: the set-up below and the
   // look-up of the CTA's first item read nothing that the kernel before this one writes, so they run under its
   // tail; q, the new tokens' keys and `out` are touched only after the wait.
@@ -274,7 +295,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap kv_map, const __grid_
   bool first_found = false;
   if (warp == 0)
     first_found = load_item(it, blockIdx.x, Hq, Hkv, n_entries, window, page_size, min_q_long, qo_indptr, positions,
-                            kv_indptr, kv_indices);
+                            kv_indptr, kv_indices, pooled);
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
@@ -315,7 +336,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap kv_map, const __grid_
       }
       while (cand < n_items && !found) {
         found = load_item(it, cand, Hq, Hkv, n_entries, window, page_size, min_q_long, qo_indptr, positions, kv_indptr,
-                          kv_indices);
+                          kv_indices, pooled);
         if (!found) draw();
       }
       if (!found) it.n_tiles = -1;
@@ -343,8 +364,10 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap kv_map, const __grid_
         if (!ok) break;
       }
       const int first_pg = it.lo_key / page_size, last_pg = max(first_pg, (it.k_end - 1) / page_size);
+      const int last_ppg = (max(it.pool_end, 1) - 1) / page_size;
       auto page_of = [&](int j) -> int {
-        int pg = (it.k_begin + j * KT) / page_size + lane;
+        if (MORE && j < it.n_pool) return it.ptable[min((j * KT) / page_size + lane, last_ppg)];
+        int pg = (it.k_begin + (MORE ? j - it.n_pool : j) * KT) / page_size + lane;
         pg = min(max(pg, first_pg), last_pg);
         return it.table[pg];
       };
@@ -364,10 +387,11 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap kv_map, const __grid_
           __nv_bfloat16* Ks = KV + (size_t)st * 2 * KTILE;
           const int row_k = ((page * 2) * Hkv + it.g) * page_size;
           const int row_v = row_k + Hkv * page_size;
+          const CUtensorMap* map = MORE && j < it.n_pool ? &pool_map : &kv_map;
 #pragma unroll
           for (int c = 0; c < 2; ++c) {
-            tma_load_2d(Ks + c * SUBK + lane * page_size * 64, &kv_map, kv_full + st, c * 64, row_k);
-            tma_load_2d(Ks + KTILE + c * SUBK + lane * page_size * 64, &kv_map, kv_full + st, c * 64, row_v);
+            tma_load_2d(Ks + c * SUBK + lane * page_size * 64, map, kv_full + st, c * 64, row_k);
+            tma_load_2d(Ks + KTILE + c * SUBK + lane * page_size * 64, map, kv_full + st, c * 64, row_v);
           }
         }
       }
@@ -476,6 +500,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap kv_map, const __grid_
       const int lim = live ? t.pos0 + qi : -1;
       const int lo = bspec::mask_lo(t.pos0 + qi, window);
       const int my_k_end = it.k_end_t[tt];
+      const int last_block = live && pooled.size > 0 ? bspec::pooled_seen(t.pos0 + qi, window, pooled.size) - 1 : -1;
+      const float slope = slopes != nullptr ? slopes[h] * inv_scale : 0.f;      // in units of the raw scores
       if (!q_by_tma) {
         // Q tile: this thread copies its own row (16 chunks of 16 bytes) into the swizzled operand layout.  The
         // S products of the item before are long complete: this thread has waited for that item's last P V,
@@ -501,8 +527,10 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap kv_map, const __grid_
         ok = mbar_wait(s_full + 2 * tt + b, (n >> 1) & 1u, abort_flag, status, 36);
         if (!ok) break;
         tc_fence_after();
-        const int key0 = it.k_begin + j * KT;
-        const bool need_mask = key0 + KT - 1 > lim || key0 < lo || key0 + KT > my_k_end;
+        const bool blocks = MORE && j < it.n_pool;                // a tile of pooled blocks: the numbers are blocks'
+        const int key0 = blocks ? j * KT : it.k_begin + (MORE ? j - it.n_pool : j) * KT;
+        const int hi_j = blocks ? last_block : lim, lo_j = blocks ? 0 : lo, end_j = blocks ? it.pool_end : my_k_end;
+        const bool need_mask = key0 + KT - 1 > hi_j || key0 < lo_j || key0 + KT > end_j;
         // the whole S row into registers, then the S buffer is free for the key tile after next
         uint32_t sv[2][32];
         const uint32_t s_addr = tmem + (uint32_t)(tt * 128) + b * 64u + lane_addr;
@@ -518,6 +546,22 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap kv_map, const __grid_
             for (int i = 0; i < 32; ++i) {
               const float e2x = ex2(__uint_as_float(sv[c][i]) * cap_x2);
               sv[c][i] = __float_as_uint(cap_raw * (1.f - __fdividef(2.f, 1.f + e2x)));
+            }
+        }
+        if (slopes != nullptr) {
+          // the distance bias slope * (key - query), in raw units, two keys at a time
+          const float at = slope * (float)(key0 - t.pos0 - qi);
+          uint64_t bias2 = pack2(at, at + slope);
+          const uint64_t step2 = pack2(2.f * slope, 2.f * slope);
+#pragma unroll
+          for (int c = 0; c < 2; ++c)
+#pragma unroll
+            for (int i = 0; i < 32; i += 2) {
+              float b0, b1;
+              unpack2(add2(pack2(__uint_as_float(sv[c][i]), __uint_as_float(sv[c][i + 1])), bias2), b0, b1);
+              sv[c][i] = __float_as_uint(b0);
+              sv[c][i + 1] = __float_as_uint(b1);
+              bias2 = add2(bias2, step2);
             }
         }
         // P = 2^(scale * S - m) for the row, its sum returned; scaling and the row sum handle two values per
@@ -569,7 +613,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap kv_map, const __grid_
 #pragma unroll
               for (int i = 0; i < 32; ++i) {
                 const int key = key0 + 32 * c + i;
-                if (!(key <= lim && key >= lo && key < my_k_end)) sv[c][i] = 0xff800000u;      // -inf
+                if (!(key <= hi_j && key >= lo_j && key < end_j)) sv[c][i] = 0xff800000u;      // -inf
                 mx4[i & 3] = fmaxf(mx4[i & 3], __uint_as_float(sv[c][i]));
               }
           } else {
@@ -714,7 +758,9 @@ BSPEC_API int bspec_attention_prefill_tc_capped(const void* q, long long q_row_s
                                                 const int* positions, const int* kv_indptr, const int* kv_indices,
                                                 int n_entries, long long n_tokens, int max_q_len, int Hq, int Hkv,
                                                 int hd, int page_size, float scale, int window, int min_q_long,
-                                                int* work, const float* sink_l2, float softcap, cudaStream_t stream);
+                                                int* work, const float* sink_l2, float softcap, const float* slopes,
+                                                int pool, const void* pool_cache, const int* pool_indptr,
+                                                const int* pool_indices, long long pool_pages, cudaStream_t stream);
 BSPEC_API int bspec_attention_prefill_tc(const void* q, long long q_row_stride, void* out, int* status,
                                          long long n_pages, const void* cache, const int* qo_indptr,
                                          const int* positions, const int* kv_indptr, const int* kv_indices,
@@ -736,23 +782,35 @@ BSPEC_API int bspec_attention_prefill_tc_masked(const void* q, long long q_row_s
                                                 int* work, const float* sink_l2, cudaStream_t stream) {
   return bspec_attention_prefill_tc_capped(q, q_row_stride, out, status, n_pages, cache, qo_indptr, positions, kv_indptr,
                                            kv_indices, n_entries, n_tokens, max_q_len, Hq, Hkv, hd, page_size, scale,
-                                           window, min_q_long, work, sink_l2, 0.f, stream);
+                                           window, min_q_long, work, sink_l2, 0.f, nullptr, 0, nullptr, nullptr, nullptr, 0,
+                                           stream);
 }
 
-// The same with a soft cap c > 0 on the scaled scores (c tanh(s / c)); 0 is none.
+// The same with a soft cap c > 0 on the scaled scores (c tanh(s / c)), 0 is none; ``slopes`` (may be null): float32 per
+// query head, slope * (query - key) is taken off a token's scaled score; ``pool`` P > 0, with a window: before the window
+// a query also sees one entry per block of P tokens that lies wholly before it, from pages of the same layout.
 BSPEC_API int bspec_attention_prefill_tc_capped(const void* q, long long q_row_stride, void* out, int* status,
                                                 long long n_pages, const void* cache, const int* qo_indptr,
                                                 const int* positions, const int* kv_indptr, const int* kv_indices,
                                                 int n_entries, long long n_tokens, int max_q_len, int Hq, int Hkv,
                                                 int hd, int page_size, float scale, int window, int min_q_long,
-                                                int* work, const float* sink_l2, float softcap, cudaStream_t stream) {
+                                                int* work, const float* sink_l2, float softcap, const float* slopes,
+                                                int pool, const void* pool_cache, const int* pool_indptr,
+                                                const int* pool_indices, long long pool_pages, cudaStream_t stream) {
   if (n_entries <= 0 || max_q_len <= 0) return 0;
   if (softcap < 0.f || !(scale > 0.f)) return (int)cudaErrorInvalidValue;
   if (hd != HD || Hq % Hkv != 0 || page_size % 8 != 0 || KT % page_size != 0 || status == nullptr || n_pages <= 0 ||
       n_tokens <= 0 || work == nullptr)
     return (int)cudaErrorInvalidValue;
-  CUtensorMap kv_map, q_map;
+  if (pool < 0 || (pool > 0 && (window <= 0 || slopes != nullptr || pool_cache == nullptr || pool_indptr == nullptr ||
+                                pool_pages <= 0)))
+    return (int)cudaErrorInvalidValue;
+  CUtensorMap kv_map, q_map, pool_map;
   if (!make_map_2d_bf16(&kv_map, cache, n_pages * 2 * Hkv * page_size, HD, page_size, 64)) return (int)cudaErrorInvalidValue;
+  pool_map = kv_map;                                             // not read without pooled blocks
+  if (pool > 0 && !make_map_2d_bf16(&pool_map, pool_cache, pool_pages * 2 * Hkv * page_size, HD, page_size, 64))
+    return (int)cudaErrorInvalidValue;
+  const Pooled pooled = {pool, pool_indptr, pool_indices};
   const int G = Hq / Hkv;
   // Q through TMA when a tile's 128 rows are whole tokens (G divides 128) and the rows are 16-byte aligned;
   // otherwise the softmax threads copy their rows
@@ -762,20 +820,24 @@ BSPEC_API int bspec_attention_prefill_tc_capped(const void* q, long long q_row_s
   static bool attr_set_dev[bspec::kMaxDevices] = {};            // per device
   bool& attr_set = attr_set_dev[bspec::current_device()];
   if (!attr_set) {
-    const cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                               (int)smem_bytes());
-    if (e != cudaSuccess) return (int)e;
+    for (const void* kernel : {(const void*)attn_prefill_tc_kernel<false>, (const void*)attn_prefill_tc_kernel<true>}) {
+      const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_bytes());
+      if (e != cudaSuccess) return (int)e;
+    }
     attr_set = true;
   }
   const long long blocks = ((long long)max_q_len * G + QT * ROWS - 1) / (QT * ROWS);
   const long long n_items = blocks * Hkv * n_entries;
   if (n_items > (1ll << 30)) return (int)cudaErrorInvalidValue;
   const int grid = (int)(n_items < bspec::sm_count() ? n_items : bspec::sm_count());
-  BSPEC_LAUNCH((attn_prefill_tc_kernel), dim3(grid), THREADS, smem_bytes(), stream, kv_map, q_map,
-               (const __nv_bfloat16*)q, q_row_stride, (__nv_bfloat16*)out, status, qo_indptr, positions, kv_indptr,
-               kv_indices, Hq, Hkv, n_entries, (int)n_items, page_size, scale * 1.4426950408889634f, window, min_q_long,
-               q_by_tma, work, sink_l2, softcap > 0.f ? softcap / scale : 0.f,
-               softcap > 0.f ? 2.f * scale * 1.4426950408889634f / softcap : 0.f);
+#define GO(MORE)                                                                                                   \
+  BSPEC_LAUNCH((attn_prefill_tc_kernel<MORE>), dim3(grid), THREADS, smem_bytes(), stream, kv_map, q_map, \
+               (const __nv_bfloat16*)q, q_row_stride, (__nv_bfloat16*)out, status, qo_indptr, positions, kv_indptr, \
+               kv_indices, Hq, Hkv, n_entries, (int)n_items, page_size, scale * 1.4426950408889634f, window, min_q_long, \
+               q_by_tma, work, sink_l2, softcap > 0.f ? softcap / scale : 0.f, \
+               softcap > 0.f ? 2.f * scale * 1.4426950408889634f / softcap : 0.f, slopes, 1.f / scale, pool_map, pooled)
+  if (slopes != nullptr || pool > 0) GO(true); else GO(false);
+#undef GO
   return BSPEC_LAUNCH_CHECK();
 }
 

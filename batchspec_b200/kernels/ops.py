@@ -132,13 +132,15 @@ _SIGNATURES = {
     "bspec_attention_bf16_masked": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong,
                                     c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                                     c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p,
-                                    c_longlong, c_void_p, c_float, c_void_p],
+                                    c_longlong, c_void_p, c_float, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_longlong,
+                                    c_void_p],
     "bspec_attention_prefill_tc_masked": [c_void_p, c_longlong, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p,
                                           c_void_p, c_void_p, c_void_p, c_int, c_longlong, c_int, c_int, c_int, c_int,
                                           c_int, c_float, c_int, c_int, c_void_p, c_void_p, c_void_p],
     "bspec_attention_prefill_tc_capped": [c_void_p, c_longlong, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p,
                                           c_void_p, c_void_p, c_void_p, c_int, c_longlong, c_int, c_int, c_int, c_int,
-                                          c_int, c_float, c_int, c_int, c_void_p, c_void_p, c_float, c_void_p],
+                                          c_int, c_float, c_int, c_int, c_void_p, c_void_p, c_float, c_void_p, c_int, c_void_p,
+                                          c_void_p, c_void_p, c_longlong, c_void_p],
     "bspec_gemm_tc_plan": [c_int, c_int, c_int, c_int, c_void_p],
     "bspec_gemm_tc": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p],
     "bspec_gemm_tc_act": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p],
@@ -783,30 +785,38 @@ def gate_mul(x: torch.Tensor, gate: Optional[torch.Tensor], out: torch.Tensor, f
 def paged_attention(qkv: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, ctx, tables, n_heads: int,
                     n_kv_heads: int, head_dim: int, scale: float, window: int = 0, chunk: int = 0,
                     sink: Optional[torch.Tensor] = None, sink_l2: Optional[torch.Tensor] = None,
-                    softcap: float = 0.0, slopes: Optional[torch.Tensor] = None, pooled=None) -> None:
+                    softcap: float = 0.0, slopes: Optional[torch.Tensor] = None,
+                    slopes_l2: Optional[torch.Tensor] = None, pooled=None) -> None:
     """Causal attention of the step's tokens over their requests' cached keys.
     ``qkv``: [n, >= n_heads*head_dim] rows with the (already rotated) query heads
     first.  ``ctx`` gives qo_indptr / positions / n_entries / max_q_len, ``tables``
     the block tables of the cache group.  bfloat16 with head_dim 64/128/256 runs
     on the tensor-core kernels; everything else on the generic float32-math kernel.
     ``window`` > 0 keeps the last ``window`` keys, ``chunk`` > 0 the keys of the query's own chunk of ``chunk``
-    positions (one of the two at most).  ``sink`` (float32 per query head, with ``sink_l2`` its ``sink_table``) adds
+    positions (one of the two at most).  ``slopes`` (float32 per query head, with ``slopes_l2`` its ``sink_table``):
+    slope * (query - key) is taken off a score.  ``pooled`` = (P, pages, tables), with a window: before the window the
+    mean key and value of every block of P tokens is seen too.  ``sink`` (float32 per query head, with ``sink_l2`` its ``sink_table``) adds
     exp(sink) to the softmax denominator.  ``softcap`` c > 0 turns a scaled score s into c tanh(s / c)."""
     _require_cuda(qkv, out, cache, sink, sink_l2)
     assert qkv.stride(1) == 1 and out.is_contiguous() and out.dtype == qkv.dtype == cache.dtype
     assert not (window and chunk) and window >= 0 and chunk >= 0
     assert sink is None or (sink.dtype == torch.float32 and sink.numel() == n_heads and sink_l2 is not None
                             and sink_l2.dtype == torch.float32 and sink_l2.numel() == n_heads)
+    assert slopes is None or (slopes.dtype == torch.float32 and slopes.numel() == n_heads and slopes_l2 is not None
+                              and slopes_l2.dtype == torch.float32 and slopes_l2.numel() == n_heads and pooled is None)
     mask = int(window) if window else -int(chunk)      # the kernels take a chunk mask as a negative window
     lib = load_library()
-    if (qkv.dtype == torch.bfloat16 and head_dim in (64, 128, 256) and not FORCE_GENERIC_ATTENTION
-            and slopes is None and pooled is None):
+    plan = None
+    if qkv.dtype == torch.bfloat16 and head_dim in (64, 128, 256) and not FORCE_GENERIC_ATTENTION:
         # Everything that depends on the step and the layer's sizes only is worked out once per step (all layers of
         # a model ask the same question), the scratch included: the layers run one after the other on one stream.
         key = ("attention", n_heads, n_kv_heads, head_dim, id(tables), BALANCED_ATTENTION, USE_TMA_ATTENTION)
         plan = ctx.extras.get(key)
         if plan is None:
             plan = ctx.extras[key] = _attention_plan(qkv.device, ctx, tables, n_heads, n_kv_heads, head_dim)
+        if pooled is not None and not (plan[0] and plan[1] and head_dim <= 128):
+            plan = None                  # pooled blocks run on the kernels that load K/V through TMA
+    if plan is not None:
         (tma, balanced, n_splits, short, run_decode, run_prefill, prefill_tc, o_part, ml_part, counters, status, qo, pos,
          tok_entry, kv_indptr, kv_indices, kv_len) = plan
         if prefill_tc:
@@ -816,7 +826,7 @@ def paged_attention(qkv: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, c
                 kv_indptr, kv_indices, ctx.n_entries, qkv.shape[0], ctx.max_q_len, n_heads, n_kv_heads, head_dim,
                 tables.page_size,
                 float(scale), mask, short + 1, _work_counter(qkv.device).data_ptr(), _ptr(sink_l2), float(softcap),
-                _stream()),
+                _ptr(slopes), *_pool_args(pooled, cache, tables.page_size), _stream()),
                 "attention_prefill_tc")
             run_prefill = 0
             if not run_decode:
@@ -826,7 +836,7 @@ def paged_attention(qkv: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, c
             cache.shape[0] if tma else 0, cache.data_ptr(), qo, pos, tok_entry, kv_indptr, kv_indices, ctx.n_entries,
             ctx.n_tokens, ctx.max_q_len, n_heads, n_kv_heads, head_dim, tables.page_size, float(scale), mask,
             n_splits, short, run_decode, run_prefill, balanced, kv_len, cache.shape[0], _ptr(sink_l2), float(softcap),
-            _stream()),
+            _ptr(slopes_l2), *_pool_args(pooled, cache, tables.page_size), _stream()),
             "attention_bf16")
         global _launches
         _launches += 1 if run_decode and run_prefill else 0

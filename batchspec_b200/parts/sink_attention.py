@@ -86,6 +86,7 @@ class SinkAttention(Mixer):
             raise ValueError(f"{n_heads} heads need {n_heads} slopes, got {len(bias_slopes)}")
         self.slopes = None if bias_slopes is None else torch.tensor([float(x) for x in bias_slopes], dtype=torch.float32,
                                                                     device=runtime.device)
+        self.slopes_l2 = None if self.slopes is None else ops.sink_table(self.slopes)
         self.position = build_part(POSITION_ENCODINGS, position, runtime)
         self.wqkv = self.wo = self.b = self.sinks = self.sinks_l2 = self.q_norm = self.k_norm = None
         # values that are the keys, at sizes the tensor-core kernels take: those kernels read keys and values from
@@ -189,7 +190,7 @@ class SinkAttention(Mixer):
                 direct = not self.gate and out_scale == 1.0 and out.is_contiguous()
                 heads = out if direct else torch.empty((n, H * vd), dtype=x.dtype, device=x.device)
                 ops.paged_attention(q, heads, cache.kv, ctx, tables, H, G, hd, self.scale, self.window, self.chunk,
-                                    self.sinks, self.sinks_l2, self.softcap, self.slopes, pooled)
+                                    self.sinks, self.sinks_l2, self.softcap, self.slopes, self.slopes_l2, pooled)
                 if not direct and self.gate_per_head and out_scale == 1.0 and out.is_contiguous():
                     # one logit per head: the heads [n, H * vd] read as [H, n, vd]
                     ops.gate_heads(heads.view(n, H, vd).transpose(0, 1), gate, out)

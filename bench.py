@@ -786,7 +786,168 @@ def finolix_kernels_alone(z, pk, iters=20):
     return out
 
 
+PODIZEN_SIZES = {
+    # the Finolix sizes (width, heads, experts) with the Tokolorn window; blocks of 16 tokens before it, a retention with
+    # as many heads as the attention, a shared expert of twice an expert's inner size
+    "w2048": dict(VABANEX_SIZES["w2048"], window=1024, streams=4, pool=16, dim_a=128, chunk=1024, inner=4096, state=16,
+                  dt_rank=128),
+    "w4096": dict(VABANEX_SIZES["w4096"], window=1024, streams=4, pool=16, dim_a=128, chunk=1024, inner=8192, state=16,
+                  dt_rank=256),
+}
+
+
+def podizen_config_json(z, layers, vocab=32000):
+    """Attention with a distance bias and, side by side, pooled attention and retention in turn, each with routed experts."""
+    H, G, hd = z["heads"], z["kv_heads"], z["dim_a"]
+    mlp = dict(kind="moe", expert=dict(ff=z["expert_ff"]), shared=dict(ff=2 * z["expert_ff"]),
+               router=dict(experts=z["experts"], top=z["top"], groups=dict(count=z["groups"], keep=z["keep"])))
+    att = dict(type="attention", mlp=mlp, mixer=dict(heads=H, kv_heads=G, dim=hd, vdim=hd, scale=hd ** -0.5,
+                                                     mask=dict(size=z["window"])))
+    par = dict(type="parallel", mlp=mlp, mixer=dict(
+        left=dict(heads=H, kv_heads=G, dim=hd, vdim=hd, scale=hd ** -0.5, mask=dict(size=z["window"], pool=z["pool"]),
+                  rot=dict(base=500000.0, dims=hd)),
+        right=dict(heads=H, dim=hd, vdim=hd, decay=[1.0 - 2.0 ** (-(5.0 + 6.0 * i / (H - 1))) for i in range(H)],
+                   rot=dict(base=10000.0, dims=hd))))
+    return dict(architecture="Podizen", vocab=vocab, width=z["width"], norm=dict(eps=1e-5),
+                layers=[(att, par)[i % 2] for i in range(layers)])
+
+
+def podizen_kernels_alone(z, pk, iters=20):
+    """The design's own kernels by themselves, each beside its like at equal sizes: attention with a distance bias, and
+    with pooled blocks before the window, against the same kernels with the window alone (a prompt of 4,096 tokens: FLOP/s
+    over the visible pairs against the measured product peak; a decode step of 64 requests x 4,096 tokens: bytes of the
+    visible keys, values and blocks against the measured copy rate); the blocks' means; the q/k/v preparation with weighted
+    norms, with and without the blocks' means; the branch join (norm, sum, history, average over depth, norm) against add +
+    RMS norm; the retention's recurrence and rotation against the lightning recurrence; the norm and gate per head; routed
+    experts with softmax groups and a shared expert against those without."""
+    import torch
+    from itertools import accumulate
+    from types import SimpleNamespace
+    from batchspec_b200.kernels import ops
+    from batchspec_b200.parts.base import FEED_FORWARDS, PartSpec, Runtime, build_part
+    ops.require("state_mixers", "joins", "moe")
+    dev = "cuda:0"
+    Hq, G, hd, ps, W, P, d = z["heads"], z["kv_heads"], z["dim_a"], 16, z["window"], z["pool"], z["width"]
+    out = {}
+    slopes = torch.tensor([2.0 ** (-8.0 * (h + 1) / Hq) for h in range(Hq)], device=dev)
+    slopes_l2 = ops.sink_table(slopes)
+    by = lambda ms, nbytes: dict(ms=round(ms, 4), gbs=round(nbytes / ms / 1e6, 1), frac_of_measured=round(nbytes / ms / 1e6 / pk["hbm_gbs"], 4))
+    i32 = lambda x: torch.as_tensor(x, dtype=torch.int32, device=dev)
+
+    def step_ctx(q_lens, ctx_len):
+        n, B = sum(q_lens), len(q_lens)
+        per, pper = -(-ctx_len // ps), -(-(ctx_len // P) // ps)
+        ctx = SimpleNamespace(qo_indptr=i32([0] + list(accumulate(q_lens))), n_entries=B, n_tokens=n, max_q_len=max(q_lens),
+                              positions=i32(torch.cat([torch.arange(ctx_len - q, ctx_len) for q in q_lens])),
+                              tok_entry=i32(torch.cat([torch.full((q,), i) for i, q in enumerate(q_lens)])),
+                              max_kv_len=ctx_len, kv_len=i32([ctx_len] * B), state_slots=i32(list(range(B))),
+                              extras={"min_q_len": min(q_lens)})
+        table = lambda k: SimpleNamespace(kv_indptr=torch.arange(B + 1, dtype=torch.int32, device=dev) * k,
+                                          kv_indices=torch.randperm(B * k, device=dev).to(torch.int32), page_size=ps)
+        return ctx, table(per), table(pper), n, B, per, pper
+
+    for name, q_lens, ctx_len in (("prompt_4096", [4096], 4096), ("decode_64x4096", [1] * 64, 4096)):
+        ctx, tables, ptables, n, B, per, pper = step_ctx(q_lens, ctx_len)
+        cache = torch.randn(B * per, 2, ps * G * hd, device=dev).bfloat16()
+        pooled = (P, torch.randn(B * pper, 2, ps * G * hd, device=dev).bfloat16(), ptables)
+        q = torch.randn(n, Hq * hd, device=dev).bfloat16()
+        o = torch.empty(n, Hq * hd, device=dev, dtype=torch.bfloat16)
+        for label, kw in (("bias", dict(slopes=slopes, slopes_l2=slopes_l2)), ("pooled", dict(pooled=pooled)), ("window", {})):
+            ctx.extras = {"min_q_len": min(q_lens)}
+            ms = _time(lambda: ops.paged_attention(q, o, cache, ctx, tables, Hq, G, hd, hd ** -0.5, W, **kw), iters)
+            seen = lambda p: min(p + 1, W) + (max(0, p - W + 1) // P if label == "pooled" else 0)
+            pairs = sum(seen(p) for p in range(ctx_len - q_lens[0], ctx_len)) * len(q_lens)
+            if name.startswith("prompt"):
+                flops = 4.0 * Hq * hd * pairs
+                out[f"attention_{name}_{label}"] = dict(ms=round(ms, 4), tflops=round(flops / ms / 1e9, 1),
+                                                        frac_of_measured=round(flops / ms / 1e9 / pk["bf16_tflops"], 4))
+            else:
+                out[f"attention_{name}_{label}"] = by(ms, pairs * 2 * G * hd * 2)
+        if name.startswith("prompt"):
+            ms = _time(lambda: ops.pool_append(cache, ctx, tables, pooled, G, hd, hd), iters)
+            out["pool_append_4096"] = by(ms, n * 2 * G * hd * 2 * (1 + 1 / P))
+        width = (Hq + 2 * G) * hd
+        qkv32 = torch.randn(n, width, device=dev)
+        nw = torch.ones(hd, device=dev, dtype=torch.bfloat16)
+        freq = ops.rope_frequency_table(torch.pow(torch.tensor(500000.0, dtype=torch.float64), -torch.arange(0, hd // 2, dtype=torch.float64) * 2 / hd), dev)
+        for label, kw in (("pooled", dict(pooled=pooled)), ("plain", {})):
+            if label == "pooled" and name.startswith("prompt"):
+                continue
+            ms = _time(lambda: ops.qkv_prepare(qkv32, Hq, G, hd, hd, None, freq, hd, False, 1.0, 1e-5, ctx.positions, ctx.tok_entry,
+                                               tables.kv_indptr, tables.kv_indices, cache, ps, q_norm=nw, k_norm=nw, norm_first=True,
+                                               **kw), iters)
+            out[f"qkv_prepare_{name}_{label}"] = by(ms, n * width * (4 + 2))
+        del cache, pooled, q, o, qkv32
+    # branches on their way into the residual: a mid-layer join, a pair, and a layer's end after three earlier layers
+    for n in (4096, 64):
+        x, y, y2 = torch.randn(n, d, device=dev), torch.randn(n, d, device=dev).bfloat16(), torch.randn(n, d, device=dev).bfloat16()
+        w = torch.ones(d, device=dev)
+        hist, coef = torch.randn(5, n, d, device=dev), torch.tensor([0.1, 0.1, 0.1, 0.7], device=dev)
+        o = torch.empty(n, d, device=dev, dtype=torch.bfloat16)
+        join = dict(dst=x, out=o, post=w, branch_eps=1e-5, norm_w=w, eps=1e-5)
+        ms = _time(lambda: ops.branch_join(x, y, **join), iters)
+        out[f"branch_join_{n}"] = by(ms, n * d * (8 + 2 + 2))
+        ms = _time(lambda: ops.branch_join(x, ops.NormedPair(y, y2, w, w, 1e-5), **join), iters)
+        out[f"branch_join_pair_{n}"] = by(ms, n * d * (8 + 4 + 2))
+        ms = _time(lambda: ops.branch_join(x, y, hist=hist, slot=3, store=True, coef=coef, **join), iters)
+        out[f"branch_join_depth_{n}"] = by(ms, n * d * (8 + 2 + 2 + 4 * 3 + 4))
+        ms = _time(lambda: ops.add_rmsnorm(x, y, w, 1e-5, o, 1.0, True), iters)
+        out[f"add_rmsnorm_{n}"] = by(ms, n * d * (8 + 2 + 2))
+    # retention beside lightning attention: the same recurrence, rotated q and k instead of silu; the norm per head
+    H, dk, dv = Hq, hd, hd
+    decay = torch.linspace(0.97, 0.9995, H, device=dev)
+    norm_w = torch.ones(H * dv, device=dev)
+    freq = ops.rope_frequency_table(torch.pow(torch.tensor(10000.0, dtype=torch.float64), -torch.arange(0, dk // 2, dtype=torch.float64) * 2 / dk), dev)
+    for name, q_lens in (("prompt_2048", [2048]), ("prompt_8x2048", [2048] * 8), ("decode_64", [1] * 64)):
+        ctx, _, _, n, B, _, _ = step_ctx(q_lens, max(q_lens[0], P))
+        ld = 2 * H * dk + 2 * H * dv
+        proj = torch.randn(n, ld, device=dev)
+        state = torch.zeros(B, H * dv * dk, device=dev)
+        run = lambda **kw: ops.lightning_recurrence(proj, 0, H * dk, 2 * H * dk, decay, state, ctx, H, dk, dv, **kw)
+        inside = dict(inv_freq=freq, rotary_dim=dk) if name.startswith("decode") else {}
+        ms = _time(lambda: run(activation=None, k_scale=dk ** -0.5, **inside), iters)
+        ms_l = _time(run, iters)
+        rec = dict(retention_ms=round(ms, 4), lightning_ms=round(ms_l, 4))
+        if name.startswith("decode"):
+            nbytes = B * H * dk * dv * 4 * 2
+            rec.update(retention_frac_of_measured=round(nbytes / ms / 1e6 / pk["hbm_gbs"], 4),
+                       lightning_frac_of_measured=round(nbytes / ms_l / 1e6 / pk["hbm_gbs"], 4))
+        else:
+            rec["retention_fp32_tflops"] = round(5.0 * n * H * dk * dv / ms / 1e9, 2)
+            rec["lightning_fp32_tflops"] = round(5.0 * n * H * dk * dv / ms_l / 1e9, 2)
+            ms = _time(lambda: ops.rope_inplace(proj[:, :2 * H * dk].unflatten(1, (2 * H, dk)), ctx.positions, freq, dk), iters)
+            rec["rope"] = by(ms, n * 2 * H * dk * 8)
+        o32, gate = run(), proj[:, 2 * H * dk + H * dv:]
+        ms = _time(lambda: ops.gated_rmsnorm(o32, gate, None, 1e-5, H, dv, torch.bfloat16), iters)
+        rec["norm_per_head"] = by(ms, n * H * dv * (4 + 4 + 2))
+        ms = _time(lambda: ops.gated_rmsnorm(o32, gate, norm_w, 1e-5, 1, H * dv, torch.bfloat16, "sigmoid"), iters)
+        rec["norm_over_all_heads"] = by(ms, n * H * dv * (4 + 4 + 2))
+        out[f"retention_{name}"] = rec
+        del proj, state
+    # routed experts: softmax over all, groups, renormalised, with a shared expert, against the softmax over the chosen
+    rt = Runtime(torch.bfloat16, torch.device(dev))
+    E, top, ff = z["experts"], z["top"], z["expert_ff"]
+    for label, kw, shared in (("routed_shared", dict(bias=False, scores="softmax", n_groups=z["groups"], keep_groups=z["keep"],
+                                                     shared=2 * ff), 2 * ff),
+                              ("routed_softmax", dict(bias=False, scores="softmax", n_groups=z["groups"], keep_groups=z["keep"]), 0),
+                              ("routed_glu", {}, 0)):
+        part = build_part(FEED_FORWARDS, PartSpec("routed_glu", dict(dim=d, intermediate=ff, n_experts=E, top=top, **kw)), rt)
+        part.bind({k: (torch.randn(ps_.shape, device=dev) * 0.02).bfloat16() for k, ps_ in part.param_specs().items()})
+        for n in (4096, 64):
+            x = torch.randn(n, d, device=dev).bfloat16()
+            ms = _time(lambda: part.forward(x, None), iters)
+            flops = 2.0 * n * 3 * d * (top * ff + shared)
+            rec = dict(ms=round(ms, 4), tflops=round(flops / ms / 1e9, 1), frac_of_measured=round(flops / ms / 1e9 / pk["bf16_tflops"], 4))
+            if n == 64:                     # decode: the weights of the experts that were chosen are read once
+                nbytes = (min(E, n * top) * ff + shared) * 3 * d * 2
+                rec["weights_frac_of_measured"] = round(nbytes / ms / 1e6 / pk["hbm_gbs"], 4)
+            out[f"{label}_{n}"] = rec
+        del part
+    return out
+
+
 DESIGNS = {
+    "podizen": (PODIZEN_SIZES, podizen_config_json, podizen_kernels_alone, "kernels_alone"),
     "finolix": (FINOLIX_SIZES, finolix_config_json, finolix_kernels_alone, "kernels_alone"),
     "tokolorn": (TOKOLORN_SIZES, tokolorn_config_json, tokolorn_kernels_alone, "kernels_alone"),
     "vabanex": (VABANEX_SIZES, vabanex_config_json, latent_attention_alone, "latent_attention_alone"),
@@ -813,6 +974,8 @@ def run_design(a) -> int:
             models.append(("lupusun", lupusun_config_json(z, layers)))
         if a.design == "finolix":         # its closest model, the other one with latent attention and routed experts
             models.append(("vabanex", vabanex_config_json(z, layers)))
+        if a.design == "podizen":         # its closest models: the same kinds of mixers, and routed gated experts
+            models += [("tokolorn", tokolorn_config_json(dict(z, dim=z["dim_a"]), layers)), ("finolix", finolix_config_json(z, layers))]
         for label, cj in models:
             cfg = config_from_json_dict(cj)
             eng = Engine(dtype="bfloat16", device="cuda:0")
@@ -894,7 +1057,7 @@ def main() -> int:
     ap.add_argument("--skip-points", action="store_true", help="only the headline batch (no prefill, b1, b64, e2e)")
     ap.add_argument("--skip-workloads", action="store_true",
                     help="leave out e2e at batch 64 and the 3B / long-context workloads (about a minute)")
-    ap.add_argument("--design", default=None, choices=["vabanex", "lupusun", "tokolorn", "finolix"],
+    ap.add_argument("--design", default=None, choices=["vabanex", "lupusun", "tokolorn", "finolix", "podizen"],
                     help="instead of the headline workload: this design at real layer sizes beside the Llama model of equal size")
     a = ap.parse_args()
     if a.impl == "reference":
