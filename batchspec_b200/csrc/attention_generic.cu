@@ -221,13 +221,43 @@ __device__ __forceinline__ float pooled_mean(const T* __restrict__ cache, const 
                                              size_t part, int width, int p0, int pool, int page_size,
                                              long long n_pages) {
   float s = 0.f;
-#pragma unroll 4
+#pragma unroll 8
   for (int r = 0; r < pool; ++r) {
     const int p = p0 + r, page = table[p / page_size];
     if (bspec::in_range(page, n_pages, 116))
       s += to_f32(cache[(size_t)page * page_elems + part + (size_t)(p % page_size) * width]);
   }
   return s / (float)pool;
+}
+
+__device__ __forceinline__ void row4(const float* p, float (&f)[4]) {
+  const float4 v = *reinterpret_cast<const float4*>(p);
+  f[0] = v.x, f[1] = v.y, f[2] = v.z, f[3] = v.w;
+}
+__device__ __forceinline__ void row4(const __nv_bfloat16* p, float (&f)[4]) {
+  const uint2 v = *reinterpret_cast<const uint2*>(p);
+  const __nv_bfloat162 a = *reinterpret_cast<const __nv_bfloat162*>(&v.x), b = *reinterpret_cast<const __nv_bfloat162*>(&v.y);
+  f[0] = __low2float(a), f[1] = __high2float(a), f[2] = __low2float(b), f[3] = __high2float(b);
+}
+
+// The same for four columns at once (head sizes that are multiples of 4); each column's arithmetic is the same.
+template <typename T>
+__device__ __forceinline__ void pooled_mean4(float (&m)[4], const T* __restrict__ cache, const int* __restrict__ table,
+                                             size_t page_elems, size_t part, int width, int p0, int pool, int page_size,
+                                             long long n_pages) {
+  m[0] = m[1] = m[2] = m[3] = 0.f;
+#pragma unroll 8
+  for (int r = 0; r < pool; ++r) {
+    const int p = p0 + r, page = table[p / page_size];
+    if (bspec::in_range(page, n_pages, 116)) {
+      float v[4];
+      row4(cache + (size_t)page * page_elems + part + (size_t)(p % page_size) * width, v);
+#pragma unroll
+      for (int c = 0; c < 4; ++c) m[c] += v[c];
+    }
+  }
+#pragma unroll
+  for (int c = 0; c < 4; ++c) m[c] = m[c] / (float)pool;
 }
 
 __device__ __forceinline__ void prep_sincos(int pos, const float* __restrict__ inv_freq, int half, int j, float* s,
@@ -372,6 +402,14 @@ qkv_prepare_kernel(const float* __restrict__ qkv, long long ld, int Hq, int Hkv,
     if (bspec::in_range(b / page_size, pool_indptr[e + 1] - pool_indptr[e], 117) &&
         bspec::in_range(ptab[b / page_size], pool_pages, 118)) {
       T* to = pool_cache + (size_t)ptab[b / page_size] * page_elems + head + (size_t)(b % page_size) * width;
+      if (vec) {
+        for (int d = 4 * lane; d < width; d += 128) {
+          float m[4];
+          pooled_mean4<T>(m, cache, kv_indices + kv_indptr[e], page_elems, head + d, width, b * pool, pool, page_size, n_pages);
+          prep_store4(to + d, m[0], m[1], m[2], m[3]);
+        }
+        return;
+      }
       for (int d = lane; d < width; d += 32)
         to[d] = from_f32<T>(pooled_mean<T>(cache, kv_indices + kv_indptr[e], page_elems, head + d, width, b * pool, pool,
                                            page_size, n_pages));
@@ -380,8 +418,8 @@ qkv_prepare_kernel(const float* __restrict__ qkv, long long ld, int Hq, int Hkv,
 }
 
 // The pooled entries of the blocks that a step's portions complete: block (x, e, z) takes the x-th such block of
-// entry e; a thread per column of [k of every kv head | v of every kv head].
-template <typename T>
+// entry e; a thread per column (VEC: per four columns) of [k of every kv head | v of every kv head].
+template <typename T, bool VEC>
 __global__ void __launch_bounds__(256)
 pool_append_kernel(const T* __restrict__ cache, const int* __restrict__ qo_indptr, const int* __restrict__ positions,
                    const int* __restrict__ kv_indptr, const int* __restrict__ kv_indices, T* __restrict__ pool_cache,
@@ -394,7 +432,7 @@ pool_append_kernel(const T* __restrict__ cache, const int* __restrict__ qo_indpt
   const int pos0 = positions[t0];
   const int b = pos0 / pool + (int)blockIdx.x;
   if ((long long)(b + 1) * pool > pos0 + nt) return;
-  const int col = blockIdx.z * blockDim.x + threadIdx.x;
+  const int col = (VEC ? 4 : 1) * (blockIdx.z * blockDim.x + threadIdx.x);
   if (col >= Hkv * (hd + vd)) return;
   const bool is_v = col >= Hkv * hd;
   const int width = is_v ? vd : hd, c = is_v ? col - Hkv * hd : col;
@@ -405,9 +443,15 @@ pool_append_kernel(const T* __restrict__ cache, const int* __restrict__ qo_indpt
   if (!bspec::in_range(b / page_size, pool_indptr[e + 1] - pool_indptr[e], 117) ||
       !bspec::in_range(ptab[b / page_size], pool_pages, 118))
     return;
-  pool_cache[(size_t)ptab[b / page_size] * page_elems + head + (size_t)(b % page_size) * width + d] =
-      from_f32<T>(pooled_mean<T>(cache, kv_indices + kv_indptr[e], page_elems, head + d, width, b * pool, pool,
-                                 page_size, n_pages));
+  T* to = pool_cache + (size_t)ptab[b / page_size] * page_elems + head + (size_t)(b % page_size) * width + d;
+  if (VEC) {
+    float m[4];
+    pooled_mean4<T>(m, cache, kv_indices + kv_indptr[e], page_elems, head + d, width, b * pool, pool, page_size, n_pages);
+    prep_store4(to, m[0], m[1], m[2], m[3]);
+  } else {
+    *to = from_f32<T>(pooled_mean<T>(cache, kv_indices + kv_indptr[e], page_elems, head + d, width, b * pool, pool,
+                                     page_size, n_pages));
+  }
 }
 }  // namespace
 
@@ -418,15 +462,16 @@ BSPEC_API int bspec_pool_append(const void* cache, int dtype, const int* qo_indp
                                 int page_size, int pool, long long n_pages, long long pool_pages, cudaStream_t stream) {
   if (n_entries <= 0 || max_q_len <= 0) return 0;
   if (pool <= 0 || Hkv <= 0 || hd <= 0 || vd < 0 || page_size <= 0 || n_entries > 65535) return (int)cudaErrorInvalidValue;
-  const dim3 grid((max_q_len + pool - 1) / pool, n_entries, (Hkv * (hd + vd) + 255) / 256);
+  const bool vec = hd % 4 == 0 && vd % 4 == 0;
+  const int items = Hkv * (hd + vd) / (vec ? 4 : 1), threads = items >= 256 ? 256 : ((items + 31) / 32) * 32;
+  const dim3 grid((max_q_len + pool - 1) / pool, n_entries, (items + threads - 1) / threads);
   if (grid.z > 65535) return (int)cudaErrorInvalidConfiguration;
-  if (dtype == BSPEC_F32)
-    BSPEC_LAUNCH((pool_append_kernel<float>), grid, 256, 0, stream, (const float*)cache, qo_indptr, positions, kv_indptr,
-                 kv_indices, (float*)pool_cache, pool_indptr, pool_indices, Hkv, hd, vd, page_size, pool, n_pages, pool_pages);
-  else
-    BSPEC_LAUNCH((pool_append_kernel<__nv_bfloat16>), grid, 256, 0, stream, (const __nv_bfloat16*)cache, qo_indptr,
-                 positions, kv_indptr, kv_indices, (__nv_bfloat16*)pool_cache, pool_indptr, pool_indices, Hkv, hd, vd,
-                 page_size, pool, n_pages, pool_pages);
+#define LP(T, V)                                                                                                     \
+  BSPEC_LAUNCH((pool_append_kernel<T, V>), grid, threads, 0, stream, (const T*)cache, qo_indptr, positions, kv_indptr, \
+               kv_indices, (T*)pool_cache, pool_indptr, pool_indices, Hkv, hd, vd, page_size, pool, n_pages, pool_pages)
+  if (dtype == BSPEC_F32) { if (vec) LP(float, true); else LP(float, false); }
+  else { if (vec) LP(__nv_bfloat16, true); else LP(__nv_bfloat16, false); }
+#undef LP
   return BSPEC_LAUNCH_CHECK();
 }
 

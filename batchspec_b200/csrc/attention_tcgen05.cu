@@ -25,6 +25,8 @@
 // bounded; on expiry a code goes to `status`, all roles stop and the tensor memory is given back.
 // With pooled blocks before a window an item walks key tiles of two sources: first the request's block entries (their
 // own pages and table, the same layout), then its tokens; both are tiles of the same ring and the same softmax.
+// With a distance bias an item walks its key tiles from the last to the first: the bias grows towards the query, by tens
+// of units a tile for the steep heads, so in ascending order nearly every tile would move the maximum and rescale O.
 #include "common.cuh"
 #include "tma.cuh"
 #include <math.h>
@@ -171,7 +173,7 @@ struct Pooled {
 __device__ __forceinline__ bool load_item(Item& it, int idx, int Hq, int Hkv, int n_entries, int window,
                                           int page_size, int min_q_long, const int* __restrict__ qo_indptr,
                                           const int* __restrict__ positions, const int* __restrict__ kv_indptr,
-                                          const int* __restrict__ kv_indices, const Pooled& pooled) {
+                                          const int* __restrict__ kv_indices, const Pooled& pooled, bool backwards) {
   const int g = idx % Hkv, ez = idx / Hkv;
   const int e = ez % n_entries, z = ez / n_entries;
   Geom& t = it.t;
@@ -207,6 +209,11 @@ __device__ __forceinline__ bool load_item(Item& it, int idx, int Hq, int Hkv, in
     }
   }
   it.n_tiles = max(it.n_kt[0], it.n_kt[1]);
+  if (backwards) {             // both Q tiles start at the item's last key tile, whole-masked for the first one or not
+#pragma unroll
+    for (int tt = 0; tt < QT; ++tt)
+      if (it.n_kt[tt] > 0) it.n_kt[tt] = it.n_tiles;
+  }
   it.k_end = max(it.k_end_t[0], it.k_end_t[1]);
   it.table = kv_indices + kv_indptr[e];
   return true;
@@ -230,8 +237,10 @@ constexpr int ITEM_RING = 8;
 // follow; nothing but the tensor memory allocation is shared between items, so the next item's keys and queries
 // are fetched, and its first two S tiles computed, while the softmax threads still finish and store the item
 // before.  The CTA that leaves last puts the counter back to zero for the next launch.
-// MORE: a distance bias or pooled blocks may be given; without it the code for both is left out.
-template <bool MORE>
+// MORE: what the launch has besides the masks, the sink and the cap; the code for the rest is left out.
+constexpr int PLAIN = 0, BIASED = 1, POOLED = 2;
+
+template <int MORE>
 __global__ void __launch_bounds__(THREADS, 1)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap kv_map, const __grid_constant__ CUtensorMap q_map,
                        const __nv_bfloat16* __restrict__ q, long long q_row_stride, __nv_bfloat16* __restrict__ out,
@@ -241,8 +250,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap kv_map, const __grid_
                        int q_by_tma, int* __restrict__ work, const float* __restrict__ sink_l2, float cap_raw,
                        float cap_x2, const float* __restrict__ slopes_in, float inv_scale,
                        const __grid_constant__ CUtensorMap pool_map, const Pooled pooled_in) {
-  const float* __restrict__ slopes = MORE ? slopes_in : nullptr;
-  const Pooled pooled = MORE ? pooled_in : Pooled{0, nullptr, nullptr};
+  const float* __restrict__ slopes = MORE == BIASED ? slopes_in : nullptr;
+  const Pooled pooled = MORE == POOLED ? pooled_in : Pooled{0, nullptr, nullptr};
   // The step's lengths, positions and block tables were uploaded before its first kernel: the set-up below and the
   // look-up of the CTA's first item read nothing that the kernel before this one writes, so they run under its
   // tail; q, the new tokens' keys and `out` are touched only after the wait.
@@ -295,7 +304,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap kv_map, const __grid_
   bool first_found = false;
   if (warp == 0)
     first_found = load_item(it, blockIdx.x, Hq, Hkv, n_entries, window, page_size, min_q_long, qo_indptr, positions,
-                            kv_indptr, kv_indices, pooled);
+                            kv_indptr, kv_indices, pooled, MORE == BIASED);
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
@@ -336,7 +345,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap kv_map, const __grid_
       }
       while (cand < n_items && !found) {
         found = load_item(it, cand, Hq, Hkv, n_entries, window, page_size, min_q_long, qo_indptr, positions, kv_indptr,
-                          kv_indices, pooled);
+                          kv_indices, pooled, MORE == BIASED);
         if (!found) draw();
       }
       if (!found) it.n_tiles = -1;
@@ -366,8 +375,9 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap kv_map, const __grid_
       const int first_pg = it.lo_key / page_size, last_pg = max(first_pg, (it.k_end - 1) / page_size);
       const int last_ppg = (max(it.pool_end, 1) - 1) / page_size;
       auto page_of = [&](int j) -> int {
-        if (MORE && j < it.n_pool) return it.ptable[min((j * KT) / page_size + lane, last_ppg)];
-        int pg = (it.k_begin + (MORE ? j - it.n_pool : j) * KT) / page_size + lane;
+        if (MORE == BIASED) j = it.n_tiles - 1 - j;
+        if (MORE == POOLED && j < it.n_pool) return it.ptable[min((j * KT) / page_size + lane, last_ppg)];
+        int pg = (it.k_begin + (MORE == POOLED ? j - it.n_pool : j) * KT) / page_size + lane;
         pg = min(max(pg, first_pg), last_pg);
         return it.table[pg];
       };
@@ -387,7 +397,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap kv_map, const __grid_
           __nv_bfloat16* Ks = KV + (size_t)st * 2 * KTILE;
           const int row_k = ((page * 2) * Hkv + it.g) * page_size;
           const int row_v = row_k + Hkv * page_size;
-          const CUtensorMap* map = MORE && j < it.n_pool ? &pool_map : &kv_map;
+          const CUtensorMap* map = MORE == POOLED && j < it.n_pool ? &pool_map : &kv_map;
 #pragma unroll
           for (int c = 0; c < 2; ++c) {
             tma_load_2d(Ks + c * SUBK + lane * page_size * 64, map, kv_full + st, c * 64, row_k);
@@ -527,8 +537,9 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap kv_map, const __grid_
         ok = mbar_wait(s_full + 2 * tt + b, (n >> 1) & 1u, abort_flag, status, 36);
         if (!ok) break;
         tc_fence_after();
-        const bool blocks = MORE && j < it.n_pool;                // a tile of pooled blocks: the numbers are blocks'
-        const int key0 = blocks ? j * KT : it.k_begin + (MORE ? j - it.n_pool : j) * KT;
+        const bool blocks = MORE == POOLED && j < it.n_pool;      // a tile of pooled blocks: the numbers are blocks'
+        const int kt = MORE == BIASED ? it.n_tiles - 1 - j : (MORE == POOLED ? j - it.n_pool : j);
+        const int key0 = blocks ? j * KT : it.k_begin + kt * KT;
         const int hi_j = blocks ? last_block : lim, lo_j = blocks ? 0 : lo, end_j = blocks ? it.pool_end : my_k_end;
         const bool need_mask = key0 + KT - 1 > hi_j || key0 < lo_j || key0 + KT > end_j;
         // the whole S row into registers, then the S buffer is free for the key tile after next
@@ -548,22 +559,6 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap kv_map, const __grid_
               sv[c][i] = __float_as_uint(cap_raw * (1.f - __fdividef(2.f, 1.f + e2x)));
             }
         }
-        if (slopes != nullptr) {
-          // the distance bias slope * (key - query), in raw units, two keys at a time
-          const float at = slope * (float)(key0 - t.pos0 - qi);
-          uint64_t bias2 = pack2(at, at + slope);
-          const uint64_t step2 = pack2(2.f * slope, 2.f * slope);
-#pragma unroll
-          for (int c = 0; c < 2; ++c)
-#pragma unroll
-            for (int i = 0; i < 32; i += 2) {
-              float b0, b1;
-              unpack2(add2(pack2(__uint_as_float(sv[c][i]), __uint_as_float(sv[c][i + 1])), bias2), b0, b1);
-              sv[c][i] = __float_as_uint(b0);
-              sv[c][i + 1] = __float_as_uint(b1);
-              bias2 = add2(bias2, step2);
-            }
-        }
         // P = 2^(scale * S - m) for the row, its sum returned; scaling and the row sum handle two values per
         // instruction (fma/add.f32x2), the exponentials all go to the special-function unit (masked scores are -inf
         // and come out as exactly 0).  Each half of P goes back into tensor memory as soon as it is complete, over
@@ -571,9 +566,12 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap kv_map, const __grid_
         // second half's arithmetic: the P V product takes its A operand from there.  What the columns held before
         // (P of the key tile two before this one) was read by a product that was issued, and so completed, before
         // this S.  The stores are warp-wide: every path to this point is taken by the whole warp.
-        auto exponentials = [&](float neg_m) -> float {
+        // ``bias`` at the tile's first key and ``step`` from key to key (base-2 units): a distance bias that is not in the
+        // scores yet.
+        auto exponentials = [&](float neg_m, float bias, float step) -> float {
           uint32_t packed[32];
-          const uint64_t scale2 = pack2(scale_log2, scale_log2), neg_m2 = pack2(neg_m, neg_m);
+          const uint64_t scale2 = pack2(scale_log2, scale_log2), step2 = pack2(2.f * step, 2.f * step);
+          uint64_t neg_m2 = MORE == BIASED ? pack2(neg_m + bias, neg_m + bias + step) : pack2(neg_m, neg_m);
           uint64_t l2[2] = {pack2(0.f, 0.f), pack2(0.f, 0.f)};
 #pragma unroll
           for (int c = 0; c < 2; ++c) {
@@ -581,6 +579,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap kv_map, const __grid_
             for (int i = 0; i < 32; i += 2) {
               float p0, p1;
               unpack2(fma2(pack2(__uint_as_float(sv[c][i]), __uint_as_float(sv[c][i + 1])), scale2, neg_m2), p0, p1);
+              if (MORE == BIASED) neg_m2 = add2(neg_m2, step2);
               p0 = ex2(p0);
               p1 = ex2(p1);
               l2[(i >> 1) & 1] = add2(l2[(i >> 1) & 1], pack2(p0, p1));
@@ -600,11 +599,27 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap kv_map, const __grid_
         float corr = 1.f, row_sum = 0.f;
         bool full_path = __any_sync(0xffffffffu, need_mask || m_ref == -INFINITY);
         if (!full_path) {
-          row_sum = exponentials(-m_ref);
+          row_sum = exponentials(-m_ref, slope * scale_log2 * (float)(key0 - t.pos0 - qi), slope * scale_log2);
           full_path = __any_sync(0xffffffffu, !(row_sum <= 16384.f));
           if (full_path) tc_wait_st();          // the stores above land before the ones that replace them
         }
         if (full_path) {
+          if (MORE == BIASED) {
+            // the distance bias slope * (key - query), in raw units, two keys at a time
+            const float at = slope * (float)(key0 - t.pos0 - qi);
+            uint64_t bias2 = pack2(at, at + slope);
+            const uint64_t step2 = pack2(2.f * slope, 2.f * slope);
+#pragma unroll
+            for (int c = 0; c < 2; ++c)
+#pragma unroll
+              for (int i = 0; i < 32; i += 2) {
+                float b0, b1;
+                unpack2(add2(pack2(__uint_as_float(sv[c][i]), __uint_as_float(sv[c][i + 1])), bias2), b0, b1);
+                sv[c][i] = __float_as_uint(b0);
+                sv[c][i + 1] = __float_as_uint(b1);
+                bias2 = add2(bias2, step2);
+              }
+          }
           // maximum of the raw scores (the scale is positive), masked entries set to -inf in place
           float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
           if (need_mask) {                   // a tile on the diagonal, at the window's edge or at the end of the keys
@@ -631,7 +646,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap kv_map, const __grid_
             l *= corr;
           }
           __syncwarp();
-          row_sum = exponentials((m_ref == -INFINITY) ? 0.f : -m_ref);
+          row_sum = exponentials((m_ref == -INFINITY) ? 0.f : -m_ref, 0.f, 0.f);
         }
         l += row_sum;
         // rescale this row of O if its scale moved (the warp decides together: the TMEM access is warp-wide); the
@@ -820,7 +835,8 @@ BSPEC_API int bspec_attention_prefill_tc_capped(const void* q, long long q_row_s
   static bool attr_set_dev[bspec::kMaxDevices] = {};            // per device
   bool& attr_set = attr_set_dev[bspec::current_device()];
   if (!attr_set) {
-    for (const void* kernel : {(const void*)attn_prefill_tc_kernel<false>, (const void*)attn_prefill_tc_kernel<true>}) {
+    for (const void* kernel : {(const void*)attn_prefill_tc_kernel<PLAIN>, (const void*)attn_prefill_tc_kernel<BIASED>,
+                               (const void*)attn_prefill_tc_kernel<POOLED>}) {
       const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_bytes());
       if (e != cudaSuccess) return (int)e;
     }
@@ -836,7 +852,7 @@ BSPEC_API int bspec_attention_prefill_tc_capped(const void* q, long long q_row_s
                kv_indices, Hq, Hkv, n_entries, (int)n_items, page_size, scale * 1.4426950408889634f, window, min_q_long, \
                q_by_tma, work, sink_l2, softcap > 0.f ? softcap / scale : 0.f, \
                softcap > 0.f ? 2.f * scale * 1.4426950408889634f / softcap : 0.f, slopes, 1.f / scale, pool_map, pooled)
-  if (slopes != nullptr || pool > 0) GO(true); else GO(false);
+  if (slopes != nullptr) GO(BIASED); else if (pool > 0) GO(POOLED); else GO(PLAIN);
 #undef GO
   return BSPEC_LAUNCH_CHECK();
 }

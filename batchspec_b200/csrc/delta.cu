@@ -325,12 +325,26 @@ gated_rmsnorm_kernel(const float* __restrict__ o, const float* __restrict__ gate
   if (item >= n * H) return;
   const int t = item / H, h = item - t * H;
   const float* x = o + ((size_t)t * H + h) * V;
+  const float* gp = gate + (size_t)t * gate_stride + (size_t)h * V;
+  T* op = out + ((size_t)t * H + h) * V;
+  if (V == 128 && ((reinterpret_cast<uintptr_t>(gp) | reinterpret_cast<uintptr_t>(x)) & 15) == 0) {   // four numbers per lane
+    const float4 v = *reinterpret_cast<const float4*>(x + 4 * lane), g = *reinterpret_cast<const float4*>(gp + 4 * lane);
+    const float xv[4] = {v.x, v.y, v.z, v.w}, gv[4] = {g.x, g.y, g.z, g.w};
+    const float r = 1.f / sqrtf(warp_sum(v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w) / (float)V + eps);
+    T o4[4];
+#pragma unroll
+    for (int c = 0; c < 4; ++c) {
+      const float wv = w != nullptr ? load_as_f32(w, w_dtype, 4 * lane + c) : 1.f;
+      o4[c] = from_f32<T>(xv[c] * r * wv * (gate_kind == 1 ? 1.f / (1.f + expf(-gv[c])) : silu_f(gv[c])));
+    }
+    if constexpr (sizeof(T) == 4) *reinterpret_cast<float4*>(op + 4 * lane) = *reinterpret_cast<float4*>(o4);
+    else *reinterpret_cast<uint2*>(op + 4 * lane) = *reinterpret_cast<uint2*>(o4);
+    return;
+  }
   float ss = 0.f;
   for (int j = lane; j < V; j += 32) ss += x[j] * x[j];
   ss = warp_sum(ss);
   const float r = 1.f / sqrtf(ss / (float)V + eps);
-  const float* gp = gate + (size_t)t * gate_stride + (size_t)h * V;
-  T* op = out + ((size_t)t * H + h) * V;
   for (int j = lane; j < V; j += 32) op[j] = from_f32<T>(x[j] * r * (w != nullptr ? load_as_f32(w, w_dtype, j) : 1.f) * (gate_kind == 1 ? 1.f / (1.f + expf(-gp[j])) : silu_f(gp[j])));
 }
 

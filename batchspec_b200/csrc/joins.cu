@@ -58,40 +58,46 @@ template <> __device__ __forceinline__ void store4<__nv_bfloat16>(__nv_bfloat16*
   *reinterpret_cast<uint2*>(p) = v;
 }
 
-// Two block-wide sums at once, each with the order of block_sum.  scratch: 64 floats.
-__device__ __forceinline__ void block_sum2(float& a, float& b, float* scratch) {
+// Block-wide sums with a fixed tree; every call of a kernel has 32 floats of its own, so one barrier is enough.
+__device__ __forceinline__ float sum_once(float v, float* scratch) {
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = (blockDim.x + 31) >> 5;
+  v = warp_sum(v);
+  if (lane == 0) scratch[warp] = v;
+  __syncthreads();
+  return warp_sum(lane < nwarps ? scratch[lane] : 0.f);
+}
+__device__ __forceinline__ void sum_once2(float& a, float& b, float* scratch) {
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = (blockDim.x + 31) >> 5;
   a = warp_sum(a);
   b = warp_sum(b);
-  __syncthreads();
   if (lane == 0) { scratch[warp] = a; scratch[32 + warp] = b; }
   __syncthreads();
   a = warp_sum(lane < nwarps ? scratch[lane] : 0.f);
   b = warp_sum(lane < nwarps ? scratch[32 + lane] : 0.f);
 }
 
-template <typename TD, typename TO, int VPT, bool PAIR>
+template <typename TD, typename TO, int VPT, bool PAIR, bool DEPTH>
 __global__ void branch_join_kernel(const JoinArgs a) {
   bspec::pdl_prologue(73);
-  __shared__ float scratch[64];
+  __shared__ float scratch[128];
   const int d = a.d;
   long long row = a.rows != nullptr ? a.rows[blockIdx.x] : (long long)blockIdx.x;
   if (!bspec::in_range(row, a.n_src, 115)) return;
   const size_t base = (size_t)row * d, obase = (size_t)blockIdx.x * d;
-  float x[VPT][4], y[VPT][4], z[PAIR ? VPT : 1][4], h[VPT][4];
+  float x[VPT][4], y[VPT][4], z[PAIR ? VPT : 1][4], h[DEPTH ? VPT : 1][4];
   float sa = 0.f, sb = 0.f;
 #pragma unroll
   for (int k = 0; k < VPT; ++k) {
     const int i = 4 * (threadIdx.x + k * blockDim.x);
 #pragma unroll
-    for (int c = 0; c < 4; ++c) x[k][c] = y[k][c] = h[k][c] = 0.f;
+    for (int c = 0; c < 4; ++c) x[k][c] = y[k][c] = h[DEPTH ? k : 0][c] = 0.f;
     if (i < d) {
       if (a.src != nullptr) load4<float>(a.src + base + i, x[k]);
       if (a.delta != nullptr) load4<TD>(reinterpret_cast<const TD*>(a.delta) + base + i, y[k]);
       if (PAIR) load4<TD>(reinterpret_cast<const TD*>(a.delta_b) + base + i, z[PAIR ? k : 0]);
     }
   }
-  if (a.coef != nullptr) {
+  if (DEPTH) {
 #pragma unroll 2
     for (int j = 0; j < a.slot; ++j) {
       const float w = a.coef[j];
@@ -103,7 +109,7 @@ __global__ void branch_join_kernel(const JoinArgs a) {
           float v[4];
           load4<float>(hp + i, v);
 #pragma unroll
-          for (int c = 0; c < 4; ++c) h[k][c] += w * v[c];
+          for (int c = 0; c < 4; ++c) h[DEPTH ? k : 0][c] += w * v[c];
         }
       }
     }
@@ -119,7 +125,7 @@ __global__ void branch_join_kernel(const JoinArgs a) {
           sb += z[PAIR ? k : 0][c] * z[PAIR ? k : 0][c];
         }
     }
-    block_sum2(sa, sb, scratch);
+    sum_once2(sa, sb, scratch);
     const float ra = 1.f / sqrtf(sa / (float)d + a.branch_eps), rb = 1.f / sqrtf(sb / (float)d + a.branch_eps);
 #pragma unroll
     for (int k = 0; k < VPT; ++k) {
@@ -140,7 +146,7 @@ __global__ void branch_join_kernel(const JoinArgs a) {
     for (int k = 0; k < VPT; ++k)
 #pragma unroll
       for (int c = 0; c < 4; ++c) ss += y[k][c] * y[k][c];           // zeros beyond the row
-    const float r = 1.f / sqrtf(block_sum(ss, scratch) / (float)d + a.branch_eps);
+    const float r = 1.f / sqrtf(sum_once(ss, scratch + 64) / (float)d + a.branch_eps);
 #pragma unroll
     for (int k = 0; k < VPT; ++k) {
       const int i = 4 * (threadIdx.x + k * blockDim.x);
@@ -152,7 +158,7 @@ __global__ void branch_join_kernel(const JoinArgs a) {
       }
     }
   }
-  const float own = a.coef != nullptr ? a.coef[a.slot] : 1.f;
+  const float own = DEPTH ? a.coef[a.slot] : 1.f;
   float ss = 0.f;
 #pragma unroll
   for (int k = 0; k < VPT; ++k) {
@@ -161,16 +167,16 @@ __global__ void branch_join_kernel(const JoinArgs a) {
 #pragma unroll
       for (int c = 0; c < 4; ++c) x[k][c] += y[k][c];
       if (a.store) store4<float>(a.hist + (size_t)a.slot * a.hist_stride + base + i, x[k]);
-      if (a.coef != nullptr)
+      if (DEPTH)
 #pragma unroll
-        for (int c = 0; c < 4; ++c) x[k][c] = h[k][c] + own * x[k][c];
+        for (int c = 0; c < 4; ++c) x[k][c] = h[DEPTH ? k : 0][c] + own * x[k][c];
       if (a.dst != nullptr) store4<float>(a.dst + obase + i, x[k]);
 #pragma unroll
       for (int c = 0; c < 4; ++c) ss += x[k][c] * x[k][c];
     }
   }
   if (a.out == nullptr) return;
-  const float r = a.norm_w != nullptr ? 1.f / sqrtf(block_sum(ss, scratch) / (float)d + a.eps) : 1.f;
+  const float r = a.norm_w != nullptr ? 1.f / sqrtf(sum_once(ss, scratch + 96) / (float)d + a.eps) : 1.f;
 #pragma unroll
   for (int k = 0; k < VPT; ++k) {
     const int i = 4 * (threadIdx.x + k * blockDim.x);
@@ -189,7 +195,7 @@ template <typename TD, typename TO>
 __global__ void branch_join_any_kernel(const JoinArgs a) {
   bspec::pdl_prologue(73);
   extern __shared__ float ys[];                       // [d] the branch, then the new row
-  __shared__ float scratch[64];
+  __shared__ float scratch[128];
   const int d = a.d;
   long long row = a.rows != nullptr ? a.rows[blockIdx.x] : (long long)blockIdx.x;
   if (!bspec::in_range(row, a.n_src, 115)) return;
@@ -203,7 +209,7 @@ __global__ void branch_join_any_kernel(const JoinArgs a) {
       sa += u * u;
       sb += v * v;
     }
-    block_sum2(sa, sb, scratch);
+    sum_once2(sa, sb, scratch);
   }
   const float ra = 1.f / sqrtf(sa / (float)d + a.branch_eps), rb = 1.f / sqrtf(sb / (float)d + a.branch_eps);
   float ss = 0.f;
@@ -213,7 +219,7 @@ __global__ void branch_join_any_kernel(const JoinArgs a) {
     ys[i] = y;                                        // a thread reads back only its own columns
     ss += y * y;
   }
-  const float rp = a.post != nullptr ? 1.f / sqrtf(block_sum(ss, scratch) / (float)d + a.branch_eps) : 1.f;
+  const float rp = a.post != nullptr ? 1.f / sqrtf(sum_once(ss, scratch + 64) / (float)d + a.branch_eps) : 1.f;
   ss = 0.f;
   for (int i = threadIdx.x; i < d; i += blockDim.x) {
     float x = (a.src != nullptr ? a.src[base + i] : 0.f) + ys[i] * rp * (a.post != nullptr ? a.post[i] : 1.f);
@@ -228,7 +234,7 @@ __global__ void branch_join_any_kernel(const JoinArgs a) {
     ss += x * x;
   }
   if (a.out == nullptr) return;
-  const float r = a.norm_w != nullptr ? 1.f / sqrtf(block_sum(ss, scratch) / (float)d + a.eps) : 1.f;
+  const float r = a.norm_w != nullptr ? 1.f / sqrtf(sum_once(ss, scratch + 96) / (float)d + a.eps) : 1.f;
   for (int i = threadIdx.x; i < d; i += blockDim.x)
     reinterpret_cast<TO*>(a.out)[obase + i] = from_f32<TO>(ys[i] * r * (a.norm_w != nullptr ? a.norm_w[i] : 1.f));
 }
@@ -239,18 +245,20 @@ int launch_join(const JoinArgs& a, int n, cudaStream_t stream) {
   if (d % 4 == 0 && d <= 4 * 4 * 1024) {
     const int quads = d / 4;
     int threads = quads >= 1024 ? 1024 : ((quads + 31) / 32) * 32;
-    // Many rows: several quads per thread, so that a thread has more loads in flight and several rows share an SM.
+    // Many rows: four quads per thread, so that a thread has more loads in flight and several rows share an SM.
     // Only for bfloat16 output: in float32 a row's sums keep one order, whatever else is in the step.
-    if (sizeof(TO) == 2 && n >= 512 && quads >= 128) threads = (((quads + 1) / 2 + 31) / 32) * 32;
+    if (sizeof(TO) == 2 && n >= 512 && quads >= 128) threads = (((quads + 3) / 4 + 31) / 32) * 32;
     if (threads > 1024) threads = 1024;
     const int vpt = (quads + threads - 1) / threads;
-#define LJ(V)                                                                                              \
-  do {                                                                                                     \
-    if (a.delta_b != nullptr) BSPEC_LAUNCH((branch_join_kernel<TD, TO, V, true>), n, threads, 0, stream, a); \
-    else BSPEC_LAUNCH((branch_join_kernel<TD, TO, V, false>), n, threads, 0, stream, a);                     \
+#define LJP(V, P)                                                                                              \
+  do {                                                                                                         \
+    if (a.coef != nullptr) BSPEC_LAUNCH((branch_join_kernel<TD, TO, V, P, true>), n, threads, 0, stream, a);     \
+    else BSPEC_LAUNCH((branch_join_kernel<TD, TO, V, P, false>), n, threads, 0, stream, a);                      \
   } while (0)
+#define LJ(V) do { if (a.delta_b != nullptr) LJP(V, true); else LJP(V, false); } while (0)
     if (vpt <= 1) LJ(1); else if (vpt <= 2) LJ(2); else LJ(4);
 #undef LJ
+#undef LJP
     return BSPEC_LAUNCH_CHECK();
   }
   const size_t smem = (size_t)d * sizeof(float);

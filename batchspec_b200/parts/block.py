@@ -180,6 +180,8 @@ class LearnedDepthAverage(Part):
         return {"weight": ParamSpec((self.count,), role="vector", init="ones_normal")}
 
     def bind(self, params):
+        if torch.device(self.runtime.device).type == "cuda":
+            ops.require("joins")                  # the kernels of csrc/joins.cu
         self.weight = params["weight"].to(torch.float32).contiguous()
 
 

@@ -90,6 +90,14 @@ def test_tensor_names_block_kinds_and_needs():
     assert cache.layer_caches[0].pooled is None and cache.groups[2].pool.num_pages == 5 + 3
 
 
+def test_presets_by_name_build():
+    from batchspec_b200.config import get_config
+    for name in ("tiny-podizen", "podizen-w2048"):
+        cfg = get_config(name)
+        m = get_model(cfg, Runtime(torch.bfloat16, torch.device("cpu")))
+        assert cfg.architecture == "Podizen" and len(m.blocks) == len(cfg.layers)
+
+
 # ---------------------------------------------------------------------------------- pooled blocks in the cache manager
 
 def pooled_manager(window, pool, page=4, pages=40, requests=3):
