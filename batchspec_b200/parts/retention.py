@@ -1,9 +1,9 @@
-"""Retention: linear attention with rotary positions, a fixed decay per head and neither softmax nor denominator.
+"""Retention: a decaying [key x value] state per head, read by rotated queries and written by rotated keys.
 
 With h the token's normed input and H heads:
 
     q, k = Wq h, Wk h   (H x dim, both rotated by position),   v = Wv h   (H x v_dim),   k <- k / sqrt(dim)
-    S_t = decay_h S_(t-1) + k_t v_t^T,   o_t = S_t^T q_t
+    per head:  S <- decay S + k v^T,   o = S^T q         S from zero, a token reads its own write
     out = Wo (concat_heads(o / rms(o)) * silu(Wg h))              every head normed by itself, no weight
 
 Everything between the projections and the output projection is float32.  The state of a request is one float32 row

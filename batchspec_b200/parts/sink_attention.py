@@ -13,9 +13,9 @@
   all heads and no tensor (0.0 adds one to the denominator);
 * ``softcap`` c: a scaled score s becomes c tanh(s / c);
 * ``bias_slopes``: a distance bias, slope_h * (i - j) taken off the scaled score of query i and key j;
-* ``pool`` P, with a window W: beside the W tokens a query sees one entry for each block of P tokens that lies wholly
-  before its window (last position at most i - W): the mean of the block's keys and of its values, as the cache holds
-  them; tokens that have left the window and whose block is not yet seen are not seen at all;
+* ``pool`` P, with a window W: the positions are cut into blocks of P from 0 on, and query i also attends, in the same
+  softmax, to one entry per block whose last position is at most i - W: the mean of the block's cached keys with the
+  mean of its values.  A token between its window and its block's turn has no influence;
 * ``values_are_keys``: there is no value projection, a key as projected is its own value, and only keys are cached;
 * ``gate``: the concatenated heads are multiplied element by element by sigmoid(Wg h) before the output projection;
   ``gate="head"``: Wg has one row per head and the head's whole output is multiplied by one number.

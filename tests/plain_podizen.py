@@ -207,8 +207,7 @@ def forward(cfg: dict, tensors: Dict[str, torch.Tensor], tokens: Sequence[int], 
 
 # ---------------------------------------------------------------------------------------------- a model folder
 def read_tensors(path) -> Dict[str, torch.Tensor]:
-    """A safetensors file: an 8-byte little-endian length, that many bytes of JSON (name -> dtype, shape, offsets), the
-    data.  bfloat16 comes back as float32 with the same values."""
+    """All tensors of a safetensors file by name; bfloat16 comes back as float32 with the same values."""
     import struct
     import numpy as np
     raw = Path(path).read_bytes()
