@@ -8,7 +8,7 @@ Here all bookkeeping is on the host: a pool is a LIFO free list shared by all
 requests, a request holds ceil(len / page_size) table entries per group (none when
 empty), finished requests' pages go back to the list and are handed out again, and
 a windowed group also gives back pages that the window has passed (their table
-entries become -1; no kernel reads them), and a chunked group the pages before the
+entries become -1; no kernel reads them; pages of first tokens that stay visible are kept), and a chunked group the pages before the
 chunk that the next position falls into.
 
 A mixer that also keeps one entry per whole block of P tokens (``CacheSpec.pool``) gets a second group for
@@ -119,6 +119,11 @@ class CacheGroup:
             n *= s
         return n
 
+    @property
+    def kept_pages(self) -> int:
+        """Leading pages that are never given back while the request lives."""
+        return -(-self.spec.keep // self.page_size)
+
     def pages_for(self, length: int) -> int:
         """Table entries of a request of ``length`` tokens: only whole blocks of ``stride`` tokens have an entry."""
         return -(-(length // self.stride) // self.page_size)
@@ -131,7 +136,7 @@ class RequestCache:
     length: int = 0
     tables: List[List[int]] = field(default_factory=list)   # per group: page id per logical page, -1 once released
     serial: int = 0     # which admission this is: a request that is released and admitted again gets a new one
-    dead: List[int] = field(default_factory=list)   # per group: how many leading pages were given back (all -1)
+    dead: List[int] = field(default_factory=list)   # per group: pages before this one were given back (-1), the kept ones aside
 
 
 class CacheManager:
@@ -160,7 +165,7 @@ class CacheManager:
 
         def join_group(run, c: CacheSpec, stride: int) -> Tuple[int, int]:
             group_page = int(c.page_size or self.page_size)
-            key = (c.policy, c.window, tuple(c.entry_shape), c.tensors, group_page, c.pool, stride)
+            key = (c.policy, c.window, tuple(c.entry_shape), c.tensors, group_page, c.pool, c.keep, stride)
             if key not in key_to_group:
                 key_to_group[key] = len(self.groups)
                 if isinstance(num_pages, (list, tuple)):
@@ -182,7 +187,7 @@ class CacheManager:
             if c.pool:
                 if c.pool < 0:
                     raise ValueError(f"run {e}: a pooled block holds at least one token, got {c}")
-                run_pooled[e] = join_group(e, replace(c, policy="full", window=None, pool=0), c.pool)
+                run_pooled[e] = join_group(e, replace(c, policy="full", window=None, pool=0, keep=0), c.pool)
         if allocate:
             for grp in self.groups:
                 # zeroed once: kernels may load (and mask) rows of a page that no token has been written to yet,
@@ -256,13 +261,13 @@ class CacheManager:
         """Per group, the most pages one request of ``total_len`` tokens holds at any time when it is fed in
         portions of at most ``portion`` tokens: all of them in a group that keeps every key; in a window's group
         the pages from the oldest key a query still reads to the end of the portion being written (the pages the
-        window has passed were given back at the commit before)."""
+        window has passed were given back at the commit before), and those of first tokens that stay."""
         out = []
         for g in self.groups:
             ps = g.page_size
             n = g.pages_for(total_len)
             if g.spec.policy in ("window", "chunk"):
-                n = min(n, (max(g.spec.window, g.spec.pool) - 1 + max(1, portion) + ps - 1) // ps + 1)
+                n = min(n, (max(g.spec.window, g.spec.pool) - 1 + max(1, portion) + ps - 1) // ps + 1 + g.kept_pages)
             out.append(n)
         return out
 
@@ -318,7 +323,7 @@ class CacheManager:
             else:
                 continue
             dead = first_needed // g.page_size             # pages wholly before first_needed
-            was = rc.dead[gi]                              # those before ``was`` went back at earlier commits
+            was = max(rc.dead[gi], g.kept_pages)           # those before ``was`` went back at earlier commits, or stay
             if dead > was:
                 g.pool.free(table[was:dead])
                 table[was:dead] = [-1] * (dead - was)
@@ -344,7 +349,8 @@ class CacheManager:
             assert set(held).isdisjoint(g.pool._free), "a held page is on the free list"
             assert len(set(g.pool._free)) == len(g.pool._free), "a page is on the free list twice"
         for rc in self.requests.values():
-            for table, dead in zip(rc.tables, rc.dead):
-                assert all(p < 0 for p in table[:dead]) and all(p >= 0 for p in table[dead:]), \
-                    "pages are given back from the front only"
+            for g, table, dead in zip(self.groups, rc.tables, rc.dead):
+                kept = min(g.kept_pages, len(table))
+                assert all(p < 0 for p in table[kept:dead]) and all(p >= 0 for p in table[:kept] + table[max(kept, dead):]), \
+                    "pages are given back from the front only, those of kept first tokens never"
         assert len(self.requests) == self.slots.n - self.slots.num_free

@@ -74,8 +74,9 @@ struct TileGeom {
   int e, g, q_begin, q_len, pos0, G, rows_total;
 };
 
-// Pooled blocks before a window: ``size`` tokens each (0: none), with their block tables.  Their entries are keys of a
-// second source, visited before the tokens: key number b is block b, seen by a query if b < pooled_seen(query).
+// What a query sees before its window, with block tables: pooled blocks of ``size`` tokens each (0: none), or the first
+// -size tokens (their own pages and tables).  Either are keys of a second source, visited before the tokens of the
+// window: key number b of it is seen by a query if b < pooled_seen(query).
 struct Pooled {
   int size;
   const int* indptr;
@@ -668,7 +669,7 @@ __device__ __forceinline__ void piece_at(Piece& pc, long long pos, long long sha
   pc.k_begin = pc.k_end = pc.lo_key = 0;
   if (pc.row0 >= t.rows_total) return;
   int skip = 0;                                  // the request's tiles of pooled blocks come before its tokens' tiles
-  if (pool > 0) {
+  if (pool != 0) {
     pc.pool_end = bspec::pooled_seen(t.pos0 + t.q_len - 1, window, pool);
     skip = (pc.pool_end + KT - 1) / KT;
     pc.n_pool = max(0, min(t1, skip) - t0);
@@ -703,7 +704,7 @@ __device__ __forceinline__ bool make_shares(Shares& sh, int* cum, int* pos0_of, 
       pos0 = kv_len != nullptr ? len_after - ql : positions[qb];
       const int lo_entry = bspec::mask_lo(pos0, window);
       tiles = (pos0 + ql - (lo_entry / KT) * KT + KT - 1) / KT;
-      if (pool > 0) tiles += (bspec::pooled_seen(pos0 + ql - 1, window, pool) + KT - 1) / KT;
+      if (pool != 0) tiles += (bspec::pooled_seen(pos0 + ql - 1, window, pool) + KT - 1) / KT;
     }
     pos0_of[e] = pos0;
     rows_of[e] = qb | (tiles > 0 ? ql << 26 : 0);
@@ -823,7 +824,7 @@ __device__ __forceinline__ void join_parts(float* Wt, __nv_bfloat16* __restrict_
   bar_consumers();
 }
 
-// MORE: a distance bias or pooled blocks may be given; without it the code for both is left out.
+// MORE: a distance bias, or pooled blocks or kept first tokens, may be given; without it the code for both is left out.
 template <int HD, bool MORE>
 __global__ void __launch_bounds__(DECODE_TMA_THREADS, HD <= 64 ? 3 : (HD <= 128 ? 2 : 1))
 attn_decode_shares_kernel(const __grid_constant__ CUtensorMap kv_map, const __nv_bfloat16* __restrict__ q,
@@ -909,7 +910,7 @@ attn_decode_shares_kernel(const __grid_constant__ CUtensorMap kv_map, const __nv
         const uint32_t ph = (tile_no / TMA_STAGES) & 1u;
         const bool blocks = MORE && k < pc.n_pool;
         const int key0 = blocks ? pc.pool_k0 + k * KT : pc.k_begin + (k - pc.n_pool) * KT;
-        if (!waited && (tile_no >= TMA_STAGES || key0 + KT > (blocks ? pc.t.pos0 / pooled.size : pc.t.pos0))) {
+        if (!waited && (tile_no >= TMA_STAGES || key0 + KT > (blocks && pooled.size > 0 ? pc.t.pos0 / pooled.size : pc.t.pos0))) {
           bspec::pdl_wait();           // this tile holds new keys, or a stage must first be released by consumers
           waited = true;
         }
@@ -970,7 +971,7 @@ attn_decode_shares_kernel(const __grid_constant__ CUtensorMap kv_map, const __nv
         const int qi = row / t.G;
         lim[r] = row < t.rows_total ? t.pos0 + qi : -1;
         lo[r] = bspec::mask_lo(t.pos0 + qi, window);
-        blk[r] = pooled.size > 0 && row < t.rows_total ? bspec::pooled_seen(t.pos0 + qi, window, pooled.size) - 1 : -1;
+        blk[r] = pooled.size != 0 && row < t.rows_total ? bspec::pooled_seen(t.pos0 + qi, window, pooled.size) - 1 : -1;
       }
       float sl[2];
       row_slopes(sl, slopes_l2, pc.g, t.G, pc.row0, t.rows_total);
@@ -1245,7 +1246,7 @@ attn_prefill_tma_kernel(const __grid_constant__ CUtensorMap kv_map, const __nv_b
   const int hi_key = t.pos0 + qi_hi;
   const int lo_key = bspec::mask_lo(t.pos0 + qi_lo, window);
   const int k_begin = (lo_key / KT) * KT, k_end = hi_key + 1;
-  const int pool_end = pooled.size > 0 ? bspec::pooled_seen(hi_key, window, pooled.size) : 0;
+  const int pool_end = pooled.size != 0 ? bspec::pooled_seen(hi_key, window, pooled.size) : 0;
   const int n_pool = (pool_end + KT - 1) / KT;                                // tiles of pooled blocks, before the tokens'
   const int n_tiles = n_pool + (k_end - k_begin + KT - 1) / KT;
   const int* table = kv_indices + kv_indptr[e];
@@ -1301,7 +1302,7 @@ attn_prefill_tma_kernel(const __grid_constant__ CUtensorMap kv_map, const __nv_b
     const int qi = row / t.G;
     lim[r] = row < t.rows_total ? t.pos0 + qi : -1;
     lo[r] = bspec::mask_lo(t.pos0 + qi, window);
-    blk[r] = pooled.size > 0 && row < t.rows_total ? bspec::pooled_seen(t.pos0 + qi, window, pooled.size) - 1 : -1;
+    blk[r] = pooled.size != 0 && row < t.rows_total ? bspec::pooled_seen(t.pos0 + qi, window, pooled.size) - 1 : -1;
   }
   float sl[2];
   row_slopes(sl, slopes_l2, g, t.G, wrow0, t.rows_total);
@@ -1522,11 +1523,11 @@ int launch(const __nv_bfloat16* q, long long q_row_stride, __nv_bfloat16* out, f
     resident_dev[cur_dev] = bspec::sm_count() * (per_sm > 0 ? per_sm : 1);
   });
   const int resident = resident_dev[cur_dev];      // of the plain kernel; a grid above what is resident only costs time
-  const bool more = slopes_l2 != nullptr || pooled.size > 0;
+  const bool more = slopes_l2 != nullptr || pooled.size != 0;
   // Pooled blocks are served by the kernels that load K/V through TMA: equal shares for the short requests, 128-row
   // tiles (HD <= 128) for the others.  Where those cannot run, the call is refused (not run without the blocks).
   CUtensorMap pool_map;
-  if (pooled.size > 0 && (pool_rows <= 0 || !make_map_2d_bf16(&pool_map, pool_cache, pool_rows, HD, page_size, 64)))
+  if (pooled.size != 0 && (pool_rows <= 0 || !make_map_2d_bf16(&pool_map, pool_cache, pool_rows, HD, page_size, 64)))
     return (int)cudaErrorInvalidValue;
   if (run_decode) {
     const int short_q = max_q_len < max_q_short ? max_q_len : max_q_short;
@@ -1543,13 +1544,13 @@ int launch(const __nv_bfloat16* q, long long q_row_stride, __nv_bfloat16* out, f
         BSPEC_LAUNCH((attn_decode_shares_kernel<HD, MORE>), dim3(resident), DECODE_TMA_THREADS, decode_shares_smem<HD>(), \
                      stream, kv_map, q, q_row_stride, out, o_part, ml_part, tile_counters, status, qo_indptr, positions, \
                      kv_len, kv_indptr, kv_indices, n_entries, Hq, Hkv, page_size, scale_log2, softcap, window, n_splits, \
-                     short_q, row_tiles, max_q_short, sink_l2, slopes_l2, pooled.size > 0 ? pool_map : kv_map, pooled)
+                     short_q, row_tiles, max_q_short, sink_l2, slopes_l2, pooled.size != 0 ? pool_map : kv_map, pooled)
         if (more) GO(true); else GO(false);
 #undef GO
         launched = true;
        }
       }
-      if (!launched && pooled.size > 0) return (int)cudaErrorInvalidValue;
+      if (!launched && pooled.size != 0) return (int)cudaErrorInvalidValue;
       if (!launched && make_map_2d_bf16(&kv_map, cache, kv_rows, HD, page_size, 64)) {
         BSPEC_LAUNCH((attn_decode_tma_kernel<HD>), grid, DECODE_TMA_THREADS, decode_tma_smem<HD>(), stream, kv_map, q,
                      q_row_stride, out, o_part, ml_part, tile_counters, status, qo_indptr, positions, kv_indptr,
@@ -1558,7 +1559,7 @@ int launch(const __nv_bfloat16* q, long long q_row_stride, __nv_bfloat16* out, f
         launched = true;
       }
     }
-    if (!launched && pooled.size > 0) return (int)cudaErrorInvalidValue;
+    if (!launched && pooled.size != 0) return (int)cudaErrorInvalidValue;
     if (!launched)
       BSPEC_LAUNCH((attn_decode_kernel<HD>), grid, NTHREADS, decode_smem<HD>(), stream,
                    q, q_row_stride, out, o_part, ml_part, tile_counters, cache, qo_indptr, positions, kv_indptr,
@@ -1578,7 +1579,7 @@ int launch(const __nv_bfloat16* q, long long q_row_stride, __nv_bfloat16* out, f
 #define GO(MORE) \
         BSPEC_LAUNCH((attn_prefill_tma_kernel<HD, MORE>), grid, PREFILL_TMA_THREADS, prefill_tma_smem<HD>(), stream, kv_map, \
                      q, q_row_stride, out, status, qo_indptr, positions, kv_indptr, kv_indices, Hq, Hkv, page_size, \
-                     scale_log2, softcap, window, max_q_short + 1, sink_l2, slopes_l2, pooled.size > 0 ? pool_map : kv_map, \
+                     scale_log2, softcap, window, max_q_short + 1, sink_l2, slopes_l2, pooled.size != 0 ? pool_map : kv_map, \
                      pooled)
         if (more) GO(true); else GO(false);
 #undef GO
@@ -1586,7 +1587,7 @@ int launch(const __nv_bfloat16* q, long long q_row_stride, __nv_bfloat16* out, f
       }
      }
     }
-    if (!launched && pooled.size > 0) return (int)cudaErrorInvalidValue;
+    if (!launched && pooled.size != 0) return (int)cudaErrorInvalidValue;
     if (!launched) {
       dim3 grid((max_q_len * G + 63) / 64, Hkv, n_entries);
       BSPEC_LAUNCH((attn_prefill_kernel<HD>), grid, NTHREADS, prefill_smem<HD>(), stream,
@@ -1641,6 +1642,8 @@ BSPEC_API int bspec_attention_bf16(const void* q, long long q_row_stride, void* 
 // null): float32 per query head, a slope times log2(e); slope * (query - key) is taken off a token's score.  ``pool`` P >
 // 0, with a window: before the window a query also sees one entry per block of P tokens that lies wholly before it
 // (pages of the same layout; needs n_pages, ``balanced`` for short requests, and head_dim <= 128 for the others).
+// ``pool`` < 0, on the same terms: the request's first -pool tokens stay visible (pool_cache and its tables are the
+// tokens' own).
 BSPEC_API int bspec_attention_bf16_masked(const void* q, long long q_row_stride, void* out, float* o_part, float* ml_part,
                                           int* tile_counters, int* status, long long n_pages, const void* cache,
                                           const int* qo_indptr, const int* positions, const int* tok_entry,
@@ -1652,7 +1655,7 @@ BSPEC_API int bspec_attention_bf16_masked(const void* q, long long q_row_stride,
                                           const int* pool_indptr, const int* pool_indices, long long pool_pages,
                                           cudaStream_t stream) {
   if (n_entries <= 0 || n_tokens <= 0) return 0;
-  if (pool < 0 || (pool > 0 && (window <= 0 || slopes_l2 != nullptr || pool_cache == nullptr || pool_indptr == nullptr)))
+  if (pool != 0 && (window <= 0 || slopes_l2 != nullptr || pool_cache == nullptr || pool_indptr == nullptr))
     return (int)cudaErrorInvalidValue;
   const Pooled pooled = {pool, pool_indptr, pool_indices};
   if (Hq % Hkv != 0 || n_splits < 1 || n_splits > 64) return (int)cudaErrorInvalidValue;

@@ -19,7 +19,8 @@
 // ``slopes`` (float32 per query head, or null): slope_h * (query - key) is taken off a token's score.  ``pool`` P > 0
 // (with a window W): before the window a query also sees one entry per block of P tokens that lies wholly before it,
 // floor((query - W + 1) / P) of them; they have pages and a table of their own (same page layout, entry b = block b)
-// and take part in the same softmax, first.
+// and take part in the same softmax, first.  ``pool`` < 0 (with a window): the request's first -pool tokens stay visible
+// when the window has passed them; they are visited first, from the tokens' own pages.
 #include "common.cuh"
 #include <math.h>
 using namespace bspec;
@@ -109,6 +110,10 @@ attn_generic_kernel(const T* __restrict__ q, long long q_row_stride, T* __restri
     }
     m = m_new;
   };
+  if (pool < 0) {
+    const int kept = bspec::pooled_seen(pos, window, pool);
+    for (int kb = 0; kb < kept; kb += 32) visit(kb, 0, kept - 1, table, cache, n_pages, slope);
+  }
   if (pool > 0) {
     const int blocks = bspec::pooled_seen(pos, window, pool);
     for (int kb = 0; kb < blocks; kb += 32)
@@ -150,7 +155,7 @@ static int launch_attention_generic(const void* q, long long q_row_stride, void*
                                     const float* slopes, int pool, const void* pool_cache, const int* pool_indptr,
                                     const int* pool_indices, long long pool_pages, cudaStream_t stream) {
   if (n_entries <= 0 || max_q_len <= 0) return 0;
-  if (pool < 0 || (pool > 0 && (window <= 0 || v_is_k || pool_cache == nullptr || pool_indptr == nullptr)))
+  if ((pool != 0 && window <= 0) || (pool > 0 && (v_is_k || pool_cache == nullptr || pool_indptr == nullptr)))
     return (int)cudaErrorInvalidValue;
   if (v_is_k && vd != hd) return (int)cudaErrorInvalidValue;
   if (hd > MAX_HD || hd <= 0 || vd > MAX_HD || vd <= 0 || Hq % Hkv != 0) return (int)cudaErrorInvalidValue;
@@ -183,8 +188,8 @@ BSPEC_API int bspec_attention_generic(const void* q, long long q_row_stride, voi
 
 // The same with values of their own size ``vd``, a chunk mask (0: none), a sink per query head (null: none), a soft
 // cap on the scores (0: none), values that are the keys, a sigmoid gate on the output (per number, or per head), an
-// output scale and stride, a distance bias (slopes per query head, null: none) and pooled blocks before the window
-// (0: none).
+// output scale and stride, a distance bias (slopes per query head, null: none) and pooled blocks or kept first tokens
+// before the window (pool > 0 or < 0; 0: none).
 BSPEC_API int bspec_attention_masked(const void* q, long long q_row_stride, void* out, const void* cache, int dtype,
                                      const int* qo_indptr, const int* positions, const int* kv_indptr,
                                      const int* kv_indices, int n_entries, int max_q_len, int Hq, int Hkv, int hd,

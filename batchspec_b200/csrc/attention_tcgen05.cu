@@ -24,7 +24,8 @@
 // Tensor memory: 2 x 2 S buffers of 64 columns, 2 O accumulators of 128 (all 512 columns).  Every mbarrier wait is
 // bounded; on expiry a code goes to `status`, all roles stop and the tensor memory is given back.
 // With pooled blocks before a window an item walks key tiles of two sources: first the request's block entries (their
-// own pages and table, the same layout), then its tokens; both are tiles of the same ring and the same softmax.
+// own pages and table, the same layout), then its tokens; both are tiles of the same ring and the same softmax.  First
+// tokens that stay visible when the window has passed them are such a source too, in the tokens' own pages.
 // With a distance bias an item walks its key tiles from the last to the first: the bias grows towards the query, by tens
 // of units a tile for the steep heads, so in ascending order nearly every tile would move the maximum and rescale O.
 #include "common.cuh"
@@ -160,7 +161,7 @@ struct Item {
   const int* ptable;
 };
 
-// Pooled blocks before the window: ``size`` tokens each (0: none), with their block tables.
+// Before the window: pooled blocks of ``size`` tokens each (0: none), or the first -size tokens, with their block tables.
 struct Pooled {
   int size;
   const int* indptr;
@@ -192,7 +193,7 @@ __device__ __forceinline__ bool load_item(Item& it, int idx, int Hq, int Hkv, in
   it.lo_key = bspec::mask_lo(t.pos0 + qi_lo, window);
   it.k_begin = (it.lo_key / KT) * KT;
   it.pool_end = 0;
-  if (pooled.size > 0)
+  if (pooled.size != 0)
     it.pool_end = bspec::pooled_seen(t.pos0 + min(t.q_len - 1, (it.row0 + QT * ROWS - 1) / t.G), window, pooled.size);
   it.n_pool = (it.pool_end + KT - 1) / KT;
   it.ptable = it.n_pool > 0 ? pooled.indices + pooled.indptr[e] : nullptr;
@@ -510,7 +511,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap kv_map, const __grid_
       const int lim = live ? t.pos0 + qi : -1;
       const int lo = bspec::mask_lo(t.pos0 + qi, window);
       const int my_k_end = it.k_end_t[tt];
-      const int last_block = live && pooled.size > 0 ? bspec::pooled_seen(t.pos0 + qi, window, pooled.size) - 1 : -1;
+      const int last_block = live && pooled.size != 0 ? bspec::pooled_seen(t.pos0 + qi, window, pooled.size) - 1 : -1;
       const float slope = slopes != nullptr ? slopes[h] * inv_scale : 0.f;      // in units of the raw scores
       if (!q_by_tma) {
         // Q tile: this thread copies its own row (16 chunks of 16 bytes) into the swizzled operand layout.  The
@@ -803,7 +804,8 @@ BSPEC_API int bspec_attention_prefill_tc_masked(const void* q, long long q_row_s
 
 // The same with a soft cap c > 0 on the scaled scores (c tanh(s / c)), 0 is none; ``slopes`` (may be null): float32 per
 // query head, slope * (query - key) is taken off a token's scaled score; ``pool`` P > 0, with a window: before the window
-// a query also sees one entry per block of P tokens that lies wholly before it, from pages of the same layout.
+// a query also sees one entry per block of P tokens that lies wholly before it, from pages of the same layout; ``pool`` <
+// 0: the request's first -pool tokens instead, from the pages given there (the tokens' own).
 BSPEC_API int bspec_attention_prefill_tc_capped(const void* q, long long q_row_stride, void* out, int* status,
                                                 long long n_pages, const void* cache, const int* qo_indptr,
                                                 const int* positions, const int* kv_indptr, const int* kv_indices,
@@ -817,13 +819,12 @@ BSPEC_API int bspec_attention_prefill_tc_capped(const void* q, long long q_row_s
   if (hd != HD || Hq % Hkv != 0 || page_size % 8 != 0 || KT % page_size != 0 || status == nullptr || n_pages <= 0 ||
       n_tokens <= 0 || work == nullptr)
     return (int)cudaErrorInvalidValue;
-  if (pool < 0 || (pool > 0 && (window <= 0 || slopes != nullptr || pool_cache == nullptr || pool_indptr == nullptr ||
-                                pool_pages <= 0)))
+  if (pool != 0 && (window <= 0 || slopes != nullptr || pool_cache == nullptr || pool_indptr == nullptr || pool_pages <= 0))
     return (int)cudaErrorInvalidValue;
   CUtensorMap kv_map, q_map, pool_map;
   if (!make_map_2d_bf16(&kv_map, cache, n_pages * 2 * Hkv * page_size, HD, page_size, 64)) return (int)cudaErrorInvalidValue;
   pool_map = kv_map;                                             // not read without pooled blocks
-  if (pool > 0 && !make_map_2d_bf16(&pool_map, pool_cache, pool_pages * 2 * Hkv * page_size, HD, page_size, 64))
+  if (pool != 0 && !make_map_2d_bf16(&pool_map, pool_cache, pool_pages * 2 * Hkv * page_size, HD, page_size, 64))
     return (int)cudaErrorInvalidValue;
   const Pooled pooled = {pool, pool_indptr, pool_indices};
   const int G = Hq / Hkv;
@@ -852,7 +853,7 @@ BSPEC_API int bspec_attention_prefill_tc_capped(const void* q, long long q_row_s
                kv_indices, Hq, Hkv, n_entries, (int)n_items, page_size, scale * 1.4426950408889634f, window, min_q_long, \
                q_by_tma, work, sink_l2, softcap > 0.f ? softcap / scale : 0.f, \
                softcap > 0.f ? 2.f * scale * 1.4426950408889634f / softcap : 0.f, slopes, 1.f / scale, pool_map, pooled)
-  if (slopes != nullptr) GO(BIASED); else if (pool > 0) GO(POOLED); else GO(PLAIN);
+  if (slopes != nullptr) GO(BIASED); else if (pool != 0) GO(POOLED); else GO(PLAIN);
 #undef GO
   return BSPEC_LAUNCH_CHECK();
 }

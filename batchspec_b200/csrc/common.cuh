@@ -43,10 +43,13 @@ __device__ __forceinline__ float warp_max(float v) {
 __device__ __forceinline__ int mask_lo(int pos, int window) {
   return window > 0 ? max(0, pos - window + 1) : (window < 0 ? (pos / -window) * -window : 0);
 }
-// Blocks of ``pool`` positions that lie wholly before the window of a query at ``pos``: block b is seen when its last
-// position b pool + pool - 1 is at most pos - window.
+// Keys of a second source that a query at ``pos`` sees before its window, keys 0 .. of that source.  ``pool`` > 0: blocks of
+// ``pool`` positions that lie wholly before the window (block b when its last position b pool + pool - 1 is at most
+// pos - window).  ``pool`` < 0: the request's first -pool tokens as far as they lie before the window (the others are
+// seen as keys of the window).
 __device__ __forceinline__ int pooled_seen(int pos, int window, int pool) {
-  return pos - window + 1 > 0 ? (pos - window + 1) / pool : 0;
+  const int before = max(0, pos - window + 1);
+  return pool > 0 ? before / pool : min(-pool, before);
 }
 // A softmax sink is a logit per head that adds exp(sink) to the denominator and nothing to the numerator.  With the running maximum ``m`` and sum ``l``
 // in base-2 units and ``sink_l2`` = sink * log2(e) per query head (null: none): the sum with the sink's term.

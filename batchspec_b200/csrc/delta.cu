@@ -10,7 +10,7 @@
 //   delta_recurrence  per (request, head, 32 or 8 value columns): the token loop over the portion with the state in
 //                     registers (a column of S is spread over four lanes), state read at the start and written at
 //                     the end; the request's blocks also move the convolutions' inputs on
-//   gated_rmsnorm     per (token, head): o / rms(o) * w * silu(gate)
+//   gated_rmsnorm     per (token, head): o / rms(o) * w * silu(gate), with options other mixers use
 //
 // The order of every sum depends on the sizes alone, not on how a request was cut into portions or on what else is
 // in the step.
@@ -313,39 +313,62 @@ delta_recurrence_kernel(const float* __restrict__ mix, const float* __restrict__
   }
 }
 
-// out[t, h*V + j] = o[t, h, j] / sqrt(mean_j o^2 + eps) * w[j] * act(gate[t, h*V + j]), act = silu (gate_kind 0) or
-// sigmoid (1), w null: no weight; one warp per (token, head).
+// out[t, h*V + j] = x / sqrt(mean_j x^2 + eps) * w[j] * act(gate[t, h*V + j]) * out_scale with x = o[t, h, j], or
+// o[t, h, j] / den[t, h] when ``den`` is given; w null: no weight.  ``flags``: bit 0 act = sigmoid (else silu), bit 1 the
+// gate comes before the norm (x is multiplied by act(gate) and normed then), bit 2 w has a number for every column
+// h*V + j instead of one set for all groups.  One warp per (token, group).
+constexpr int GN_SIGMOID = 1, GN_GATE_FIRST = 2, GN_FULL_WEIGHT = 4;
+
+__device__ __forceinline__ float gn_act(float g, int flags) {
+  return (flags & GN_SIGMOID) ? 1.f / (1.f + expf(-g)) : silu_f(g);
+}
+
 template <typename T>
 __global__ void __launch_bounds__(128)
 gated_rmsnorm_kernel(const float* __restrict__ o, const float* __restrict__ gate, long long gate_stride,
-                     const void* __restrict__ w, int w_dtype, T* __restrict__ out, int n, int H, int V, float eps,
-                     int gate_kind) {
+                     const void* __restrict__ w, int w_dtype, T* __restrict__ out, long long out_stride, int n, int H, int V,
+                     float eps, int flags, const float* __restrict__ den, float out_scale) {
   bspec::pdl_prologue(62);
   const int item = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (item >= n * H) return;
   const int t = item / H, h = item - t * H;
   const float* x = o + ((size_t)t * H + h) * V;
   const float* gp = gate + (size_t)t * gate_stride + (size_t)h * V;
-  T* op = out + ((size_t)t * H + h) * V;
-  if (V == 128 && ((reinterpret_cast<uintptr_t>(gp) | reinterpret_cast<uintptr_t>(x)) & 15) == 0) {   // four numbers per lane
+  const size_t w0 = (flags & GN_FULL_WEIGHT) ? (size_t)h * V : 0;
+  const bool first = flags & GN_GATE_FIRST;
+  T* op = out + (size_t)t * out_stride + (size_t)h * V;
+  const float d = den != nullptr ? den[item] : 1.f;
+  if (V == 128 && ((reinterpret_cast<uintptr_t>(gp) | reinterpret_cast<uintptr_t>(x)) & 15) == 0 &&
+      (reinterpret_cast<uintptr_t>(op) & (4 * sizeof(T) - 1)) == 0) {                  // four numbers per lane
     const float4 v = *reinterpret_cast<const float4*>(x + 4 * lane), g = *reinterpret_cast<const float4*>(gp + 4 * lane);
-    const float xv[4] = {v.x, v.y, v.z, v.w}, gv[4] = {g.x, g.y, g.z, g.w};
-    const float r = 1.f / sqrtf(warp_sum(v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w) / (float)V + eps);
+    float xv[4] = {v.x, v.y, v.z, v.w}, gv[4] = {g.x, g.y, g.z, g.w};
+#pragma unroll
+    for (int c = 0; c < 4; ++c) {
+      gv[c] = gn_act(gv[c], flags);
+      if (den != nullptr) xv[c] = xv[c] / d;
+      if (first) xv[c] *= gv[c];
+    }
+    const float r = 1.f / sqrtf(warp_sum(xv[0] * xv[0] + xv[1] * xv[1] + xv[2] * xv[2] + xv[3] * xv[3]) / (float)V + eps);
     T o4[4];
 #pragma unroll
     for (int c = 0; c < 4; ++c) {
-      const float wv = w != nullptr ? load_as_f32(w, w_dtype, 4 * lane + c) : 1.f;
-      o4[c] = from_f32<T>(xv[c] * r * wv * (gate_kind == 1 ? 1.f / (1.f + expf(-gv[c])) : silu_f(gv[c])));
+      const float wv = w != nullptr ? load_as_f32(w, w_dtype, w0 + 4 * lane + c) : 1.f;
+      o4[c] = from_f32<T>(xv[c] * r * wv * (first ? 1.f : gv[c]) * out_scale);
     }
     if constexpr (sizeof(T) == 4) *reinterpret_cast<float4*>(op + 4 * lane) = *reinterpret_cast<float4*>(o4);
     else *reinterpret_cast<uint2*>(op + 4 * lane) = *reinterpret_cast<uint2*>(o4);
     return;
   }
   float ss = 0.f;
-  for (int j = lane; j < V; j += 32) ss += x[j] * x[j];
+  for (int j = lane; j < V; j += 32) {
+    const float y = (den != nullptr ? x[j] / d : x[j]) * (first ? gn_act(gp[j], flags) : 1.f);
+    ss += y * y;
+  }
   ss = warp_sum(ss);
   const float r = 1.f / sqrtf(ss / (float)V + eps);
-  for (int j = lane; j < V; j += 32) op[j] = from_f32<T>(x[j] * r * (w != nullptr ? load_as_f32(w, w_dtype, j) : 1.f) * (gate_kind == 1 ? 1.f / (1.f + expf(-gp[j])) : silu_f(gp[j])));
+  for (int j = lane; j < V; j += 32)
+    op[j] = from_f32<T>((den != nullptr ? x[j] / d : x[j]) * r * (w != nullptr ? load_as_f32(w, w_dtype, w0 + j) : 1.f) *
+                        gn_act(gp[j], flags) * out_scale);
 }
 
 // The same for wide groups (all heads normed together: V in the thousands), where a warp per group would leave a
@@ -354,15 +377,22 @@ gated_rmsnorm_kernel(const float* __restrict__ o, const float* __restrict__ gate
 template <typename T>
 __global__ void __launch_bounds__(256)
 gated_rmsnorm_wide_kernel(const float* __restrict__ o, const float* __restrict__ gate, long long gate_stride,
-                          const void* __restrict__ w, int w_dtype, T* __restrict__ out, int H, int V, float eps,
-                          int gate_kind) {
+                          const void* __restrict__ w, int w_dtype, T* __restrict__ out, long long out_stride, int H, int V,
+                          float eps, int flags, const float* __restrict__ den, float out_scale) {
   bspec::pdl_prologue(62);
   __shared__ float part[8];
   const int item = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int t = item / H, h = item - t * H;
   const float* x = o + ((size_t)t * H + h) * V;
+  const float* gp = gate + (size_t)t * gate_stride + (size_t)h * V;
+  const size_t w0 = (flags & GN_FULL_WEIGHT) ? (size_t)h * V : 0;
+  const bool first = flags & GN_GATE_FIRST;
+  const float d = den != nullptr ? den[item] : 1.f;
   float ss = 0.f;
-  for (int j = threadIdx.x; j < V; j += 256) ss += x[j] * x[j];
+  for (int j = threadIdx.x; j < V; j += 256) {
+    const float y = (den != nullptr ? x[j] / d : x[j]) * (first ? gn_act(gp[j], flags) : 1.f);
+    ss += y * y;
+  }
   ss = warp_sum(ss);
   if (lane == 0) part[warp] = ss;
   __syncthreads();
@@ -370,10 +400,10 @@ gated_rmsnorm_wide_kernel(const float* __restrict__ o, const float* __restrict__
 #pragma unroll
   for (int i = 0; i < 8; ++i) tot += part[i];
   const float r = 1.f / sqrtf(tot / (float)V + eps);
-  const float* gp = gate + (size_t)t * gate_stride + (size_t)h * V;
-  T* op = out + ((size_t)t * H + h) * V;
+  T* op = out + (size_t)t * out_stride + (size_t)h * V;
   for (int j = threadIdx.x; j < V; j += 256)
-    op[j] = from_f32<T>(x[j] * r * (w != nullptr ? load_as_f32(w, w_dtype, j) : 1.f) * (gate_kind == 1 ? 1.f / (1.f + expf(-gp[j])) : silu_f(gp[j])));
+    op[j] = from_f32<T>((den != nullptr ? x[j] / d : x[j]) * r * (w != nullptr ? load_as_f32(w, w_dtype, w0 + j) : 1.f) *
+                        gn_act(gp[j], flags) * out_scale);
 }
 }  // namespace
 
@@ -419,24 +449,23 @@ BSPEC_API int bspec_delta_recurrence(const float* mix, const float* gates, const
 }
 
 BSPEC_API int bspec_gated_rmsnorm(const float* o, const float* gate, long long gate_stride, const void* w, int w_dtype,
-                                  void* out, int out_dtype, int n, int H, int V, float eps, int gate_kind,
-                                  cudaStream_t stream) {
+                                  void* out, int out_dtype, long long out_stride, int n, int H, int V, float eps, int flags,
+                                  const float* den, float out_scale, cudaStream_t stream) {
   if (n <= 0) return 0;
-  if (V >= 512) {                                            // the choice rests on the group's size alone
-    if (out_dtype == BSPEC_F32)
-      BSPEC_LAUNCH((gated_rmsnorm_wide_kernel<float>), n * H, 256, 0, stream, o, gate, gate_stride, w, w_dtype,
-                   (float*)out, H, V, eps, gate_kind);
-    else
-      BSPEC_LAUNCH((gated_rmsnorm_wide_kernel<__nv_bfloat16>), n * H, 256, 0, stream, o, gate, gate_stride, w, w_dtype,
-                   (__nv_bfloat16*)out, H, V, eps, gate_kind);
-    return BSPEC_LAUNCH_CHECK();
+  const bool wide = V >= 512;                                // the choice rests on the group's size alone
+#define GN(KERNEL, T, BLOCKS, THREADS, ...) \
+  BSPEC_LAUNCH((KERNEL<T>), BLOCKS, THREADS, 0, stream, o, gate, gate_stride, w, w_dtype, (T*)out, out_stride, __VA_ARGS__, H, V, \
+               eps, flags, den, out_scale)
+#define GNW(T) \
+  BSPEC_LAUNCH((gated_rmsnorm_wide_kernel<T>), n * H, 256, 0, stream, o, gate, gate_stride, w, w_dtype, (T*)out, out_stride, H, \
+               V, eps, flags, den, out_scale)
+  if (out_dtype == BSPEC_F32) {
+    if (wide) GNW(float); else GN(gated_rmsnorm_kernel, float, (n * H + 3) / 4, 128, n);
+  } else {
+    if (wide) GNW(__nv_bfloat16); else GN(gated_rmsnorm_kernel, __nv_bfloat16, (n * H + 3) / 4, 128, n);
   }
-  const int blocks = (n * H + 3) / 4;
-  if (out_dtype == BSPEC_F32)
-    BSPEC_LAUNCH((gated_rmsnorm_kernel<float>), blocks, 128, 0, stream, o, gate, gate_stride, w, w_dtype, (float*)out, n, H, V, eps, gate_kind);
-  else
-    BSPEC_LAUNCH((gated_rmsnorm_kernel<__nv_bfloat16>), blocks, 128, 0, stream, o, gate, gate_stride, w, w_dtype,
-                 (__nv_bfloat16*)out, n, H, V, eps, gate_kind);
+#undef GNW
+#undef GN
   return BSPEC_LAUNCH_CHECK();
 }
 

@@ -2,7 +2,7 @@
 //
 // branch_join, one block per row; every part of it is optional:
 //   y  = delta,  or the pair  delta / rms(delta) * wa + delta_b / rms(delta_b) * wb
-//   x  = src + y,  or with a weight ``post``:  src + y / rms(y) * post
+//   x  = src + extra + y,  or with a weight ``post``:  src + extra + y / rms(y) * post      (``extra``: a second branch)
 //   hist[slot] = x                                                      (``store``)
 //   x  = sum_{j < slot} coef[j] hist[j] + coef[slot] x                  (``coef``: the average over the layers so far)
 //   dst = x
@@ -23,6 +23,7 @@ struct JoinArgs {
   const int* rows;           // [n] or null
   const void* delta;         // [*, d] or null
   const void* delta_b;       // the second of a pair, or null
+  const void* extra;         // [*, d] another branch, added as it is (of delta's type), or null
   const float* wa;           // [d] weights of the pair
   const float* wb;
   const float* post;         // [d] or null
@@ -93,6 +94,12 @@ __global__ void branch_join_kernel(const JoinArgs a) {
     for (int c = 0; c < 4; ++c) x[k][c] = y[k][c] = h[DEPTH ? k : 0][c] = 0.f;
     if (i < d) {
       if (a.src != nullptr) load4<float>(a.src + base + i, x[k]);
+      if (a.extra != nullptr) {
+        float v[4];
+        load4<TD>(reinterpret_cast<const TD*>(a.extra) + base + i, v);
+#pragma unroll
+        for (int c = 0; c < 4; ++c) x[k][c] += v[c];
+      }
       if (a.delta != nullptr) load4<TD>(reinterpret_cast<const TD*>(a.delta) + base + i, y[k]);
       if (PAIR) load4<TD>(reinterpret_cast<const TD*>(a.delta_b) + base + i, z[PAIR ? k : 0]);
     }
@@ -222,7 +229,9 @@ __global__ void branch_join_any_kernel(const JoinArgs a) {
   const float rp = a.post != nullptr ? 1.f / sqrtf(sum_once(ss, scratch + 64) / (float)d + a.branch_eps) : 1.f;
   ss = 0.f;
   for (int i = threadIdx.x; i < d; i += blockDim.x) {
-    float x = (a.src != nullptr ? a.src[base + i] : 0.f) + ys[i] * rp * (a.post != nullptr ? a.post[i] : 1.f);
+    float x = a.src != nullptr ? a.src[base + i] : 0.f;
+    if (a.extra != nullptr) x += to_f32(reinterpret_cast<const TD*>(a.extra)[base + i]);
+    x += ys[i] * rp * (a.post != nullptr ? a.post[i] : 1.f);
     if (a.store) a.hist[(size_t)a.slot * a.hist_stride + base + i] = x;
     if (a.coef != nullptr) {
       float h = 0.f;
@@ -273,17 +282,17 @@ int launch_join(const JoinArgs& a, int n, cudaStream_t stream) {
 
 // Every pointer but the sizes may be null where the comment at the top calls its part optional.
 BSPEC_API int bspec_branch_join(const float* src, float* dst, const int* rows, const void* delta, const void* delta_b,
-                                int delta_dtype, const float* wa, const float* wb, const float* post,
+                                const void* extra, int delta_dtype, const float* wa, const float* wb, const float* post,
                                 float branch_eps, float* hist, long long hist_stride, int slot, int store,
                                 const float* coef, const float* norm_w, float eps, void* out, int out_dtype, int n,
                                 long long n_src, int d, cudaStream_t stream) {
   if (n <= 0) return 0;
   if (d <= 0 || slot < 0 || ((store || coef != nullptr) && hist == nullptr) ||
       (delta_b != nullptr && (delta == nullptr || wa == nullptr || wb == nullptr)) ||
-      (post != nullptr && delta == nullptr))
+      ((post != nullptr || extra != nullptr) && delta == nullptr))
     return (int)cudaErrorInvalidValue;
   JoinArgs a;
-  a.src = src; a.dst = dst; a.rows = rows; a.delta = delta; a.delta_b = delta_b; a.wa = wa; a.wb = wb; a.post = post;
+  a.src = src; a.dst = dst; a.rows = rows; a.delta = delta; a.delta_b = delta_b; a.extra = extra; a.wa = wa; a.wb = wb; a.post = post;
   a.hist = hist; a.coef = coef; a.norm_w = norm_w; a.out = out; a.hist_stride = hist_stride; a.n_src = n_src;
   a.slot = slot; a.store = store; a.d = d; a.branch_eps = branch_eps; a.eps = eps;
   if (delta_dtype == BSPEC_F32)

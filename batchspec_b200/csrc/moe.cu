@@ -16,7 +16,8 @@
 //             (act: GELU on the outputs, or none; the operand A may be gated instead: its rows are [gate | up] and
 //             silu(gate) * up is formed while they are staged, which is how gated experts run their down projection)
 //   combine   out[t, :] = add[t, :] + sum_k weight[t, k] * Y[inv[t*top + k], :], k ascending, float32 (``add``: a
-//             shared expert's rows, or none)
+//             shared expert's rows, or none, perhaps times sigmoid of a logit per token; a chosen identity expert has
+//             no row in Y, its row is the token's own input)
 //
 // Nothing here reads a count on the host: grids are sized by upper bounds and surplus blocks leave at once, so the
 // kernels can be captured in a graph.
@@ -36,7 +37,7 @@ template <typename T>
 __global__ void __launch_bounds__(ROUTE_THREADS)
 moe_route_kernel(const T* __restrict__ h, int d, const T* __restrict__ wr, const void* __restrict__ corr,
                  int corr_dtype, int E, int G, int keep, int top, float scale, int* __restrict__ ids,
-                 float* __restrict__ wts, const float* __restrict__ logits, int rule) {
+                 float* __restrict__ wts, const float* __restrict__ logits, long long ld_logits, int rule) {
   bspec::pdl_prologue(50);
   const int scores = rule & ROUTE_SCORES;
   const bool softmax_top = scores == ROUTE_SOFTMAX_TOP;
@@ -47,7 +48,7 @@ moe_route_kernel(const T* __restrict__ h, int d, const T* __restrict__ wr, const
   const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   if (logits != nullptr) {            // the logits were formed by a matrix product (many tokens)
     for (int e = threadIdx.x; e < E; e += blockDim.x) {
-      const float z = logits[(size_t)t * E + e], b = corr != nullptr ? load_as_f32(corr, corr_dtype, e) : 0.f;
+      const float z = logits[(size_t)t * ld_logits + e], b = corr != nullptr ? load_as_f32(corr, corr_dtype, e) : 0.f;
       const float s = softmax_top ? z + b : (scores == ROUTE_SOFTMAX ? z : 1.f / (1.f + expf(-z)));
       sc[e] = s;
       ch[e] = softmax_top ? s : s + b;
@@ -145,6 +146,8 @@ moe_route_kernel(const T* __restrict__ h, int d, const T* __restrict__ wr, const
   }
 }
 
+// Numbers E and above are choices without rows of their own in the grouped products (identity experts): they are sorted
+// behind all experts' rows and get no tiles.
 // One block of 1024 threads.  tiles: int [max_tiles][3] = {expert, first sorted row, rows}; n_tiles_out: int [1].
 __global__ void __launch_bounds__(1024)
 moe_plan_kernel(const int* __restrict__ ids, int slots, int E, int BM, int* __restrict__ perm, int* __restrict__ inv,
@@ -180,11 +183,11 @@ moe_plan_kernel(const int* __restrict__ ids, int slots, int E, int BM, int* __re
     *n_tiles_out = nt;
   }
   __syncthreads();
-  for (int e = warp; e < E; e += nwarps) {
+  for (int e = warp; e <= E; e += nwarps) {
     int at = cnt[e];
     for (int s0 = 0; s0 < slots; s0 += 32) {
       const int s = s0 + lane;
-      const bool mine = s < slots && ids[s] == e;
+      const bool mine = s < slots && min(ids[s], E) == e;
       const unsigned mask = __ballot_sync(0xffffffffu, mine);
       if (mine) {
         const int r = at + __popc(mask & ((1u << lane) - 1u));
@@ -200,11 +203,11 @@ moe_plan_kernel(const int* __restrict__ ids, int slots, int E, int BM, int* __re
 // their warps reach the expert's counter, so the placement (not any value: a row's result does not depend on where
 // it lies) may differ from run to run.
 __global__ void __launch_bounds__(256)
-moe_rank_kernel(const int* __restrict__ ids, int slots, int* __restrict__ counts, int* __restrict__ rank) {
+moe_rank_kernel(const int* __restrict__ ids, int slots, int E, int* __restrict__ counts, int* __restrict__ rank) {
   bspec::pdl_prologue(57);
   const int s = blockIdx.x * blockDim.x + threadIdx.x;
   const bool live = s < slots;
-  const int e = live ? ids[s] : -1;
+  const int e = live ? min(ids[s], E) : -1;
   const unsigned same = __match_any_sync(0xffffffffu, e);
   const int lane = threadIdx.x & 31;
   const int leader = __ffs(same) - 1;
@@ -239,11 +242,11 @@ __global__ void moe_offsets_kernel(const int* __restrict__ counts, int E, int BM
 
 __global__ void __launch_bounds__(256)
 moe_place_kernel(const int* __restrict__ ids, const int* __restrict__ rank, const int* __restrict__ offsets, int slots,
-                 int* __restrict__ perm, int* __restrict__ inv) {
+                 int E, int* __restrict__ perm, int* __restrict__ inv) {
   bspec::pdl_prologue(59);
   const int s = blockIdx.x * blockDim.x + threadIdx.x;
   if (s >= slots) return;
-  const int r = offsets[ids[s]] + rank[s];
+  const int r = offsets[min(ids[s], E)] + rank[s];
   perm[r] = s;
   inv[s] = r;
 }
@@ -519,27 +522,35 @@ __global__ void moe_gather_kernel(const T* __restrict__ h, const int* __restrict
   }
 }
 
+// ``ids`` (may be null): choices of E and above are identity experts, whose row is the token's own h.  ``add_gate`` (may be
+// null): one logit per token, rows of stride ld_gate; ``add`` is multiplied by its sigmoid.
 template <typename TY, typename TO>
 __global__ void moe_combine_kernel(const TY* __restrict__ y, const int* __restrict__ inv, const float* __restrict__ wts,
-                                   int top, TO* __restrict__ out, int d, const TO* __restrict__ add) {
+                                   int top, TO* __restrict__ out, int d, const TO* __restrict__ add,
+                                   const int* __restrict__ ids, int E, const TO* __restrict__ h,
+                                   const float* __restrict__ add_gate, long long ld_gate) {
   bspec::pdl_prologue(54);
   const int t = blockIdx.x;
+  const float ag = add_gate != nullptr ? 1.f / (1.f + expf(-add_gate[(size_t)t * ld_gate])) : 1.f;
   for (int i = 2 * threadIdx.x; i < d; i += 2 * blockDim.x) {
     float a0 = 0.f, a1 = 0.f;
     if (add != nullptr) {
-      a0 = to_f32(add[(size_t)t * d + i]);
-      if (i + 1 < d) a1 = to_f32(add[(size_t)t * d + i + 1]);
+      a0 = ag * to_f32(add[(size_t)t * d + i]);
+      if (i + 1 < d) a1 = ag * to_f32(add[(size_t)t * d + i + 1]);
     }
-    const bool pair = i + 1 < d && (d % 2) == 0;
     for (int k = 0; k < top; ++k) {
       const float w = wts[(size_t)t * top + k];
+      if (ids != nullptr && ids[(size_t)t * top + k] >= E) {
+        a0 += w * to_f32(h[(size_t)t * d + i]);
+        if (i + 1 < d) a1 += w * to_f32(h[(size_t)t * d + i + 1]);
+        continue;
+      }
       const TY* row = y + (size_t)inv[(size_t)t * top + k] * d + i;
       a0 += w * to_f32(row[0]);
       if (i + 1 < d) a1 += w * to_f32(row[1]);
     }
     out[(size_t)t * d + i] = from_f32<TO>(a0);
     if (i + 1 < d) out[(size_t)t * d + i + 1] = from_f32<TO>(a1);
-    (void)pair;
   }
 }
 
@@ -547,9 +558,9 @@ __global__ void moe_combine_kernel(const TY* __restrict__ y, const int* __restri
 
 BSPEC_API int bspec_moe_route(const void* h, int dtype, int n, int d, const void* wr, const void* corr, int corr_dtype,
                               int E, int G, int keep, int top, float scale, int* ids, float* wts,
-                              const float* logits, int rule, cudaStream_t stream) {
+                              const float* logits, long long ld_logits, int rule, cudaStream_t stream) {
   if (n <= 0) return 0;
-  if (E <= 0 || E > MAX_EXPERTS || top <= 0 || top > E || G <= 0 || E % G || keep <= 0 || keep > G ||
+  if ((logits != nullptr && ld_logits < E) || E <= 0 || E > MAX_EXPERTS || top <= 0 || top > E || G <= 0 || E % G || keep <= 0 || keep > G ||
       (long long)keep * (E / G) < top)
     return (int)cudaErrorInvalidValue;
   const size_t smem = (size_t)((d > 1024 ? d : 1024) + 2 * E + 8) * sizeof(float);
@@ -557,16 +568,16 @@ BSPEC_API int bspec_moe_route(const void* h, int dtype, int n, int d, const void
   if (dtype == BSPEC_F32) {
     if (smem > 48 * 1024) cudaFuncSetAttribute(moe_route_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     BSPEC_LAUNCH((moe_route_kernel<float>), n, ROUTE_THREADS, smem, stream, (const float*)h, d, (const float*)wr, corr,
-                 corr_dtype, E, G, keep, top, scale, ids, wts, logits, rule);
+                 corr_dtype, E, G, keep, top, scale, ids, wts, logits, ld_logits, rule);
   } else {
     if (smem > 48 * 1024) cudaFuncSetAttribute(moe_route_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     BSPEC_LAUNCH((moe_route_kernel<__nv_bfloat16>), n, ROUTE_THREADS, smem, stream, (const __nv_bfloat16*)h, d,
-                 (const __nv_bfloat16*)wr, corr, corr_dtype, E, G, keep, top, scale, ids, wts, logits, rule);
+                 (const __nv_bfloat16*)wr, corr, corr_dtype, E, G, keep, top, scale, ids, wts, logits, ld_logits, rule);
   }
   return BSPEC_LAUNCH_CHECK();
 }
 
-// counts [E] and rank [slots]: scratch of the many-rows path (may be null: the one-block kernel then runs).
+// counts [E + 1] and rank [slots]: scratch of the many-rows path (may be null: the one-block kernel then runs).
 BSPEC_API int bspec_moe_plan(const int* ids, int slots, int E, int BM, int* perm, int* inv, int* offsets, int* tiles,
                              int* n_tiles, int max_tiles, int* counts, int* rank, cudaStream_t stream) {
   if (slots <= 0) return 0;
@@ -575,12 +586,12 @@ BSPEC_API int bspec_moe_plan(const int* ids, int slots, int E, int BM, int* perm
     BSPEC_LAUNCH((moe_plan_kernel), 1, 1024, 0, stream, ids, slots, E, BM, perm, inv, offsets, tiles, n_tiles, max_tiles);
     return BSPEC_LAUNCH_CHECK();
   }
-  cudaError_t err = cudaMemsetAsync(counts, 0, (size_t)E * sizeof(int), stream);
+  cudaError_t err = cudaMemsetAsync(counts, 0, (size_t)(E + 1) * sizeof(int), stream);
   if (err != cudaSuccess) return (int)err;
   const int blocks = (slots + 255) / 256;
-  BSPEC_LAUNCH((moe_rank_kernel), blocks, 256, 0, stream, ids, slots, counts, rank);
+  BSPEC_LAUNCH((moe_rank_kernel), blocks, 256, 0, stream, ids, slots, E, counts, rank);
   BSPEC_LAUNCH((moe_offsets_kernel), 1, 256, 0, stream, (const int*)counts, E, BM, offsets, tiles, n_tiles, max_tiles);
-  BSPEC_LAUNCH((moe_place_kernel), blocks, 256, 0, stream, ids, (const int*)rank, (const int*)offsets, slots, perm, inv);
+  BSPEC_LAUNCH((moe_place_kernel), blocks, 256, 0, stream, ids, (const int*)rank, (const int*)offsets, slots, E, perm, inv);
   return BSPEC_LAUNCH_CHECK();
 }
 
@@ -668,10 +679,12 @@ BSPEC_API int bspec_moe_gather(const void* h, int dtype, const int* perm, int to
 }
 
 BSPEC_API int bspec_moe_combine(const void* y, int y_dtype, const int* inv, const float* wts, int top, void* out,
-                                int out_dtype, int n, int d, const void* add, cudaStream_t stream) {
+                                int out_dtype, int n, int d, const void* add, const int* ids, int E, const void* h,
+                                const float* add_gate, long long ld_gate, cudaStream_t stream) {
   if (n <= 0) return 0;
   const int threads = d >= 1024 ? 256 : 128;
-#define LC(TY, TO) BSPEC_LAUNCH((moe_combine_kernel<TY, TO>), n, threads, 0, stream, (const TY*)y, inv, wts, top, (TO*)out, d, (const TO*)add)
+#define LC(TY, TO) BSPEC_LAUNCH((moe_combine_kernel<TY, TO>), n, threads, 0, stream, (const TY*)y, inv, wts, top, (TO*)out, d, (const TO*)add, \
+                                ids, E, (const TO*)h, add_gate, ld_gate)
   if (y_dtype == BSPEC_F32 && out_dtype == BSPEC_F32) LC(float, float);
   else if (y_dtype == BSPEC_F32) LC(float, __nv_bfloat16);
   else if (out_dtype == BSPEC_F32) LC(__nv_bfloat16, float);

@@ -75,7 +75,7 @@ class DecodeGraph:
         self.dev = torch.zeros(self.total, dtype=torch.int32, device=engine.device)
         self.row_req: List[object] = [None] * B
         self.row_pages = [[0] * ng for _ in range(B)]
-        self.row_dead = [[0] * ng for _ in range(B)]       # leading table entries of the row that are -1 on the device
+        self.row_dead = [[0] * ng for _ in range(B)]       # the row's ``RequestCache.dead`` as the device's tables show it
         self.tables_dirty = True
         self.const_uploaded = False
         self.graph: Optional[torch.cuda.CUDAGraph] = None
@@ -156,7 +156,7 @@ class DecodeGraph:
                     if fresh or len(table) < have:
                         self.row_dead[i][g] = dead              # the whole table was written, -1 entries included
                 if dead > self.row_dead[i][g]:                  # pages a window or a chunk gave back turn into -1
-                    m[base + self.row_dead[i][g]:base + dead] = -1
+                    m[base + max(self.row_dead[i][g], cache.groups[g].kept_pages):base + dead] = -1
                     self.row_dead[i][g] = dead
                     self.tables_dirty = True
             self.row_req[i] = (rid, rc.serial)

@@ -53,7 +53,7 @@ _SIGNATURES = {
     "bspec_lightning_recurrence": [c_void_p, c_longlong, c_int, c_int, c_int, c_void_p, c_void_p, c_longlong, c_void_p,
                                    c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_int,
                                    c_void_p, c_void_p],
-    "bspec_branch_join": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
+    "bspec_branch_join": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
                           c_float, c_void_p, c_longlong, c_int, c_int, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int,
                           c_longlong, c_int, c_void_p],
     "bspec_pool_append": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
@@ -78,8 +78,14 @@ _SIGNATURES = {
                             c_int, c_int, c_int, c_float, c_float, c_void_p],
     "bspec_delta_recurrence": [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_longlong, c_void_p,
                                c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
-    "bspec_gated_rmsnorm": [c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int,
-                            c_float, c_int, c_void_p],
+    "bspec_gated_rmsnorm": [c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_int, c_longlong, c_int, c_int, c_int,
+                            c_float, c_int, c_void_p, c_float, c_void_p],
+    "bspec_state_space": [c_void_p, c_longlong, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p,
+                          c_longlong, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
+                          c_int, c_int, c_void_p],
+    "bspec_matrix_memory": [c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float, c_float,
+                            c_void_p, c_longlong, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
+                            c_int, c_int, c_void_p],
     "bspec_rope_kv_append": [c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p,
                              c_void_p, c_void_p, c_void_p, c_int, c_int, c_longlong, c_void_p],
     "bspec_rope_inplace": [c_void_p, c_int, c_int, c_longlong, c_int, c_int, c_void_p, c_int, c_int, c_void_p, c_float,
@@ -111,7 +117,7 @@ _SIGNATURES = {
                                    c_void_p, c_float, c_int, c_void_p, c_void_p],
     "bspec_gate_heads": [c_void_p, c_longlong, c_longlong, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
     "bspec_moe_route": [c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float,
-                        c_void_p, c_void_p, c_void_p, c_int, c_void_p],
+                        c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_void_p],
     "bspec_moe_plan": [c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
                        c_void_p, c_void_p],
     "bspec_moe_grouped": [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
@@ -121,7 +127,8 @@ _SIGNATURES = {
     "bspec_moe_skinny_mma": [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_int,
                              c_int, c_int, c_void_p],
     "bspec_moe_gather": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p],
-    "bspec_moe_combine": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p],
+    "bspec_moe_combine": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_int,
+                          c_void_p, c_void_p, c_longlong, c_void_p],
     "bspec_sgemm_tn_batched": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_longlong, c_longlong, c_longlong,
                                c_longlong, c_longlong, c_longlong, c_int, c_void_p],
     "bspec_attention_generic": [c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
@@ -219,13 +226,14 @@ def set_pdl(on: bool) -> None:
 _TRACE_SETTERS = ["bspec_trace_set_attention_tcgen05", "bspec_trace_set_elementwise", "bspec_trace_set_attention_generic", "bspec_trace_set_attention_bf16",
                   "bspec_trace_set_gemm_fp32", "bspec_trace_set_sampling", "bspec_trace_set_gemm_tcgen05", "bspec_trace_set_latent",
                   "bspec_trace_set_moe", "bspec_trace_set_latent_mma", "bspec_trace_set_delta",
-                  "bspec_trace_set_state_mixers", "bspec_trace_set_streams", "bspec_trace_set_joins"]
+                  "bspec_trace_set_state_mixers", "bspec_trace_set_streams", "bspec_trace_set_joins",
+                  "bspec_trace_set_gated_states"]
 TRACE_KERNEL_NAMES = {1: "embed", 2: "add_rmsnorm", 3: "gather_rows_add", 4: "silu_mul", 5: "rope_kv_append",
                       6: "rope_inplace", 7: "attn_generic", 8: "attn_decode", 9: "attn_prefill", 10: "sgemm",
                       11: "sample_threshold", 12: "sample_pick", 13: "sample_final", 14: "add_layernorm", 15: "clamped_glu",
                       16: "gelu_erf", 17: "tanh_softcap", 18: "residual_update", 19: "qkv_prepare", 60: "delta_prepare",
                       61: "delta_recurrence", 62: "gated_rmsnorm", 63: "bigram_add", 64: "scale", 65: "lightning_recurrence",
-                      66: "scan_conv", 67: "selective_scan", 70: "stream_expand", 71: "stream_norm", 72: "stream_gather", 73: "branch_join", 21: "pool_append", 20: "gemm_tcgen05", 30: "attn_prefill_tc", 40: "latent_prepare",
+                      66: "scan_conv", 67: "selective_scan", 70: "stream_expand", 71: "stream_norm", 72: "stream_gather", 73: "branch_join", 74: "state_space", 75: "matrix_memory", 21: "pool_append", 20: "gemm_tcgen05", 30: "attn_prefill_tc", 40: "latent_prepare",
                       41: "latent_attn_generic", 42: "gate_heads", 43: "latent_attn_mma", 44: "latent_attn_join",
                       50: "moe_route", 51: "moe_plan", 52: "moe_grouped", 53: "moe_gather", 54: "moe_combine", 55: "moe_skinny", 56: "moe_skinny_mma", 57: "moe_rank", 58: "moe_offsets", 59: "moe_place"}
 
@@ -407,6 +415,15 @@ def relu_squared_(x: torch.Tensor) -> torch.Tensor:
 
 # ---------------------------------------------------------------------------- branches that are normed before they join
 
+class BranchSum:
+    """A branch ``main`` (a tensor, or a ``NormedPair``) and another one, ``extra`` [n, d], that join the residual together:
+    both sublayers of a layer that read the same norm."""
+    __slots__ = ("main", "extra")
+
+    def __init__(self, main, extra):
+        self.main, self.extra = main, extra
+
+
 class NormedPair:
     """Two results of one sublayer, ``a / rms(a) * wa + b / rms(b) * wb``: a branch that ``branch_join`` forms while it
     joins it (rms with ``eps``; the weights float32 [d])."""
@@ -422,17 +439,21 @@ def branch_join(src: Optional[torch.Tensor], delta, dst: Optional[torch.Tensor] 
                 slot: int = 0, store: bool = False, coef: Optional[torch.Tensor] = None,
                 rows: Optional[torch.Tensor] = None) -> None:
     """One kernel for a branch's way into the float32 residual; every part is optional.  y = ``delta`` [n, d] (or a
-    ``NormedPair``); x = ``src`` + y, with ``post`` (float32 [d]) x = src + y / rms(y) * post; ``store``: hist[slot] = x;
+    ``NormedPair``; or a ``BranchSum``, whose second branch is part of ``src`` as it were); x = ``src`` + y, with ``post`` (float32 [d]) x = src + y / rms(y) * post; ``store``: hist[slot] = x;
     ``coef`` (float32 [slot + 1]): x = sum_{j < slot} coef[j] hist[j] + coef[slot] x; ``dst`` = x; ``out`` = x / rms(x) *
     norm_w, or the cast of x without ``norm_w``.  ``hist`` float32 [slots, n, d].  ``rows`` int32: block i works on row
     rows[i] of src, delta and hist and writes row i of dst and out."""
     require("joins")
+    extra = None
+    if isinstance(delta, BranchSum):
+        delta, extra = delta.main, delta.extra
     pair = delta if isinstance(delta, NormedPair) else None
     a, b = (pair.a, pair.b) if pair is not None else (delta, None)
     if pair is not None:
         assert post is None or branch_eps == pair.eps, "one eps for all norms on a branch"
         branch_eps = pair.eps
-    _require_cuda(src, a, b, dst, out, post, norm_w, hist, coef, rows)
+    _require_cuda(src, a, b, extra, dst, out, post, norm_w, hist, coef, rows)
+    assert extra is None or (extra.dtype == a.dtype and extra.shape == a.shape and extra.is_contiguous())
     like = src if src is not None else a
     n_src, d = like.shape
     n = rows.numel() if rows is not None else n_src
@@ -446,7 +467,7 @@ def branch_join(src: Optional[torch.Tensor], delta, dst: Optional[torch.Tensor] 
     assert rows is None or (rows.dtype == torch.int32 and not store and dst is not src)
     code = _dtype_code(a.dtype) if a is not None else (_dtype_code(out.dtype) if out is not None else F32)
     _check(load_library().bspec_branch_join(
-        _ptr(src), _ptr(dst), _ptr(rows), _ptr(a), _ptr(b), code, _ptr(pair.wa) if pair else None,
+        _ptr(src), _ptr(dst), _ptr(rows), _ptr(a), _ptr(b), _ptr(extra), code, _ptr(pair.wa) if pair else None,
         _ptr(pair.wb) if pair else None, _ptr(post), float(branch_eps), _ptr(hist),
         hist.stride(0) if hist is not None else 0, int(slot), int(bool(store)), _ptr(coef), _ptr(norm_w), float(eps),
         _ptr(out), _dtype_code(out.dtype) if out is not None else code, n, n_src, d, _stream()), "branch_join")
@@ -795,7 +816,8 @@ def paged_attention(qkv: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, c
     ``window`` > 0 keeps the last ``window`` keys, ``chunk`` > 0 the keys of the query's own chunk of ``chunk``
     positions (one of the two at most).  ``slopes`` (float32 per query head, with ``slopes_l2`` its ``sink_table``):
     slope * (query - key) is taken off a score.  ``pooled`` = (P, pages, tables), with a window: before the window the
-    mean key and value of every block of P tokens is seen too.  ``sink`` (float32 per query head, with ``sink_l2`` its ``sink_table``) adds
+    mean key and value of every block of P tokens is seen too; with P < 0 the request's first -P tokens (``cache`` and
+    ``tables`` once more).  ``sink`` (float32 per query head, with ``sink_l2`` its ``sink_table``) adds
     exp(sink) to the softmax denominator.  ``softcap`` c > 0 turns a scaled score s into c tanh(s / c)."""
     _require_cuda(qkv, out, cache, sink, sink_l2)
     assert qkv.stride(1) == 1 and out.is_contiguous() and out.dtype == qkv.dtype == cache.dtype
@@ -889,13 +911,14 @@ def qkv_prepare(qkv: torch.Tensor, n_heads: int, n_kv_heads: int, head_dim: int,
 
 
 def _pool_args(pooled, cache, page_size: int):
-    """(P, pages, table starts, table, number of pages) of the kernels that read or write pooled entries; their pages
-    have the layout and the number of rows of the tokens' pages."""
+    """(P, pages, table starts, table, number of pages) of the kernels that read or write what lies before a window: pooled
+    entries (P > 0; their pages have the layout and the number of rows of the tokens' pages), or the first -P tokens
+    (P < 0, with the tokens' own pages and tables)."""
     if pooled is None:
         return 0, None, None, None, 0
     pool, pages, tables = pooled
     assert pages.dtype == cache.dtype and pages.is_contiguous() and pages.shape[1:] == cache.shape[1:]
-    assert tables.page_size == page_size and pool > 0
+    assert tables.page_size == page_size and pool != 0
     return int(pool), pages.data_ptr(), tables.kv_indptr.data_ptr(), tables.kv_indices.data_ptr(), pages.shape[0]
 
 
@@ -923,7 +946,7 @@ def masked_attention(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, ct
     all numbers of a head): the output is multiplied by sigmoid(gate);
     ``out_scale`` multiplies it.  ``slopes`` (float32 per query head): slope * (query - key) is taken off a score.
     ``pooled`` = (P, pages, tables), with a window: before the window the mean key and value of every block of P tokens
-    is seen too.  ``out`` may be a view of the leading columns of wider rows.  float32 arithmetic."""
+    is seen too, or with P < 0 the request's first -P tokens.  ``out`` may be a view of the leading columns of wider rows.  float32 arithmetic."""
     _require_cuda(q, out, cache, sink, gate, slopes)
     assert slopes is None or (slopes.dtype == torch.float32 and slopes.numel() == n_heads and slopes.is_contiguous())
     assert q.stride(1) == 1 and out.stride(1) == 1 and out.dtype == q.dtype == cache.dtype
@@ -984,21 +1007,84 @@ def delta_recurrence(mix: torch.Tensor, gates: torch.Tensor, proj: torch.Tensor,
 
 
 def gated_rmsnorm(o: torch.Tensor, gate: torch.Tensor, weight: Optional[torch.Tensor], eps: float, n_heads: int, v_dim: int,
-                  out_dtype: torch.dtype, gate_act: str = "silu") -> torch.Tensor:
+                  out_dtype: torch.dtype, gate_act: str = "silu", gate_first: bool = False,
+                  den: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None, out_scale: float = 1.0) -> torch.Tensor:
     """o float32 [n, H * V]; gate a float32 view [n, H * V] of rows that may be wider.  Returns
-    o / rms_V(o) * weight * act(gate) in ``out_dtype``, act = "silu" or "sigmoid"; ``weight`` None: no weight.  With H = 1 the norm runs over the
-    whole row."""
+    o / rms_V(o) * weight * act(gate) in ``out_dtype``, act = "silu" or "sigmoid"; ``weight`` None: no weight, V numbers:
+    the same for every head, H * V numbers: one per column.  With H = 1 the norm runs over the whole row.
+    ``gate_first``: o is multiplied by act(gate) and then normed.  ``den`` (float32 [n, H]): o is divided by it first.
+    ``out``: a view [n, H * V] of rows that may be wider, which receives the result times ``out_scale``."""
     assert gate_act in ("silu", "sigmoid")
-    _require_cuda(o, gate, weight)
+    _require_cuda(o, gate, weight, den, out)
     n = o.shape[0]
     assert o.dtype == torch.float32 and o.is_contiguous() and gate.dtype == torch.float32 and gate.stride(1) == 1
-    assert gate.shape == o.shape == (n, n_heads * v_dim) and (weight is None or weight.numel() == v_dim)
-    out = torch.empty((n, n_heads * v_dim), dtype=out_dtype, device=o.device)
+    assert gate.shape == o.shape == (n, n_heads * v_dim) and (weight is None or weight.numel() in (v_dim, n_heads * v_dim))
+    assert den is None or (den.dtype == torch.float32 and den.shape == (n, n_heads) and den.is_contiguous())
+    if out is None:
+        out = torch.empty((n, n_heads * v_dim), dtype=out_dtype, device=o.device)
+    assert out.shape == o.shape and out.dtype == out_dtype and out.stride(1) == 1
+    flags = (int(gate_act == "sigmoid") + 2 * int(bool(gate_first))
+             + (4 if weight is not None and n_heads > 1 and weight.numel() == n_heads * v_dim else 0))
     _check(load_library().bspec_gated_rmsnorm(o.data_ptr(), gate.data_ptr(), gate.stride(0), _ptr(weight),
-                                              _dtype_code(weight.dtype) if weight is not None else F32, out.data_ptr(), _dtype_code(out_dtype), n,
-                                              n_heads, v_dim, float(eps), int(gate_act == "sigmoid"), _stream()),
-           "gated_rmsnorm")
+                                              _dtype_code(weight.dtype) if weight is not None else F32, out.data_ptr(), _dtype_code(out_dtype),
+                                              out.stride(0), n, n_heads, v_dim, float(eps), flags, _ptr(den),
+                                              float(out_scale), _stream()), "gated_rmsnorm")
     return out
+
+
+# ---------------------------------------------------------------------------- recurrences with gates per token and head
+
+def state_space(xbc: torch.Tensor, conv_in: torch.Tensor, dt_raw: torch.Tensor, dt_bias: torch.Tensor, rate: torch.Tensor,
+                skip: torch.Tensor, state: torch.Tensor, tail_off: int, ctx, n_heads: int, groups: int, n_state: int,
+                v_dim: int, taps: int) -> torch.Tensor:
+    """The state space recurrence with a scalar decay per head over every entry's portion (head h uses group h // (H / G)):
+    dt = softplus(dt_raw + dt_bias); S <- exp(-rate dt) S + dt B x^T; y = S^T C + skip x.  ``xbc`` float32 [n, H V + 2 G N]
+    = [x | B | C] after the convolution, ``conv_in`` a view of the same columns before it, ``dt_raw`` a view [n, H] of the
+    same rows; ``rate`` = exp(A_log), all per-head vectors float32.  ``state[slot]`` = [S as [H, V, N] | the convolution's
+    last taps-1 inputs at ``tail_off``], read and written.  Returns y float32 [n, H V]."""
+    _require_cuda(xbc, conv_in, dt_raw, dt_bias, rate, skip, state)
+    n, C = xbc.shape[0], n_heads * v_dim + 2 * groups * n_state
+    f32 = torch.float32
+    assert xbc.dtype == f32 and xbc.shape == (n, C) and xbc.stride(1) == 1 and n_heads % groups == 0 and n_state <= 256
+    assert conv_in.dtype == f32 and conv_in.shape == (n, C) and conv_in.stride(1) == 1
+    assert dt_raw.dtype == f32 and dt_raw.shape == (n, n_heads) and dt_raw.stride(0) == conv_in.stride(0)
+    assert all(v.dtype == f32 and v.numel() == n_heads and v.is_contiguous() for v in (dt_bias, rate, skip))
+    assert state.dtype == f32 and tail_off >= n_heads * v_dim * n_state and tail_off + (taps - 1) * C <= state.shape[1]
+    out = torch.empty((n, n_heads * v_dim), dtype=f32, device=xbc.device)
+    _check(load_library().bspec_state_space(
+        xbc.data_ptr(), xbc.stride(0), conv_in.data_ptr(), dt_raw.data_ptr(), conv_in.stride(0), dt_bias.data_ptr(),
+        rate.data_ptr(), skip.data_ptr(), state.data_ptr(), state.stride(0), int(tail_off), ctx.qo_indptr.data_ptr(),
+        ctx.state_slots.data_ptr(), ctx.positions.data_ptr(), out.data_ptr(), ctx.n_entries, n_heads, groups, n_state, v_dim,
+        taps, _stream()), "state_space")
+    return out
+
+
+MATRIX_MEMORY_RECORD = 6       # float32 words per head in a request's state for the running maximum
+
+
+def matrix_memory(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, i_off: int, f_off: int, i_bias: torch.Tensor,
+                  f_bias: torch.Tensor, cap: float, q_scale: float, state: torch.Tensor, m_off: int, ctx, n_heads: int,
+                  dim: int, v_dim: int):
+    """The mLSTM recurrence over every entry's portion, per head: i = cap tanh((i_raw + i_bias) / cap), f = logsigmoid(cap
+    tanh((f_raw + f_bias) / cap)), m <- max(f + m, i); S and n decay by exp(f + m_old - m) and receive exp(i - m) k v^T and
+    exp(i - m) k.  ``proj`` float32 rows with q and k (H dim each), v (H V), i and f (H each) at their offsets; q times
+    ``q_scale``.  ``state[slot]`` = [S and n as [H, V + 1, dim] | the running maximum at ``m_off``, H records], read and
+    written.  Returns (S^T q float32 [n, H V], max(|n . q|, exp(-m)) + 1e-6 float32 [n, H])."""
+    _require_cuda(proj, i_bias, f_bias, state)
+    n, ld = proj.shape
+    f32 = torch.float32
+    assert proj.dtype == f32 and proj.stride(1) == 1 and state.dtype == f32 and 0 < dim <= 256
+    assert all(v.dtype == f32 and v.numel() == n_heads and v.is_contiguous() for v in (i_bias, f_bias))
+    assert max(q_off, k_off) + n_heads * dim <= ld and v_off + n_heads * v_dim <= ld and max(i_off, f_off) + n_heads <= ld
+    assert m_off >= n_heads * (v_dim + 1) * dim and m_off + MATRIX_MEMORY_RECORD * n_heads <= state.shape[1]
+    out = torch.empty((n, n_heads * v_dim), dtype=f32, device=proj.device)
+    den = torch.empty((n, n_heads), dtype=f32, device=proj.device)
+    _check(load_library().bspec_matrix_memory(
+        proj.data_ptr(), proj.stride(0), int(q_off), int(k_off), int(v_off), int(i_off), int(f_off), i_bias.data_ptr(),
+        f_bias.data_ptr(), float(cap), float(q_scale), state.data_ptr(), state.stride(0), int(m_off), ctx.qo_indptr.data_ptr(),
+        ctx.state_slots.data_ptr(), ctx.positions.data_ptr(), out.data_ptr(), den.data_ptr(), ctx.n_entries, n_heads, dim,
+        v_dim, _stream()), "matrix_memory")
+    return out, den
 
 
 # ---------------------------------------------------------------------------- lightning attention, selective scan
@@ -1029,16 +1115,17 @@ def lightning_recurrence(proj: torch.Tensor, q_off: int, k_off: int, v_off: int,
 
 
 def scan_conv(xz: torch.Tensor, conv: torch.Tensor, bias: torch.Tensor, state: torch.Tensor, tail_off: int, ctx,
-              inner: int, taps: int, run_dtype: torch.dtype):
+              inner: int, taps: int, run_dtype: Optional[torch.dtype] = None):
     """silu(bias + causal convolution over ``taps`` inputs) of the first ``inner`` float32 columns of ``xz``, per
     channel; inputs before a portion come from ``state[slot, tail_off:]`` ([(taps-1), inner], oldest first).  Returns
-    the result as float32 [n, inner] and in ``run_dtype`` (the same tensor when that is float32)."""
+    the result as float32 [n, inner] and in ``run_dtype`` (the same tensor when that is float32 or None)."""
     _require_cuda(xz, conv, bias, state)
     n = xz.shape[0]
     assert xz.dtype == torch.float32 and xz.stride(1) == 1 and xz.shape[1] >= inner
     assert conv.shape == (inner, taps) and conv.is_contiguous() and bias.numel() == inner and conv.dtype == bias.dtype
     assert state.dtype == torch.float32 and tail_off + (taps - 1) * inner <= state.shape[1]
     xc = torch.empty((n, inner), dtype=torch.float32, device=xz.device)
+    run_dtype = run_dtype or torch.float32
     xr = xc if run_dtype == torch.float32 else torch.empty((n, inner), dtype=run_dtype, device=xz.device)
     _check(load_library().bspec_scan_conv(
         xz.data_ptr(), xz.stride(0), conv.data_ptr(), bias.data_ptr(), _dtype_code(conv.dtype), state.data_ptr(),
@@ -1414,8 +1501,10 @@ MOE_SKINNY = True                # bfloat16 steps with fewer rows per expert: th
 
 def moe_route(h: torch.Tensor, router: torch.Tensor, correction: Optional[torch.Tensor], n_groups: int, keep: int,
               top: int, scale: float, softmax_top: bool = False, softmax: bool = False, group_max: bool = False,
-              renormalise: bool = False):
+              renormalise: bool = False, extra_rows: int = 0):
     """(expert ids int32 [n, top], weights float32 [n, top]) of every token; the rule is in ``csrc/moe.cu``.
+    ``extra_rows``: the last rows of ``router`` are no experts; their logits come back as a third result, a float32 view
+    [n, extra_rows].
     ``softmax_top``: the logits plus ``correction`` (a bias) choose, and the weights are the softmax over the chosen
     logits alone; ``softmax``: the scores are the softmax over all experts; otherwise sigmoid scores.  ``group_max``: a
     group's score is its largest choice instead of the sum of its two largest.  ``renormalise``: the weights are the
@@ -1424,29 +1513,34 @@ def moe_route(h: torch.Tensor, router: torch.Tensor, correction: Optional[torch.
     rule = (1 if softmax_top else 2 if softmax else 0) + (4 if group_max else 0) + (8 if renormalise else 0)
     _require_cuda(h, router)
     n, d = h.shape
-    E = router.shape[0]
-    assert router.shape == (E, d) and router.dtype == h.dtype and h.is_contiguous() and router.is_contiguous()
+    E = router.shape[0] - int(extra_rows)
+    assert router.shape[1] == d and router.dtype == h.dtype and h.is_contiguous() and router.is_contiguous()
     ids = torch.empty((n, top), dtype=torch.int32, device=h.device)
     wts = torch.empty((n, top), dtype=torch.float32, device=h.device)
     # many tokens: the logits as one matrix product with float32 accumulation and output; few: inside the kernel
-    logits = linear(h, router, out_dtype=torch.float32) if n > MOE_ROUTE_FUSED_MAX else None
+    logits = linear(h, router, out_dtype=torch.float32) if n > MOE_ROUTE_FUSED_MAX or extra_rows else None
     _check(load_library().bspec_moe_route(h.data_ptr(), _dtype_code(h.dtype), n, d, router.data_ptr(), _ptr(correction),
                                           _dtype_code(correction.dtype) if correction is not None else F32, E,
                                           int(n_groups), int(keep), int(top), float(scale), ids.data_ptr(),
-                                          wts.data_ptr(), _ptr(logits), rule, _stream()), "moe_route")
-    return ids, wts
+                                          wts.data_ptr(), _ptr(logits), router.shape[0], rule, _stream()), "moe_route")
+    return (ids, wts, logits[:, E:]) if extra_rows else (ids, wts)
 
 
 def moe_experts(h: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor,
-                out_dtype: torch.dtype, glu: bool = False, add: Optional[torch.Tensor] = None) -> torch.Tensor:
+                out_dtype: torch.dtype, glu: bool = False, add: Optional[torch.Tensor] = None,
+                add_gate: Optional[torch.Tensor] = None, identity: bool = False) -> torch.Tensor:
     """sum_k wts[t, k] * Wdown[e] gelu(Wup[e] h[t]) with e = ids[t, k].  ``w_up`` [E, ff, d], ``w_down`` [E, d, ff].
     ``glu``: the experts are gated, Wdown[e] (silu(Wgate[e] h) * (Wup[e] h)), and ``w_up`` holds [gate; up] as
     [E, 2 ff, d]; the first product then leaves its result as it is, and this package's grouped kernels form
     silu(gate) * up while they stage the rows of the second product (the vendor's grouped product is followed by
     ``silu_mul`` instead).
-    ``add`` [n, d] in ``out_dtype`` (a shared expert's result) is added to the sum.
+    ``add`` [n, d] in ``out_dtype`` (a shared expert's result) is added to the sum, times the sigmoid of ``add_gate`` (a
+    float32 view [n, 1] of rows that may be wider) when given.  ``identity``: numbers of E and above may be chosen; such an
+    expert's result is h[t] itself (they are sorted behind the others' rows and take part in no product).
     The (token, choice) rows are sorted by expert on the device; no count is read on the host."""
     assert add is None or (add.shape == h.shape and add.dtype == out_dtype and add.is_contiguous())
+    assert add_gate is None or (add is not None and add_gate.dtype == torch.float32 and add_gate.shape == (h.shape[0], 1))
+    assert not identity or h.dtype == out_dtype
     _require_cuda(h, ids, wts, w_up, w_down)
     lib = load_library()
     n, d = h.shape
@@ -1479,13 +1573,13 @@ def moe_experts(h: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, w_up: tor
     BM = (mma_rows if skinny_mma else 8) if skinny else (64 if slots >= 32 * E else 16)
     max_tiles = min(slots, slots // BM + E)
     many = slots > 2048                   # the plan in three kernels over all SMs (needs counters and ranks)
-    meta = torch.empty((2 * slots + E + 1 + 3 * max_tiles + 1 + (E + slots if many else 0),), dtype=torch.int32, device=dev)
+    meta = torch.empty((2 * slots + E + 1 + 3 * max_tiles + 1 + (E + 1 + slots if many else 0),), dtype=torch.int32, device=dev)
     perm, inv = meta[:slots], meta[slots:2 * slots]
     offsets = meta[2 * slots:2 * slots + E + 1]
     tiles = meta[2 * slots + E + 1:2 * slots + E + 1 + 3 * max_tiles]
     at = 2 * slots + E + 1 + 3 * max_tiles
     n_tiles = meta[at:at + 1]
-    counts, rank = (meta[at + 1:at + 1 + E], meta[at + 1 + E:]) if many else (None, None)
+    counts, rank = (meta[at + 1:at + 2 + E], meta[at + 2 + E:]) if many else (None, None)
     _check(lib.bspec_moe_plan(ids.data_ptr(), slots, E, BM, perm.data_ptr(), inv.data_ptr(), offsets.data_ptr(),
                               tiles.data_ptr(), n_tiles.data_ptr(), max_tiles, _ptr(counts), _ptr(rank), _stream()),
            "moe_plan")
@@ -1524,7 +1618,9 @@ def moe_experts(h: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, w_up: tor
                "moe_grouped_down")
     out = torch.empty((n, d), dtype=out_dtype, device=dev)
     _check(lib.bspec_moe_combine(y.data_ptr(), _dtype_code(y.dtype), inv.data_ptr(), wts.data_ptr(), top,
-                                 out.data_ptr(), _dtype_code(out_dtype), n, d, _ptr(add), _stream()), "moe_combine")
+                                 out.data_ptr(), _dtype_code(out_dtype), n, d, _ptr(add), ids.data_ptr() if identity else None,
+                                 E, h.data_ptr() if identity else None, _ptr(add_gate),
+                                 add_gate.stride(0) if add_gate is not None else 0, _stream()), "moe_combine")
     return out
 
 

@@ -11,6 +11,7 @@ from typing import Callable, Dict
 from ..parts.base import Runtime
 from .decoder import CacheNeed, DecoderModel, LayerCache
 from .finolix import build_finolix
+from .guvolix import build_guvolix
 from .llama import build_llama
 from .lupusun import build_lupusun
 from .podizen import build_podizen
@@ -38,6 +39,7 @@ register_model("Lupusun", build_lupusun)
 register_model("Tokolorn", build_tokolorn)
 register_model("Finolix", build_finolix)
 register_model("Podizen", build_podizen)
+register_model("Guvolix", build_guvolix)
 
 __all__ = ["MODEL_REGISTRY", "register_model", "get_model", "DecoderModel", "LayerCache", "CacheNeed",
-           "ModelSpec", "LayerSpec", "RunEntry", "prenorm_layer", "build_finolix", "build_llama", "build_lupusun", "build_podizen", "build_tokolorn", "build_vabanex"]
+           "ModelSpec", "LayerSpec", "RunEntry", "prenorm_layer", "build_finolix", "build_guvolix", "build_llama", "build_lupusun", "build_podizen", "build_tokolorn", "build_vabanex"]

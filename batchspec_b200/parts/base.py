@@ -61,13 +61,16 @@ class CacheSpec:
     ``pool`` P > 0: besides, every whole block of P tokens has one more entry of the
     same shape, which is kept while the request lives.  These entries have a group of
     their own (pages of as many entries, a block table: entry b is block b), and a
-    windowed group keeps the tokens of the block that is not yet whole."""
+    windowed group keeps the tokens of the block that is not yet whole.
+    ``keep``: with policy ``window``, the request's first ``keep`` tokens are read however far the window has moved;
+    their pages are not given back."""
     policy: str
     entry_shape: Tuple[int, ...]
     window: Optional[int] = None
     tensors: int = 2
     page_size: Optional[int] = None
     pool: int = 0
+    keep: int = 0
 
 
 @dataclass(frozen=True)

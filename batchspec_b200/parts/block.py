@@ -166,6 +166,31 @@ class HyperPreNormMixerBlock(Block):
         return resid, self.mixer.forward(a, ctx, cache)
 
 
+class _Parallel(Block):
+    """Both sublayers of a layer read the same norm and join the residual together: x' = x + (mixer(n) + ffn(n)), n =
+    norm1(x).  The two results go on unsummed (``ops.BranchSum``); the kernel of the next norm adds both in float32.  A
+    mixer that offers ``forward_branches`` (its result as a pair that the join forms) is asked for that."""
+
+    residual_join = BranchJoin()
+
+    def forward(self, resid, pending, ctx, cache, pending_scale: float = 1.0, pending_join=None):
+        assert pending_scale == 1.0
+        a = self.norm1.forward_join(resid, pending, pending_join)
+        y = (getattr(self.mixer, "forward_branches", None) or self.mixer.forward)(a, ctx, cache)
+        return resid, (ops.BranchSum(y, self.ffn.forward(a, ctx)) if "ffn" in self.parts else y)
+
+
+@register_part(BLOCKS, "parallel_prenorm")
+class ParallelBlock(_Parallel):
+    SLOTS = {"norm1": NORMS, "mixer": MIXERS, "ffn": FEED_FORWARDS}
+
+
+@register_part(BLOCKS, "parallel_prenorm_mixer")
+class ParallelMixerBlock(_Parallel):
+    """The same without a feed-forward."""
+    SLOTS = {"norm1": NORMS, "mixer": MIXERS}
+
+
 @register_part(DEPTH_AVERAGES, "learned")
 class LearnedDepthAverage(Part):
     """The average over depth after a layer: sum over i < ``count`` of w[i] X_i, X_0 the input of the first layer and the

@@ -16,6 +16,7 @@
 * ``pool`` P, with a window W: the positions are cut into blocks of P from 0 on, and query i also attends, in the same
   softmax, to one entry per block whose last position is at most i - W: the mean of the block's cached keys with the
   mean of its values.  A token between its window and its block's turn has no influence;
+* ``keep_first`` K, with a window: the request's first K tokens stay visible when the window has passed them;
 * ``values_are_keys``: there is no value projection, a key as projected is its own value, and only keys are cached;
 * ``gate``: the concatenated heads are multiplied element by element by sigmoid(Wg h) before the output projection;
   ``gate="head"``: Wg has one row per head and the head's whole output is multiplied by one number.
@@ -55,7 +56,7 @@ class SinkAttention(Mixer):
                  sink: bool = False, fixed_sink: Optional[float] = None, softcap: Optional[float] = None,
                  values_are_keys: bool = False, gate=False, qk_norm_weight: bool = False,
                  qk_norm_first: bool = False, bias_slopes: Optional[Sequence[float]] = None,
-                 pool: Optional[int] = None):
+                 pool: Optional[int] = None, keep_first: Optional[int] = None):
         if n_heads <= 0 or n_kv_heads <= 0 or n_heads % n_kv_heads:
             raise ValueError(f"n_heads {n_heads} must be a positive multiple of n_kv_heads {n_kv_heads}")
         self.runtime = runtime
@@ -82,6 +83,9 @@ class SinkAttention(Mixer):
         self.pool = int(pool) if pool else 0
         if self.pool < 0 or (self.pool and (not self.window or self.values_are_keys)):
             raise ValueError("pooled blocks need a window before which they lie, and values of their own")
+        self.keep = int(keep_first) if keep_first and self.window else 0      # without a window every token is seen anyway
+        if self.keep < 0 or (self.keep and self.pool):
+            raise ValueError("first tokens that stay visible are counted, and not beside pooled blocks")
         if bias_slopes is not None and len(bias_slopes) != self.n_heads:
             raise ValueError(f"{n_heads} heads need {n_heads} slopes, got {len(bias_slopes)}")
         self.slopes = None if bias_slopes is None else torch.tensor([float(x) for x in bias_slopes], dtype=torch.float32,
@@ -135,7 +139,8 @@ class SinkAttention(Mixer):
             self.sinks_l2 = ops.sink_table(self.sinks)
 
     def _tensor_cores(self, dtype) -> bool:
-        return dtype == torch.bfloat16 and self.v_dim == self.head_dim and self.head_dim in (64, 128, 256)
+        return (dtype == torch.bfloat16 and self.v_dim == self.head_dim and self.head_dim in (64, 128, 256)
+                and not (self.keep and self.slopes is not None))
 
     @property
     def out_width(self) -> int:
@@ -147,10 +152,10 @@ class SinkAttention(Mixer):
         span = self.chunk or self.window or None
         pool = self.pool
         if self.values_are_keys and not self.copy_keys:
-            return CacheSpec(policy, (self.n_kv_heads * self.head_dim,), span, tensors=1)
+            return CacheSpec(policy, (self.n_kv_heads * self.head_dim,), span, tensors=1, keep=self.keep)
         if self.v_dim == self.head_dim:
-            return CacheSpec(policy, (self.n_kv_heads, self.head_dim), span, pool=pool)
-        return CacheSpec(policy, (self.n_kv_heads * (self.head_dim + self.v_dim),), span, tensors=1, pool=pool)
+            return CacheSpec(policy, (self.n_kv_heads, self.head_dim), span, pool=pool, keep=self.keep)
+        return CacheSpec(policy, (self.n_kv_heads * (self.head_dim + self.v_dim),), span, tensors=1, pool=pool, keep=self.keep)
 
     def forward(self, x, ctx, cache):
         out = self.pre_projection(x, ctx, cache)
@@ -165,6 +170,7 @@ class SinkAttention(Mixer):
         tables = ctx.tables[cache.group]
         pos = self.position
         pooled = (self.pool, cache.pooled, ctx.tables[cache.pooled_group]) if self.pool else None
+        before = (-self.keep, cache.kv, tables) if self.keep else pooled         # what is seen before the window
         one_each = ctx.max_q_len == 1             # a token that completes a block finds the block's others in the cache
         with bucket("attn.qkv_proj"):
             proj = ops.linear(x, self.wqkv, out_dtype=torch.float32)
@@ -190,7 +196,7 @@ class SinkAttention(Mixer):
                 direct = not self.gate and out_scale == 1.0 and out.is_contiguous()
                 heads = out if direct else torch.empty((n, H * vd), dtype=x.dtype, device=x.device)
                 ops.paged_attention(q, heads, cache.kv, ctx, tables, H, G, hd, self.scale, self.window, self.chunk,
-                                    self.sinks, self.sinks_l2, self.softcap, self.slopes, self.slopes_l2, pooled)
+                                    self.sinks, self.sinks_l2, self.softcap, self.slopes, self.slopes_l2, before)
                 if not direct and self.gate_per_head and out_scale == 1.0 and out.is_contiguous():
                     # one logit per head: the heads [n, H * vd] read as [H, n, vd]
                     ops.gate_heads(heads.view(n, H, vd).transpose(0, 1), gate, out)
@@ -201,5 +207,5 @@ class SinkAttention(Mixer):
             else:
                 ops.masked_attention(q, out, cache.kv, ctx, tables, H, G, hd, vd, self.scale, self.window, self.chunk,
                                      self.sinks, self.softcap, self.values_are_keys and not self.copy_keys, gate,
-                                     out_scale, gate_per_head=self.gate_per_head, slopes=self.slopes, pooled=pooled)
+                                     out_scale, gate_per_head=self.gate_per_head, slopes=self.slopes, pooled=before)
         return out
