@@ -49,7 +49,7 @@ struct GemmParams {
                          // 1: silu(gate) * up;  2: g sigmoid(alpha g) (u + 1), g = min(gate, limit), u = clamp(up, +-limit);
                          // 3: relu(gate) * up
   float glu_alpha, glu_limit;
-  int act;               // a plain activation on every output (no gate): 0 none, 1 the square of relu
+  int act;               // a plain activation on every output (no gate): 0 none, 1 the square of relu, 2 the exact gelu
   int prefetch_kb;       // K blocks of weights (beyond the stages) to pull into the L2 before waiting on the predecessor
   // fused q/k/v projection (rope_freq != nullptr): tile t of W is head t (q heads, then k heads, then v heads)
   const float* rope_freq;    // [2][64] frequencies as two floats each (see elementwise.cu, rope_sincos)
@@ -90,6 +90,7 @@ __device__ __forceinline__ float glu_combine(int kind, float alpha, float limit,
 // A plain activation on one output (GemmParams::act).
 __device__ __forceinline__ float unary_act(int kind, float x) {
   if (kind == 1) { const float r = fmaxf(x, 0.f); return r * r; }
+  if (kind == 2) return 0.5f * x * (1.f + erff(x * 0.70710678118654752440f));
   return x;
 }
 
@@ -531,10 +532,10 @@ BSPEC_API int bspec_gemm_tc(const void* X, const void* W, void* C, int M, int N,
   return launch_gemm(X, W, C, M, N, K, out_f32, glu, status, sm_count, nullptr, stream);
 }
 
-// C = act(X W^T) with a plain activation on every output: act 1 = the square of relu.
+// C = act(X W^T) with a plain activation on every output: act 1 = the square of relu, 2 = the exact (erf) gelu.
 BSPEC_API int bspec_gemm_tc_act(const void* X, const void* W, void* C, int M, int N, int K, int out_f32, int act,
                                 int* status, int sm_count, cudaStream_t stream) {
-  if (act != 1) return (int)cudaErrorInvalidValue;
+  if (act != 1 && act != 2) return (int)cudaErrorInvalidValue;
   return launch_gemm(X, W, C, M, N, K, out_f32, 0, status, sm_count, nullptr, stream, 1.f, 0.f, act);
 }
 

@@ -1306,7 +1306,7 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype) -> torch.T
     return out
 
 
-PLAIN_ACTIVATIONS = {"relu2": (1, relu_squared_), "gelu": (0, gelu_erf_)}     # epilogue kind (0: none), in-place kernel
+PLAIN_ACTIVATIONS = {"relu2": (1, relu_squared_), "gelu": (2, gelu_erf_)}     # epilogue kind (0: none), in-place kernel
 
 
 def linear_act(x: torch.Tensor, w: torch.Tensor, activation: str) -> torch.Tensor:

@@ -99,8 +99,8 @@ class ClampedGLU(FeedForward):
 @register_part(FEED_FORWARDS, "mlp")
 class PlainMLP(FeedForward):
     """Two matrices and an activation between them: out = Wdown act(Wup x), no gate and no biases.
-    ``activation``: "relu2" (the square of relu) or "gelu" (the exact one).  Decode-sized bfloat16 steps apply the
-    square of relu in the first product's epilogue."""
+    ``activation``: "relu2" (the square of relu) or "gelu" (the exact one).  Decode-sized bfloat16 steps apply it in
+    the first product's epilogue."""
     graph_safe = True
     ACTIVATIONS = ops.PLAIN_ACTIVATIONS
 
