@@ -371,6 +371,61 @@ gated_rmsnorm_kernel(const float* __restrict__ o, const float* __restrict__ gate
                         gn_act(gp[j], flags) * out_scale);
 }
 
+// The same for groups of 4 K numbers on 16-byte boundaries, a block per (token, group) and QPT quads per thread: every
+// number is read once and waits in registers between the sum of squares and the result.
+template <typename T, int QPT>
+__global__ void gated_rmsnorm_quads_kernel(const float* __restrict__ o, const float* __restrict__ gate, long long gate_stride,
+                                           const void* __restrict__ w, int w_dtype, T* __restrict__ out,
+                                           long long out_stride, int H, int V, float eps, int flags,
+                                           const float* __restrict__ den, float out_scale) {
+  bspec::pdl_prologue(62);
+  __shared__ float part[32];
+  const int item = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
+  const int t = item / H, h = item - t * H;
+  const float* x = o + (size_t)item * V;
+  const float* gp = gate + (size_t)t * gate_stride + (size_t)h * V;
+  const size_t w0 = (flags & GN_FULL_WEIGHT) ? (size_t)h * V : 0;
+  const bool first = flags & GN_GATE_FIRST;
+  const float d = den != nullptr ? 1.f / den[item] : 1.f;
+  float y[QPT][4], a[QPT][4];
+  float ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < QPT; ++k) {
+    const int j = 4 * (threadIdx.x + k * blockDim.x);
+    const bool in = j < V;
+    const float4 xv = in ? *reinterpret_cast<const float4*>(x + j) : make_float4(0.f, 0.f, 0.f, 0.f);
+    const float4 gv = in ? *reinterpret_cast<const float4*>(gp + j) : make_float4(0.f, 0.f, 0.f, 0.f);
+    const float xs[4] = {xv.x, xv.y, xv.z, xv.w}, gs[4] = {gv.x, gv.y, gv.z, gv.w};
+#pragma unroll
+    for (int c = 0; c < 4; ++c) {
+      a[k][c] = gn_act(gs[c], flags);
+      y[k][c] = xs[c] * d * (first ? a[k][c] : 1.f);
+      ss += y[k][c] * y[k][c];
+    }
+  }
+  ss = warp_sum(ss);
+  if (warps > 1) {
+    if (lane == 0) part[warp] = ss;
+    __syncthreads();
+    ss = warp_sum(lane < warps ? part[lane] : 0.f);
+  }
+  const float r = out_scale / sqrtf(ss / (float)V + eps);
+  T* op = out + (size_t)t * out_stride + (size_t)h * V;
+#pragma unroll
+  for (int k = 0; k < QPT; ++k) {
+    const int j = 4 * (threadIdx.x + k * blockDim.x);
+    if (j >= V) break;
+    T o4[4];
+#pragma unroll
+    for (int c = 0; c < 4; ++c) {
+      const float wv = w != nullptr ? load_as_f32(w, w_dtype, w0 + j + c) : 1.f;
+      o4[c] = from_f32<T>(y[k][c] * r * wv * (first ? 1.f : a[k][c]));
+    }
+    if constexpr (sizeof(T) == 4) *reinterpret_cast<float4*>(op + j) = *reinterpret_cast<float4*>(o4);
+    else *reinterpret_cast<uint2*>(op + j) = *reinterpret_cast<uint2*>(o4);
+  }
+}
+
 // The same for wide groups (all heads normed together: V in the thousands), where a warp per group would leave a
 // decode step on a handful of warps: a block of 256 threads per (token, group), the sum of squares joined through
 // shared memory in a fixed order.
@@ -452,7 +507,21 @@ BSPEC_API int bspec_gated_rmsnorm(const float* o, const float* gate, long long g
                                   void* out, int out_dtype, long long out_stride, int n, int H, int V, float eps, int flags,
                                   const float* den, float out_scale, cudaStream_t stream) {
   if (n <= 0) return 0;
-  const bool wide = V >= 512;                                // the choice rests on the group's size alone
+  const bool wide = V >= 512;                                // the choice rests on the group's size (and the boundaries) alone
+  const int esize = out_dtype == BSPEC_F32 ? 4 : 2;
+  if (V % 4 == 0 && V > 128 && V <= 16384 && gate_stride % 4 == 0 && out_stride % 4 == 0 &&
+      ((reinterpret_cast<uintptr_t>(o) | reinterpret_cast<uintptr_t>(gate)) & 15) == 0 &&
+      (reinterpret_cast<uintptr_t>(out) & (4 * esize - 1)) == 0) {
+    const int quads = V / 4, qpt = quads <= 256 ? 1 : (quads <= 1024 ? 2 : 4);
+    const int threads = ((quads + qpt - 1) / qpt + 31) / 32 * 32;
+#define GQ(T, Q) BSPEC_LAUNCH((gated_rmsnorm_quads_kernel<T, Q>), n * H, threads, 0, stream, o, gate, gate_stride, w, w_dtype, \
+                              (T*)out, out_stride, H, V, eps, flags, den, out_scale)
+#define GQT(T) do { if (qpt == 1) GQ(T, 1); else if (qpt == 2) GQ(T, 2); else GQ(T, 4); } while (0)
+    if (out_dtype == BSPEC_F32) GQT(float); else GQT(__nv_bfloat16);
+#undef GQT
+#undef GQ
+    return BSPEC_LAUNCH_CHECK();
+  }
 #define GN(KERNEL, T, BLOCKS, THREADS, ...) \
   BSPEC_LAUNCH((KERNEL<T>), BLOCKS, THREADS, 0, stream, o, gate, gate_stride, w, w_dtype, (T*)out, out_stride, __VA_ARGS__, H, V, \
                eps, flags, den, out_scale)

@@ -21,6 +21,20 @@ namespace {
 
 __device__ __forceinline__ float softplus_f(float x) { return x > 20.f ? x : log1pf(expf(x)); }
 
+// m <- max(f + m, i), m kept as a pair (leading part, remainder) so that many small f can be added to an m of some units;
+// x = f + m_old - m and b = i - m are the logs of the decay and of the input's strength.
+__device__ __forceinline__ void advance_maximum(float& m_hi, float& m_lo, float i, float f, float& x, float& b) {
+  const float s = __fadd_rn(m_hi, f), z = __fsub_rn(s, m_hi);
+  const float err = __fadd_rn(__fadd_rn(__fsub_rn(m_hi, __fsub_rn(s, z)), __fsub_rn(f, z)), m_lo);
+  const float hi = __fadd_rn(s, err), lo = __fsub_rn(err, __fsub_rn(hi, s));
+  const float d = __fsub_rn(__fsub_rn(i, hi), lo);           // i - (f + m)
+  const bool up = d > 0.f;
+  m_hi = up ? i : hi;
+  m_lo = up ? 0.f : lo;
+  x = up ? -d : 0.f;
+  b = up ? 0.f : d;
+}
+
 // A block of COLS value columns of one head, L lanes per column (8, 16 or 32); lane r of a column keeps rows
 // 4 L g + 4 r + e (e < 4, g < NR / 4) of that column of S in registers.  Tokens are staged TT at a time in shared
 // memory, the next TT tokens' rows being fetched into registers while the recurrence runs over the current ones.  One
@@ -108,16 +122,11 @@ gated_state_kernel(const GatedStateArgs a) {
       for (int t = 0; t < GS_TT; ++t) {
         const float it = __shfl_sync(0xffffffffu, i_log, t), ft = __shfl_sync(0xffffffffu, f_log, t);
         if (t >= cnt) break;
-        // f + m as a pair: many small f are added to an m of some units
-        const float s = __fadd_rn(m_hi, ft), z = __fsub_rn(s, m_hi);
-        const float err = __fadd_rn(__fadd_rn(__fsub_rn(m_hi, __fsub_rn(s, z)), __fsub_rn(ft, z)), m_lo);
-        const float hi = __fadd_rn(s, err), lo = __fsub_rn(err, __fsub_rn(hi, s));
-        const float d = __fsub_rn(__fsub_rn(it, hi), lo);    // i - (f + m)
-        m_hi = d > 0.f ? it : hi;
-        m_lo = d > 0.f ? 0.f : lo;
+        float xt, bt;
+        advance_maximum(m_hi, m_lo, it, ft, xt, bt);
         if (lane == t) {
-          x = d > 0.f ? -d : 0.f;
-          b_log = d > 0.f ? 0.f : d;
+          x = xt;
+          b_log = bt;
           m = m_hi;
         }
       }
@@ -294,13 +303,140 @@ gated_state_kernel(const GatedStateArgs a) {
   }
 }
 
+// A step in which every portion is one token (decoding): bound by reading and writing the state once.  Nothing is staged:
+// LPC lanes share a value column of QPL x 4 LPC rows, a warp takes several columns at a time whose loads are all in flight
+// together, and every warp forms its head's gates itself.  The state was last written by an earlier step, so its loads are
+// issued before the wait on the kernel before this one (which writes q, k, v and the gates).
+constexpr int GD_WARPS = 4;
+
+template <int KIND, int LPC, int QPL, int CPL>             // CPL: columns per lane group
+__global__ void __launch_bounds__(GD_WARPS * 32)
+gated_state_decode_kernel(const GatedStateArgs a) {
+  const unsigned long long t_trace = bspec::g_trace_buf != nullptr ? bspec::global_timer() : 0ull;
+  bspec::pdl_launch_dependents();
+  constexpr int GROUPS = 32 / LPC;                           // lane groups of a warp
+  const int e = blockIdx.z, h = blockIdx.y, H = a.H, dim = a.dim, vdim = a.vdim;
+  const int columns = vdim + (KIND == MATRIX_MEMORY ? 1 : 0);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, grp = lane / LPC, r = lane % LPC;
+  const int t = a.qo_indptr[e];
+  float* row = a.state + (size_t)a.state_slots[e] * a.state_stride;
+  const int j0 = (blockIdx.x * GD_WARPS + warp) * GROUPS * CPL + grp;          // the group's columns: j0, j0 + GROUPS, ...
+  float4 s[CPL][QPL];
+#pragma unroll
+  for (int c = 0; c < CPL; ++c) {
+    const int j = j0 + c * GROUPS;
+    const float* sp = row + ((size_t)h * columns + j) * dim;
+#pragma unroll
+    for (int k = 0; k < QPL; ++k) {
+      const int i = 4 * (r + k * LPC);
+      s[c][k] = j < columns && i < dim ? *reinterpret_cast<const float4*>(sp + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+  }
+  bspec::pdl_wait();
+  bspec::trace_record(KIND == STATE_SPACE ? 74 : 75, t_trace);
+  float4 q[QPL], k4[QPL];
+  const size_t at = (size_t)t * a.ld_qkv + (size_t)(h / a.rep) * dim;
+#pragma unroll
+  for (int k = 0; k < QPL; ++k) {
+    const int i = 4 * (r + k * LPC);
+    q[k] = k4[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (i < dim) {
+      q[k] = *reinterpret_cast<const float4*>(a.q + at + i);
+      k4[k] = *reinterpret_cast<const float4*>(a.k + at + i);
+    }
+    q[k].x *= a.q_scale; q[k].y *= a.q_scale; q[k].z *= a.q_scale; q[k].w *= a.q_scale;
+  }
+  float v[CPL];
+#pragma unroll
+  for (int c = 0; c < CPL; ++c) {
+    const int j = j0 + c * GROUPS;
+    v[c] = j < vdim ? a.v[(size_t)t * a.ld_qkv + (size_t)h * vdim + j] : (j == vdim ? 1.f : 0.f);
+  }
+  float em1, b, exp_m = 0.f;
+  const float raw = a.g0[(size_t)t * a.ld_g + h];
+  if constexpr (KIND == STATE_SPACE) {
+    b = softplus_f(raw + a.p0[h]);
+    em1 = expm1f(-a.p1[h] * b);
+  } else {
+    const float* rec = row + a.aux_off + (size_t)h * M_WORDS;
+    const int pos = a.positions[t], use = __float_as_int(rec[2]) == pos ? 0 : 1;
+    float m_hi = rec[3 * use], m_lo = rec[3 * use + 1], x, b_log;
+    const float i_log = a.cap * tanhf((raw + a.p0[h]) / a.cap);
+    const float f_log = -softplus_f(-a.cap * tanhf((a.g1[(size_t)t * a.ld_g + h] + a.p1[h]) / a.cap));
+    advance_maximum(m_hi, m_lo, i_log, f_log, x, b_log);
+    em1 = expm1f(x);
+    b = expf(b_log);
+    exp_m = expf(-m_hi);
+    if (blockIdx.x == 0 && threadIdx.x == 0) {               // the other record: nobody reads it as this position's
+      float* to = row + a.aux_off + (size_t)h * M_WORDS + 3 * (1 - use);
+      to[0] = m_hi;
+      to[1] = m_lo;
+      to[2] = __int_as_float(pos + 1);
+    }
+  }
+  if (KIND == STATE_SPACE && a.taps > 1) {                   // the convolution's inputs move on by one
+    float* tail = row + a.aux_off;
+    const int C = a.channels, share = blockIdx.y * gridDim.x + blockIdx.x, shares = gridDim.y * gridDim.x;
+    for (int c = share * (GD_WARPS * 32) + threadIdx.x; c < C; c += shares * (GD_WARPS * 32)) {
+      for (int u = 0; u < a.taps - 2; ++u) tail[(size_t)u * C + c] = tail[(size_t)(u + 1) * C + c];
+      tail[(size_t)(a.taps - 2) * C + c] = a.conv_in[(size_t)t * a.ld_conv + c];
+    }
+  }
+  float acc[CPL];
+#pragma unroll
+  for (int c = 0; c < CPL; ++c) {
+    const int j = j0 + c * GROUPS;
+    const float bv = __fmul_rn(b, v[c]);
+    float* sp = row + ((size_t)h * columns + j) * dim;
+    acc[c] = 0.f;
+#pragma unroll
+    for (int k = 0; k < QPL; ++k) {
+      float4& x = s[c][k];
+      x.x = __fadd_rn(x.x, __fmaf_rn(em1, x.x, __fmul_rn(k4[k].x, bv)));
+      x.y = __fadd_rn(x.y, __fmaf_rn(em1, x.y, __fmul_rn(k4[k].y, bv)));
+      x.z = __fadd_rn(x.z, __fmaf_rn(em1, x.z, __fmul_rn(k4[k].z, bv)));
+      x.w = __fadd_rn(x.w, __fmaf_rn(em1, x.w, __fmul_rn(k4[k].w, bv)));
+      acc[c] = __fmaf_rn(x.x, q[k].x, acc[c]);
+      acc[c] = __fmaf_rn(x.y, q[k].y, acc[c]);
+      acc[c] = __fmaf_rn(x.z, q[k].z, acc[c]);
+      acc[c] = __fmaf_rn(x.w, q[k].w, acc[c]);
+      const int i = 4 * (r + k * LPC);
+      if (j < columns && i < dim) *reinterpret_cast<float4*>(sp + i) = x;
+    }
+  }
+#pragma unroll
+  for (int o = 1; o < LPC; o <<= 1)
+#pragma unroll
+    for (int c = 0; c < CPL; ++c) acc[c] += __shfl_xor_sync(0xffffffffu, acc[c], o);
+#pragma unroll
+  for (int c = 0; c < CPL; ++c) {
+    const int j = j0 + c * GROUPS;
+    if (r != c % LPC || j >= columns) continue;
+    if (KIND == MATRIX_MEMORY && j == vdim) a.den[(size_t)t * H + h] = fmaxf(fabsf(acc[c]), exp_m) + 1e-6f;
+    else a.out[((size_t)t * H + h) * vdim + j] = KIND == STATE_SPACE ? __fmaf_rn(a.p2[h], v[c], acc[c]) : acc[c];
+  }
+}
+
 template <int KIND>
-int launch_gated_state(const GatedStateArgs& a, int n_entries, cudaStream_t stream) {
+int launch_gated_state(const GatedStateArgs& a, int n_entries, int max_q_len, cudaStream_t stream) {
   if (n_entries <= 0) return 0;
   if (a.dim <= 0 || a.dim > 256 || a.vdim <= 0 || a.H <= 0 || a.H > 65535 || a.rep <= 0 || a.H % a.rep || n_entries > 65535 ||
       a.taps < 1 || a.channels < 0)
     return (int)cudaErrorInvalidValue;
   const int columns = a.vdim + (KIND == MATRIX_MEMORY ? 1 : 0);
+  const uintptr_t bases = reinterpret_cast<uintptr_t>(a.q) | reinterpret_cast<uintptr_t>(a.k) | reinterpret_cast<uintptr_t>(a.state);
+  if (max_q_len == 1 && a.dim % 4 == 0 && a.ld_qkv % 4 == 0 && a.state_stride % 4 == 0 && (bases & 15) == 0) {
+#define LD(LPC, QPL, CPL)                                                                                          \
+  BSPEC_LAUNCH((gated_state_decode_kernel<KIND, LPC, QPL, CPL>),                                                   \
+               dim3((columns + GD_WARPS * (32 / LPC) * CPL - 1) / (GD_WARPS * (32 / LPC) * CPL), a.H, n_entries),  \
+               GD_WARPS * 32, 0, stream, a)
+    if (a.dim <= 32) LD(8, 1, 4);
+    else if (a.dim <= 64) LD(16, 1, 4);
+    else if (a.dim <= 128) LD(32, 1, 8);
+    else LD(32, 2, 4);
+#undef LD
+    return BSPEC_LAUNCH_CHECK();
+  }
   const dim3 grid((columns + GS_COLS - 1) / GS_COLS, a.H, n_entries);
   // few blocks (a lone prompt): 32 lanes per column, so that an SM's one block has many warps; many blocks (a decode
   // batch): 8 lanes with more rows each, and the SMs fill with blocks
@@ -322,8 +458,8 @@ int launch_gated_state(const GatedStateArgs& a, int n_entries, cudaStream_t stre
 BSPEC_API int bspec_state_space(const float* xbc, long long ld, const float* conv_in, const float* dt, long long ld_in,
                                 const float* dt_bias, const float* rate, const float* skip, float* state,
                                 long long state_stride, long long tail_off, const int* qo_indptr, const int* state_slots,
-                                const int* positions, float* out, int n_entries, int H, int groups, int dim, int vdim,
-                                int taps, cudaStream_t stream) {
+                                const int* positions, float* out, int n_entries, int max_q_len, int H, int groups,
+                                int dim, int vdim, int taps, cudaStream_t stream) {
   if (groups <= 0 || H % groups) return (int)cudaErrorInvalidValue;
   GatedStateArgs a = {};
   a.v = xbc; a.k = xbc + (size_t)H * vdim; a.q = a.k + (size_t)groups * dim; a.ld_qkv = ld;
@@ -332,7 +468,7 @@ BSPEC_API int bspec_state_space(const float* xbc, long long ld, const float* con
   a.qo_indptr = qo_indptr; a.state_slots = state_slots; a.positions = positions; a.out = out;
   a.H = H; a.rep = H / groups; a.dim = dim; a.vdim = vdim; a.channels = H * vdim + 2 * groups * dim; a.taps = taps;
   a.q_scale = 1.f;
-  return launch_gated_state<STATE_SPACE>(a, n_entries, stream);
+  return launch_gated_state<STATE_SPACE>(a, n_entries, max_q_len, stream);
 }
 
 // proj [n, ld] float32: columns q and k (H dim each), v (H vdim), and the raw gates i and f (H each) at their offsets.
@@ -340,8 +476,8 @@ BSPEC_API int bspec_state_space(const float* xbc, long long ld, const float* con
 BSPEC_API int bspec_matrix_memory(const float* proj, long long ld, int q_off, int k_off, int v_off, int i_off, int f_off,
                                   const float* i_bias, const float* f_bias, float cap, float q_scale, float* state,
                                   long long state_stride, long long m_off, const int* qo_indptr, const int* state_slots,
-                                  const int* positions, float* out, float* den, int n_entries, int H, int dim, int vdim,
-                                  cudaStream_t stream) {
+                                  const int* positions, float* out, float* den, int n_entries, int max_q_len, int H,
+                                  int dim, int vdim, cudaStream_t stream) {
   if (!(cap > 0.f)) return (int)cudaErrorInvalidValue;
   GatedStateArgs a = {};
   a.q = proj + q_off; a.k = proj + k_off; a.v = proj + v_off; a.ld_qkv = ld;
@@ -349,7 +485,7 @@ BSPEC_API int bspec_matrix_memory(const float* proj, long long ld, int q_off, in
   a.state = state; a.state_stride = state_stride; a.aux_off = m_off;
   a.qo_indptr = qo_indptr; a.state_slots = state_slots; a.positions = positions; a.out = out; a.den = den;
   a.H = H; a.rep = 1; a.dim = dim; a.vdim = vdim; a.taps = 1; a.q_scale = q_scale; a.cap = cap;
-  return launch_gated_state<MATRIX_MEMORY>(a, n_entries, stream);
+  return launch_gated_state<MATRIX_MEMORY>(a, n_entries, max_q_len, stream);
 }
 
 BSPEC_DEFINE_TRACE_SETTER(bspec_trace_set_gated_states)

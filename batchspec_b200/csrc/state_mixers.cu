@@ -247,6 +247,56 @@ scan_conv_kernel(const float* __restrict__ xz, long long ld, const void* __restr
   if (xc_run != nullptr) xc_run[(size_t)t * inner + c] = from_f32<T>(v);
 }
 
+// The same for four taps, with four channels and TT consecutive tokens per thread, for rows whose channels start on
+// 16-byte boundaries: a thread keeps its weights and the last three inputs in registers.  Each channel's arithmetic is the
+// same.
+template <typename T, int TT>
+__global__ void __launch_bounds__(256)
+scan_conv4_kernel(const float* __restrict__ xz, long long ld, const float* __restrict__ conv, const float* __restrict__ bias,
+                  const float* __restrict__ state, long long state_stride, long long tail_off,
+                  const int* __restrict__ qo_indptr, const int* __restrict__ tok_entry,
+                  const int* __restrict__ state_slots, float* __restrict__ xc, T* __restrict__ xc_run, int n, int inner) {
+  bspec::pdl_prologue(66);
+  const int t0 = blockIdx.x * TT;
+  const int c = 4 * (blockIdx.y * blockDim.x + threadIdx.x);
+  if (c >= inner) return;
+  auto row4 = [](const float* p, float (&f)[4]) {
+    const float4 v = *reinterpret_cast<const float4*>(p);
+    f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w;
+  };
+  float w[4][4], b[4], x[TT + 3][4];                         // x[u]: the input of token t0 + u - 3
+#pragma unroll
+  for (int q = 0; q < 4; ++q) row4(conv + (size_t)(c + q) * 4, w[q]);
+  row4(bias + c, b);
+#pragma unroll
+  for (int u = 0; u < TT + 3; ++u) {
+    const int t = t0 + u - 3;
+#pragma unroll
+    for (int q = 0; q < 4; ++q) x[u][q] = 0.f;
+    if (t >= 0 && t < n) row4(xz + (size_t)t * ld + c, x[u]);
+  }
+#pragma unroll
+  for (int u = 0; u < TT; ++u) {
+    const int t = t0 + u;
+    if (t >= n) break;
+    const int e = tok_entry[t], i = t - qo_indptr[e];
+    float y[4] = {b[0], b[1], b[2], b[3]};
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {                            // oldest input first
+      float v[4] = {x[u + j][0], x[u + j][1], x[u + j][2], x[u + j][3]};
+      if (i < 3 - j) row4(state + (size_t)state_slots[e] * state_stride + tail_off + (size_t)(i + j) * inner + c, v);
+#pragma unroll
+      for (int q = 0; q < 4; ++q) y[q] += w[q][j] * v[q];
+    }
+#pragma unroll
+    for (int q = 0; q < 4; ++q) y[q] = silu_f(y[q]);
+    *reinterpret_cast<float4*>(xc + (size_t)t * inner + c) = make_float4(y[0], y[1], y[2], y[3]);
+    if (xc_run != nullptr)
+#pragma unroll
+      for (int q = 0; q < 4; ++q) xc_run[(size_t)t * inner + c + q] = from_f32<T>(y[q]);
+  }
+}
+
 constexpr int SC_THREADS = 128;
 constexpr int SC_TT = 8;
 constexpr int SC_MAX_N = 256;
@@ -413,6 +463,21 @@ BSPEC_API int bspec_scan_conv(const float* xz, long long ld, const void* conv, c
                               int n, int inner, int taps, cudaStream_t stream) {
   if (n <= 0) return 0;
   if (inner <= 0 || taps < 1) return (int)cudaErrorInvalidValue;
+  if (taps == 4 && inner % 4 == 0 && ld % 4 == 0 && tail_off % 4 == 0 && state_stride % 4 == 0 && w_dtype == BSPEC_F32 &&
+      ((reinterpret_cast<uintptr_t>(xz) | reinterpret_cast<uintptr_t>(state) | reinterpret_cast<uintptr_t>(bias) |
+        reinterpret_cast<uintptr_t>(conv) | reinterpret_cast<uintptr_t>(xc)) & 15) == 0) {
+    const int quads = inner / 4, per = quads >= 128 ? 128 : ((quads + 31) / 32) * 32;
+    const bool many = (long long)n * quads >= 1ll << 20;     // a prompt: enough threads also with eight tokens each
+    const dim3 grid4(many ? (n + 7) / 8 : n, (quads + per - 1) / per);
+    if (grid4.y > 65535) return (int)cudaErrorInvalidConfiguration;
+#define LC(T, TT) BSPEC_LAUNCH((scan_conv4_kernel<T, TT>), grid4, per, 0, stream, xz, ld, (const float*)conv, (const float*)bias, state, \
+                               state_stride, tail_off, qo_indptr, tok_entry, state_slots, xc, \
+                               run_dtype == BSPEC_F32 ? (T*)nullptr : (T*)xc_run, n, inner)
+    if (run_dtype == BSPEC_F32) { if (many) LC(float, 8); else LC(float, 1); }
+    else { if (many) LC(__nv_bfloat16, 8); else LC(__nv_bfloat16, 1); }
+#undef LC
+    return BSPEC_LAUNCH_CHECK();
+  }
   const int threads = inner >= 256 ? 256 : ((inner + 31) / 32) * 32;
   const dim3 grid(n, (inner + threads - 1) / threads);
   if (grid.y > 65535) return (int)cudaErrorInvalidConfiguration;

@@ -81,11 +81,11 @@ _SIGNATURES = {
     "bspec_gated_rmsnorm": [c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_int, c_longlong, c_int, c_int, c_int,
                             c_float, c_int, c_void_p, c_float, c_void_p],
     "bspec_state_space": [c_void_p, c_longlong, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p,
-                          c_longlong, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
+                          c_longlong, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
                           c_int, c_int, c_void_p],
     "bspec_matrix_memory": [c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float, c_float,
                             c_void_p, c_longlong, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
-                            c_int, c_int, c_void_p],
+                            c_int, c_int, c_int, c_void_p],
     "bspec_rope_kv_append": [c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p,
                              c_void_p, c_void_p, c_void_p, c_int, c_int, c_longlong, c_void_p],
     "bspec_rope_inplace": [c_void_p, c_int, c_int, c_longlong, c_int, c_int, c_void_p, c_int, c_int, c_void_p, c_float,
@@ -1054,7 +1054,7 @@ def state_space(xbc: torch.Tensor, conv_in: torch.Tensor, dt_raw: torch.Tensor, 
     _check(load_library().bspec_state_space(
         xbc.data_ptr(), xbc.stride(0), conv_in.data_ptr(), dt_raw.data_ptr(), conv_in.stride(0), dt_bias.data_ptr(),
         rate.data_ptr(), skip.data_ptr(), state.data_ptr(), state.stride(0), int(tail_off), ctx.qo_indptr.data_ptr(),
-        ctx.state_slots.data_ptr(), ctx.positions.data_ptr(), out.data_ptr(), ctx.n_entries, n_heads, groups, n_state, v_dim,
+        ctx.state_slots.data_ptr(), ctx.positions.data_ptr(), out.data_ptr(), ctx.n_entries, ctx.max_q_len, n_heads, groups, n_state, v_dim,
         taps, _stream()), "state_space")
     return out
 
@@ -1082,7 +1082,7 @@ def matrix_memory(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, i_off:
     _check(load_library().bspec_matrix_memory(
         proj.data_ptr(), proj.stride(0), int(q_off), int(k_off), int(v_off), int(i_off), int(f_off), i_bias.data_ptr(),
         f_bias.data_ptr(), float(cap), float(q_scale), state.data_ptr(), state.stride(0), int(m_off), ctx.qo_indptr.data_ptr(),
-        ctx.state_slots.data_ptr(), ctx.positions.data_ptr(), out.data_ptr(), den.data_ptr(), ctx.n_entries, n_heads, dim,
+        ctx.state_slots.data_ptr(), ctx.positions.data_ptr(), out.data_ptr(), den.data_ptr(), ctx.n_entries, ctx.max_q_len, n_heads, dim,
         v_dim, _stream()), "matrix_memory")
     return out, den
 

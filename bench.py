@@ -946,7 +946,173 @@ def podizen_kernels_alone(z, pk, iters=20):
     return out
 
 
+GUVOLIX_SIZES = {
+    # the Podizen sizes (width, heads, experts, window) with four first tokens kept, a state space of 64 heads of 64 values
+    # per 2,048 of width and 128 states, a matrix memory with as many heads as the attention, sixteen identity experts
+    "w2048": dict(PODIZEN_SIZES["w2048"], first=4, ssd_heads=64, ssd_vdim=64, ssd_state=128, ssd_groups=8, conv=4, identity=16),
+    "w4096": dict(PODIZEN_SIZES["w4096"], first=4, ssd_heads=128, ssd_vdim=64, ssd_state=128, ssd_groups=8, conv=4, identity=16),
+}
+
+
+def guvolix_config_json(z, layers, vocab=32000):
+    """Attention beside a state space and attention beside a matrix memory in turn; the first layer's feed-forward is the
+    dense one, the others are routed with identity experts and a gated shared one (as in the Finolix model of equal size)."""
+    hd = z["dim_a"]
+    left = lambda mask, scaling: dict(heads=z["heads"], kv_heads=z["kv_heads"], dim=hd, vdim=hd, scale=hd ** -0.5, mask=mask,
+                                      rot=dict(base=500000.0, dims=hd, scaling=scaling))
+    ssd = dict(left=left(dict(size=z["window"], keep_first=z["first"]), dict(factor=4.0)),
+               right=dict(heads=z["ssd_heads"], vdim=z["ssd_vdim"], state=z["ssd_state"], groups=z["ssd_groups"], conv=z["conv"],
+                          norm_groups=z["ssd_groups"]))
+    mem = dict(left=left(dict(size=z["window"]), dict(factor=8.0, low=1.0, high=4.0, original=8192)),
+               right=dict(heads=z["heads"], dim=hd, vdim=hd, gate_cap=15.0), left_scale=0.7, right_scale=0.7)
+    moe = dict(kind="moe", expert=dict(ff=z["expert_ff"]), shared=dict(ff=2 * z["expert_ff"]),
+               router=dict(experts=z["experts"], identity=z["identity"], top=z["top"]))
+    dense = dict(kind="dense", ff=z["dense_ff"])
+    return dict(architecture="Guvolix", vocab=vocab, width=z["width"], norm=dict(eps=1e-5), embedding=dict(scale=1.0),
+                layers=[dict(type=("parallel", "parallel_2")[i % 2], mixer=(ssd, mem)[i % 2], mlp=dense if i == 0 else moe)
+                        for i in range(layers)])
+
+
+def guvolix_kernels_alone(z, pk, iters=20):
+    """The design's own kernels by themselves, each beside its like at equal sizes: attention with first tokens kept behind
+    the window and a sink, against the same kernels with the window alone (a prompt of 4,096 tokens: FLOP/s over the visible
+    pairs; a decode step of 64 requests x 4,096 tokens: bytes of the visible keys and values); the join of two branches and
+    the norm, and with a normed pair, against add + RMS norm; the two gated recurrences against the lightning recurrence with
+    the state space's and with the matrix memory's sizes (prompts: float32 FLOP/s of update and read-out; decode: bytes of
+    state); the short convolution; the output norms; routed experts with identity experts and a gated shared one against
+    Podizen's; the exact gelu in a decode step's product against the square of relu."""
+    import torch
+    from itertools import accumulate
+    from types import SimpleNamespace
+    from batchspec_b200.kernels import ops
+    from batchspec_b200.parts.base import FEED_FORWARDS, PartSpec, Runtime, build_part
+    ops.require("state_mixers", "gated_states", "joins", "moe")
+    dev = "cuda:0"
+    Hq, G, hd, ps, W, d = z["heads"], z["kv_heads"], z["dim_a"], 16, z["window"], z["width"]
+    out = {}
+    by = lambda ms, nbytes: dict(ms=round(ms, 4), gbs=round(nbytes / ms / 1e6, 1), frac_of_measured=round(nbytes / ms / 1e6 / pk["hbm_gbs"], 4))
+    i32 = lambda x: torch.as_tensor(x, dtype=torch.int32, device=dev)
+
+    def step_ctx(q_lens, ctx_len):
+        n, B = sum(q_lens), len(q_lens)
+        per = -(-ctx_len // ps)
+        ctx = SimpleNamespace(qo_indptr=i32([0] + list(accumulate(q_lens))), n_entries=B, n_tokens=n, max_q_len=max(q_lens),
+                              positions=i32(torch.cat([torch.arange(ctx_len - q, ctx_len) for q in q_lens])),
+                              tok_entry=i32(torch.cat([torch.full((q,), i) for i, q in enumerate(q_lens)])),
+                              max_kv_len=ctx_len, kv_len=i32([ctx_len] * B), state_slots=i32(list(range(B))),
+                              extras={"min_q_len": min(q_lens)})
+        tables = SimpleNamespace(kv_indptr=torch.arange(B + 1, dtype=torch.int32, device=dev) * per,
+                                 kv_indices=torch.randperm(B * per, device=dev).to(torch.int32), page_size=ps)
+        return ctx, tables, n, B, per
+
+    sinks = torch.linspace(-1.0, 1.0, Hq, device=dev)
+    for name, q_lens, ctx_len in (("prompt_4096", [4096], 4096), ("decode_64x4096", [1] * 64, 4096)):
+        ctx, tables, n, B, per = step_ctx(q_lens, ctx_len)
+        cache = torch.randn(B * per, 2, ps * G * hd, device=dev).bfloat16()
+        q = torch.randn(n, Hq * hd, device=dev).bfloat16()
+        o = torch.empty(n, Hq * hd, device=dev, dtype=torch.bfloat16)
+        kept = dict(pooled=(-z["first"], cache, tables), sink=sinks, sink_l2=ops.sink_table(sinks))
+        for label, kw, k in (("kept_sink", kept, z["first"]), ("window", {}, 0)):
+            ctx.extras = {"min_q_len": min(q_lens)}
+            ms = _time(lambda: ops.paged_attention(q, o, cache, ctx, tables, Hq, G, hd, hd ** -0.5, W, **kw), iters)
+            pairs = sum(min(p + 1, W) + min(k, max(0, p + 1 - W)) for p in range(ctx_len - q_lens[0], ctx_len)) * len(q_lens)
+            if name.startswith("prompt"):
+                flops = 4.0 * Hq * hd * pairs
+                out[f"attention_{name}_{label}"] = dict(ms=round(ms, 4), tflops=round(flops / ms / 1e9, 1),
+                                                        frac_of_measured=round(flops / ms / 1e9 / pk["bf16_tflops"], 4))
+            else:
+                out[f"attention_{name}_{label}"] = by(ms, pairs * 2 * G * hd * 2)
+        del cache, q, o
+    for n in (4096, 64):
+        x, y, y2, y3 = torch.randn(n, d, device=dev), *(torch.randn(n, d, device=dev).bfloat16() for _ in range(3))
+        w = torch.ones(d, device=dev)
+        o = torch.empty(n, d, device=dev, dtype=torch.bfloat16)
+        join = dict(dst=x, out=o, norm_w=w, eps=1e-5)
+        ms = _time(lambda: ops.branch_join(x, ops.BranchSum(y, y2), **join), iters)
+        out[f"branch_join_two_{n}"] = by(ms, n * d * (8 + 4 + 2))
+        ms = _time(lambda: ops.branch_join(x, ops.BranchSum(ops.NormedPair(y, y2, w, w, 1e-5), y3), **join), iters)
+        out[f"branch_join_pair_and_one_{n}"] = by(ms, n * d * (8 + 6 + 2))
+        ms = _time(lambda: ops.add_rmsnorm(x, y, w, 1e-5, o, 1.0, True), iters)
+        out[f"add_rmsnorm_{n}"] = by(ms, n * d * (8 + 2 + 2))
+    # the recurrences, each beside the lightning recurrence of the same heads and sizes
+    Hs, V, N, Gs, taps = z["ssd_heads"], z["ssd_vdim"], z["ssd_state"], z["ssd_groups"], z["conv"]
+    I, C = Hs * V, Hs * V + 2 * Gs * N
+    H, dk, dv = Hq, hd, hd
+    conv_w, conv_b = torch.randn(C, taps, device=dev) * 0.3, torch.zeros(C, device=dev)
+    per_head = lambda k, lo, hi: torch.linspace(lo, hi, k, device=dev)
+    for name, q_lens in (("prompt_2048", [2048]), ("prompt_8x2048", [2048] * 8), ("decode_64", [1] * 64), ("decode_256", [1] * 256)):
+        ctx, _, n, B, _ = step_ctx(q_lens, q_lens[0])
+        decode = name.startswith("decode")
+        proj = torch.randn(n, I + C + Hs, device=dev)
+        xbc, dt = proj[:, I:I + C], proj[:, I + C:]
+        tail = I * N
+        state = torch.zeros(B, tail + (taps - 1) * C, device=dev)
+        ms = _time(lambda: ops.scan_conv(xbc, conv_w, conv_b, state, tail, ctx, C, taps), iters)
+        rec = dict(conv=by(ms, n * C * 8))
+        xc, _ = ops.scan_conv(xbc, conv_w, conv_b, state, tail, ctx, C, taps)
+        args = (per_head(Hs, -4.0, -1.0), per_head(Hs, 0.02, 8.0), per_head(Hs, 0.5, 1.5), state, tail, ctx, Hs, Gs, N, V, taps)
+        ms = _time(lambda: ops.state_space(xc, xbc, dt, *args), iters)
+        y = ops.state_space(xc, xbc, dt, *args)
+        norm_w = torch.ones(I, device=dev)
+        rec["norm"] = by(_time(lambda: ops.gated_rmsnorm(y, proj[:, :I], norm_w, 1e-5, Gs, I // Gs, torch.bfloat16, gate_first=True), iters),
+                         n * I * (4 + 4 + 2))
+        del state, xc, y, proj
+        ml = torch.randn(n, 2 * H * dk + 2 * H * dv + 2 * H, device=dev)
+        m_off = H * (dv + 1) * dk
+        mstate = torch.zeros(B, m_off + ops.MATRIX_MEMORY_RECORD * H, device=dev)
+        ld = ml.shape[1]
+        ib, fb = per_head(H, -1.0, 0.0), per_head(H, 2.0, 7.0)
+        run = lambda: ops.matrix_memory(ml, 0, H * dk, 2 * H * dk, ld - 2 * H, ld - H, ib, fb, 15.0, dk ** -0.5, mstate, m_off, ctx, H, dk, dv)
+        ms_m = _time(run, iters)
+        y, den = run()
+        g_off, norm_w = 2 * H * dk + H * dv, torch.ones(H * dv, device=dev)
+        rec["head_norm"] = by(_time(lambda: ops.gated_rmsnorm(y, ml[:, g_off:g_off + H * dv], norm_w, 1e-5, H, dv, torch.bfloat16, "sigmoid",
+                                                              den=den), iters), n * H * dv * (4 + 4 + 2))
+        rec["like_head_norm"] = by(_time(lambda: ops.gated_rmsnorm(y, ml[:, g_off:g_off + H * dv], None, 1e-5, H, dv, torch.bfloat16), iters),
+                                   n * H * dv * (4 + 4 + 2))
+        del mstate, y, den
+
+        def lightning(heads, k, v):
+            p = torch.randn(n, heads * (2 * k + v), device=dev)
+            st = torch.zeros(B, heads * k * v, device=dev)
+            dec = per_head(heads, 0.97, 0.9995)
+            return _time(lambda: ops.lightning_recurrence(p, 0, heads * k, 2 * heads * k, dec, st, ctx, heads, k, v, activation=None), iters)
+        for label, t, heads, k, v in (("state_space", ms, Hs, N, V), ("like_state_space", lightning(Hs, N, V), Hs, N, V),
+                                      ("matrix_memory", ms_m, H, dk, dv), ("like_matrix_memory", lightning(H, dk, dv), H, dk, dv)):
+            if decode:
+                rec[label] = by(t, B * heads * k * v * 4 * 2)
+            else:
+                rec[label] = dict(ms=round(t, 4), fp32_tflops=round(5.0 * n * heads * k * v / t / 1e9, 2))
+        out[f"recurrence_{name}"] = rec
+        del ml
+    rt = Runtime(torch.bfloat16, torch.device(dev))
+    E, top, ff = z["experts"], z["top"], z["expert_ff"]
+    for label, kw in (("routed_identity_gated_shared", dict(correction=True, identity=z["identity"], shared_gate=True)),
+                      ("routed_shared", dict(n_groups=z["groups"], keep_groups=z["keep"]))):
+        part = build_part(FEED_FORWARDS, PartSpec("routed_glu", dict(dim=d, intermediate=ff, n_experts=E, top=top, bias=False,
+                                                                     scores="softmax", shared=2 * ff, **kw)), rt)
+        part.bind({k: (torch.randn(p.shape, device=dev) * 0.02).bfloat16() for k, p in part.param_specs().items()})
+        routed = top * E / (E + (z["identity"] if "identity" in kw else 0))       # of a token's choices, with random weights
+        for n in (4096, 64):
+            x = torch.randn(n, d, device=dev).bfloat16()
+            ms = _time(lambda: part.forward(x, None), iters)
+            flops = 2.0 * n * 3 * d * (routed * ff + 2 * ff)
+            rec = dict(ms=round(ms, 4), tflops=round(flops / ms / 1e9, 1), frac_of_measured=round(flops / ms / 1e9 / pk["bf16_tflops"], 4))
+            if n == 64:                     # decode: the weights of the experts that were chosen are read once
+                rec["weights_frac_of_measured"] = round((E * ff + 2 * ff) * 3 * d * 2 / ms / 1e6 / pk["hbm_gbs"], 4)
+            out[f"{label}_{n}"] = rec
+        del part
+    F = z["dense_ff"]
+    for n in (8, 4096):
+        x, w = torch.randn(n, d, device=dev).bfloat16(), (torch.randn(F, d, device=dev) * 0.02).bfloat16()
+        for act in ("gelu", "relu2"):
+            ms = _time(lambda: ops.linear_act(x, w, act), iters)
+            out[f"up_{act}_{n}"] = by(ms, F * d * 2) if n == 8 else dict(ms=round(ms, 4), frac_of_measured=round(2.0 * n * F * d / ms / 1e9 / pk["bf16_tflops"], 4))
+    return out
+
+
 DESIGNS = {
+    "guvolix": (GUVOLIX_SIZES, guvolix_config_json, guvolix_kernels_alone, "kernels_alone"),
     "podizen": (PODIZEN_SIZES, podizen_config_json, podizen_kernels_alone, "kernels_alone"),
     "finolix": (FINOLIX_SIZES, finolix_config_json, finolix_kernels_alone, "kernels_alone"),
     "tokolorn": (TOKOLORN_SIZES, tokolorn_config_json, tokolorn_kernels_alone, "kernels_alone"),
@@ -976,6 +1142,8 @@ def run_design(a) -> int:
             models.append(("vabanex", vabanex_config_json(z, layers)))
         if a.design == "podizen":         # its closest models: the same kinds of mixers, and routed gated experts
             models += [("tokolorn", tokolorn_config_json(dict(z, dim=z["dim_a"]), layers)), ("finolix", finolix_config_json(z, layers))]
+        if a.design == "guvolix":         # its closest models: recurrences beside attention, and routed gated experts
+            models += [("podizen", podizen_config_json(z, layers)), ("finolix", finolix_config_json(z, layers))]
         for label, cj in models:
             cfg = config_from_json_dict(cj)
             eng = Engine(dtype="bfloat16", device="cuda:0")
@@ -1057,7 +1225,7 @@ def main() -> int:
     ap.add_argument("--skip-points", action="store_true", help="only the headline batch (no prefill, b1, b64, e2e)")
     ap.add_argument("--skip-workloads", action="store_true",
                     help="leave out e2e at batch 64 and the 3B / long-context workloads (about a minute)")
-    ap.add_argument("--design", default=None, choices=["vabanex", "lupusun", "tokolorn", "finolix", "podizen"],
+    ap.add_argument("--design", default=None, choices=["vabanex", "lupusun", "tokolorn", "finolix", "podizen", "guvolix"],
                     help="instead of the headline workload: this design at real layer sizes beside the Llama model of equal size")
     a = ap.parse_args()
     if a.impl == "reference":

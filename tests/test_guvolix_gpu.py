@@ -434,6 +434,28 @@ def test_matrix_memory_over_portions_and_reused_slots(ops, dtype, Hh, dk, dv, ca
     _mixer_over_steps(part, dtype, d, lambda h: P.mlstm(h, named, m, eps), dk, w)
 
 
+@pytest.mark.parametrize("run", [None, torch.bfloat16])
+@pytest.mark.parametrize("lens,C,taps", [([1, 2, 3, 4, 70, 1, 5, 30], 96, 4), ([1, 2, 3, 4, 700, 1, 5, 600], 4096, 4), ([7, 1, 2], 30, 4),
+                                         ([9, 1], 64, 1), ([2, 1, 12], 64, 6)])
+def test_short_convolution_of_unequal_portions(ops, run, lens, C, taps):
+    """Portions shorter and longer than the taps, each after inputs of its own in a scrambled slot, in rows wider than the
+    channels; the form with eight tokens per thread gives what the plain one gives."""
+    g, n = _gen(C), sum(lens)
+    xz = torch.randn(n, C + 8, device=DEV, generator=g)
+    w, b = torch.randn(C, taps, device=DEV, generator=g), torch.randn(C, device=DEV, generator=g)
+    state = torch.randn(9, 4 + taps * C, device=DEV, generator=g)
+    slots = torch.randperm(9, generator=torch.Generator().manual_seed(1))[:len(lens)].tolist()
+    got, got_run = ops.scan_conv(xz[:, 4:4 + C], w, b, state, 4, _step_ctx(lens, slots, [0] * len(lens)), C, taps, run)
+    at = 0
+    for k, slot in zip(lens, slots):
+        before = state[slot, 4:4 + (taps - 1) * C].view(taps - 1, C)
+        x = torch.cat([before, xz[at:at + k, 4:4 + C]]).double().cpu()
+        want = P.silu(P.causal_conv(x, w.cpu(), b.cpu())[taps - 1:])
+        assert (got[at:at + k].double().cpu() - want).abs().max() <= 1e-5 * (1 + want.abs().max())
+        at += k
+    assert got_run is got if run is None else torch.equal(got_run, got.to(run))
+
+
 def test_state_space_keeps_its_digits_over_a_long_prompt(ops):
     """3,000 tokens with decays from 1 - 1e-5 to 0.2 per step, in portions and then one by one, against the plain one."""
     g = _gen(1)
