@@ -438,15 +438,16 @@ int launch_gated_state(const GatedStateArgs& a, int n_entries, int max_q_len, cu
     return BSPEC_LAUNCH_CHECK();
   }
   const dim3 grid((columns + GS_COLS - 1) / GS_COLS, a.H, n_entries);
-  // few blocks (a lone prompt): 32 lanes per column, so that an SM's one block has many warps; many blocks (a decode
-  // batch): 8 lanes with more rows each, and the SMs fill with blocks
-  const bool few = (long long)grid.x * grid.y * grid.z < 4 * 148;
+  // Lanes per column, by the sizes alone: fewer lanes share more of what they read from shared memory, more lanes have a
+  // shorter chain per token.  (Measured on prompts of 2,048 tokens, 128 to 4,096 blocks, 8 / 16 / 32 lanes: 16 lanes are
+  // best for the state space from 128 blocks up, 8 for the matrix memory.)
+  constexpr bool WIDE = KIND == STATE_SPACE;
 #define LG(NR, L) \
-  BSPEC_LAUNCH_SERIALIZED((gated_state_kernel<NR, L, KIND>), grid, GS_COLS * L + 32, 0, stream, a)
+  BSPEC_LAUNCH_SERIALIZED((gated_state_kernel<NR, L, KIND>), grid, GS_COLS * (L) + 32, 0, stream, a)
   if (a.dim <= 32) LG(4, 8);
-  else if (a.dim <= 64) { if (few) LG(4, 16); else LG(8, 8); }
-  else if (a.dim <= 128) { if (few) LG(4, 32); else LG(16, 8); }
-  else { if (few) LG(8, 32); else LG(32, 8); }
+  else if (a.dim <= 64) LG(WIDE ? 4 : 8, WIDE ? 16 : 8);
+  else if (a.dim <= 128) LG(WIDE ? 8 : 16, WIDE ? 16 : 8);
+  else LG(16, 16);
 #undef LG
   return BSPEC_LAUNCH_CHECK();
 }
