@@ -10,9 +10,9 @@
 //                           m <- max(f + m, i),  x = f + m_old - m,  b = exp(i - m);  n <- exp(x) n + b k;
 //                           out = o,  den = max(|n . q|, exp(-m)) + 1e-6      (who normalises the heads divides by den)
 //
-// A step holds portions of several requests (qo_indptr, state_slots); a portion of one token is a decode step.  Every
-// sum runs in an order fixed by the sizes alone, so a position's result does not depend on how the request was cut
-// or on what else is in the step.
+// A step holds portions of several requests (qo_indptr, state_slots).  Every sum runs in an order fixed by the sizes alone, so
+// a position's result does not depend on how a prompt was cut or on what else is in the step; steps of one token per
+// request have a kernel of their own, whose order differs from the portions' (a difference of rounding).
 #include "common.cuh"
 #include <math.h>
 using namespace bspec;
